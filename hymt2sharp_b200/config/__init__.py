@@ -3,8 +3,11 @@ from .hunyuan_dense import HunyuanDenseConfig
 from .pemezen import PemezenConfig
 from .novunex import NovunexConfig
 from .rutetar import RutetarConfig
+from .pulenex import PulenexConfig
+from .sosepel import SosepelConfig
 from .registry import (Architecture, register_architecture, get_architecture,
                        known_architectures, load_config)
 
 __all__ = ["ConfigError", "ConfigReader", "read_config_json", "architecture_name", "HunyuanDenseConfig", "PemezenConfig", "NovunexConfig", "RutetarConfig",
+           "PulenexConfig", "SosepelConfig",
            "Architecture", "register_architecture", "get_architecture", "known_architectures", "load_config"]

@@ -16,6 +16,12 @@
 // cut into chunks of split_keys (a constant, so the cut depends on nothing but
 // the key's own index); each chunk's block writes an unnormalised partial and
 // `attention_merge_kernel` folds the partials in chunk order.
+//
+// Beyond that form: scores may be capped, cap * tanh(score / cap); a query's scores may be multiplied by a temperature of its
+// position, 1 + coef * ln(floor((p + 1) / every) + 1); and a head may hold several maps, each with query and key entries of
+// its own (side by side, map after map, in the query's and in the key's row) over the same values: every map's output is a
+// row of its own, [T, nh, maps, dv] in float32.  The two maps of differential attention are combined by
+// `diff_combine_kernel`: o = a1 - lambda * a2, then o / sqrt(mean(o^2) + eps) * factor over the head's dv entries.
 #include "common.cuh"
 
 namespace {
@@ -40,6 +46,10 @@ struct AttnParams {
     float scale;
     int* status;            // may be null; [0] = 2 when a row is longer than max_splits * split_keys covers
     int sink;               // the softmax has one more term in its denominator, of score 0 and without a value
+    int maps;               // maps a head: rows of q and of the keys hold maps * d entries, outputs maps rows a head
+    float softcap;          // > 0: scores become softcap * tanh(score / softcap)
+    float temp_coef;        // != 0: the temperature of the queries
+    int temp_every;
 };
 
 template <typename T, int NACC>
@@ -62,7 +72,8 @@ attention_simt_kernel(AttnParams p) {
     const int tile_tok0 = blockIdx.x * p.tokens_per_tile;
     if (tile_tok0 >= T_b) return;
     const int g = p.nh / p.nkv;
-    const int kvh = blockIdx.y / p.head_chunks, chunk = blockIdx.y % p.head_chunks;
+    const int kvh = blockIdx.y / (p.head_chunks * p.maps), map = blockIdx.y / p.head_chunks % p.maps, chunk = blockIdx.y % p.head_chunks;
+    const int kd = p.maps * d;   // entries of a key's row
 
     const int tid = threadIdx.x, r = tid / LANES_PER_ROW, c = tid % LANES_PER_ROW;
     const int row_tok = tile_tok0 + r / p.heads_per_tile;         // index among the row's new tokens
@@ -71,6 +82,8 @@ attention_simt_kernel(AttnParams p) {
     const int head = kvh * g + head_in_group;
     const int row_pos = kv_len - T_b + row_tok;                   // absolute position of the query
     const int row_lo = p.window > 0 ? max(0, row_pos - p.window + 1) : 0;
+    float row_scale = p.scale;
+    if (p.temp_coef != 0.f) row_scale *= 1.0f + p.temp_coef * logf((float)((row_pos + 1) / p.temp_every + 1));
 
     // key range of the whole tile
     const int last_tok = min(T_b, tile_tok0 + p.tokens_per_tile) - 1;
@@ -89,7 +102,7 @@ attention_simt_kernel(AttnParams p) {
         const int tk = tile_tok0 + rr / p.heads_per_tile;
         const int hg = chunk * p.heads_per_tile + rr % p.heads_per_tile;
         const bool ok = rr < p.tokens_per_tile * p.heads_per_tile && tk < T_b && hg < g;
-        Qs[i] = ok ? to_float(((const T*)p.q)[((size_t)(tok0 + tk) * p.nh + kvh * g + hg) * d + x]) : 0.f;
+        Qs[i] = ok ? to_float(((const T*)p.q)[(((size_t)(tok0 + tk) * p.nh + kvh * g + hg) * p.maps + map) * d + x]) : 0.f;
     }
 
     float acc[NACC];
@@ -102,13 +115,13 @@ attention_simt_kernel(AttnParams p) {
         __syncthreads();
         // a tile of 32 keys lies inside one block (block_tokens is a multiple of 32)
         const int block = table[k0 / p.block_tokens];
-        const size_t base = (((size_t)block * p.nkv + kvh) * p.block_tokens + (k0 % p.block_tokens)) * d;
+        const size_t base = (((size_t)block * p.nkv + kvh) * p.block_tokens + (k0 % p.block_tokens)) * kd + map * d;
         const T* kp = (const T*)p.k_cache + base;
         const int valid = min(KEY_TILE, kv_len - k0);
         for (int i = tid; i < KEY_TILE * d; i += blockDim.x) {
             const int j = i / d, x = i - j * d;
             const bool ok = j < valid && block >= 0;
-            Ks[j * (d + 1) + x] = ok ? to_float(kp[i]) : 0.f;
+            Ks[j * (d + 1) + x] = ok ? to_float(kp[(size_t)j * kd + x]) : 0.f;
         }
         if (!p.v_from_k) {
             const T* vp = (const T*)p.v_cache + (((size_t)block * p.nkv + kvh) * p.block_tokens + (k0 % p.block_tokens)) * dv;
@@ -129,7 +142,9 @@ attention_simt_kernel(AttnParams p) {
             const float* kr = Ks + j * (d + 1);
             for (int x = 0; x < d; x++) dot = fmaf(qr[x], kr[x], dot);
             const bool visible = row_ok && key >= row_lo && key <= row_pos && key >= key_begin && key < key_end;
-            s[kk] = visible ? dot * p.scale : -INFINITY;
+            float sc = dot * row_scale;
+            if (p.softcap > 0.f) sc = p.softcap * tanhf(sc / p.softcap);
+            s[kk] = visible ? sc : -INFINITY;
             tile_max = fmaxf(tile_max, s[kk]);
         }
 #pragma unroll
@@ -165,7 +180,7 @@ attention_simt_kernel(AttnParams p) {
     }
 
     if (!row_ok) return;
-    const size_t row_index = (size_t)(tok0 + row_tok) * p.nh + head;
+    const size_t row_index = ((size_t)(tok0 + row_tok) * p.nh + head) * p.maps + map;
     if (p.split_keys > 0) {
         float* pa = p.part_acc + (row_index * p.max_splits + split) * dv;
 #pragma unroll
@@ -187,11 +202,12 @@ attention_simt_kernel(AttnParams p) {
             l = l * up + expf(-M);
         }
         const float inv = l > 0.f ? up / l : 0.f;
-        T* o = (T*)p.out + row_index * dv;
 #pragma unroll
         for (int i = 0; i < NACC; i++) {
             const int x = c + i * LANES_PER_ROW;
-            if (x < dv) o[x] = from_float<T>(acc[i] * inv);
+            if (x >= dv) continue;
+            if (p.maps > 1) ((float*)p.out)[row_index * dv + x] = acc[i] * inv;   // (several maps: combined in float32 afterwards)
+            else ((T*)p.out)[row_index * dv + x] = from_float<T>(acc[i] * inv);
         }
     }
 }
@@ -203,8 +219,8 @@ inline int merge_threads(int dv) { return dv > 256 ? 256 : (dv > 128 ? 128 : 64)
 // out[row] = sum_s acc_s * exp(m_s - M) / sum_s l_s * exp(m_s - M), chunks in index order.
 template <typename T>
 __global__ void attention_merge_kernel(AttnParams p, int total_tokens) {
-    const int row = blockIdx.x;  // token * nh + head
-    const int t = row / p.nh;
+    const int row = blockIdx.x;  // (token * nh + head) * maps + map
+    const int t = row / (p.nh * p.maps);
     // the batch row of token t: cu_seqlens is short, a linear scan is enough
     int b = 0;
     while (p.cu_seqlens[b + 1] <= t) b++;
@@ -264,7 +280,34 @@ __global__ void attention_merge_kernel(AttnParams p, int total_tokens) {
     }
 }
 
+// out[t, h] = unit_rms(a[t, h, 0] - lambda * a[t, h, 1]) * factor over dv entries; a warp a (token, head)
+template <typename TO>
+__global__ void __launch_bounds__(128)
+diff_combine_kernel(TO* __restrict__ out, const float* __restrict__ a, long rows, int dv, float lambda, float eps, float factor) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const long row = (long)blockIdx.x * 4 + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31;
+    if (row >= rows) return;
+    const float* a1 = a + (size_t)row * 2 * dv;
+    const float* a2 = a1 + dv;
+    float ss = 0.f;
+    for (int x = lane; x < dv; x += 32) { const float o = fmaf(-lambda, a2[x], a1[x]); ss = fmaf(o, o, ss); }
+    const float scale = factor / sqrtf(warp_sum(ss) / (float)dv + eps);
+    for (int x = lane; x < dv; x += 32) out[(size_t)row * dv + x] = from_float<TO>(fmaf(-lambda, a2[x], a1[x]) * scale);
+}
+
 }  // namespace
+
+HYMT2_API int hymt2_diff_combine(void* out, int out_dtype, const float* a, int tokens, int nh, int dv, float lambda, float eps, float factor,
+                                 cudaStream_t stream) {
+    if (tokens == 0) return HYMT2_OK;
+    HYMT2_REQUIRE(tokens > 0 && nh > 0 && dv > 0, "diff_combine: bad sizes");
+    const long rows = (long)tokens * nh;
+    HYMT2_DISPATCH_DTYPE(out_dtype, TO, launch_pdl(diff_combine_kernel<TO>, dim3((unsigned)((rows + 3) / 4)), dim3(128), 0, stream, (TO*)out, a,
+                                                   rows, dv, lambda, eps, factor));
+    return hymt2_check_launch("diff_combine");
+}
 
 // The merge alone, for other kernels that write partials in the same layout
 // (part_acc [token, head, split, d], part_ml [token, head, split, (max, sum)]).
@@ -274,7 +317,7 @@ int hymt2_attention_merge_launch(void* out, int dtype, const int* cu_seqlens, co
     AttnParams p{};
     p.status = status;
     p.out = out; p.cu_seqlens = cu_seqlens; p.slot_ids = slot_ids; p.kv_lens = kv_lens;
-    p.part_acc = part_acc; p.part_ml = part_ml; p.nh = nh; p.d = d; p.dv = d; p.window = window;
+    p.part_acc = part_acc; p.part_ml = part_ml; p.nh = nh; p.d = d; p.dv = d; p.window = window; p.maps = 1;
     p.split_keys = split_keys; p.max_splits = max_splits;
     HYMT2_DISPATCH_DTYPE(dtype, T, (attention_merge_kernel<T><<<tokens * nh, merge_threads(d), 0, stream>>>(p, tokens)));
     return hymt2_check_launch("attention_merge");
@@ -294,7 +337,8 @@ static int attention_simt_general(void* out, const void* q, const void* k_cache,
                                   const int* cu_seqlens, const int* slot_ids, const int* kv_lens,
                                   int batch, int tokens, int max_new_tokens, int nh, int nkv, int d, int dv,
                                   float scale, int window, int split_keys, int max_splits,
-                                  float* part_acc, float* part_ml, cudaStream_t stream, int* status, int sink = 0) {
+                                  float* part_acc, float* part_ml, cudaStream_t stream, int* status, int sink = 0,
+                                  int maps = 1, float softcap = 0.f, float temp_coef = 0.f, int temp_every = 1) {
     if (tokens == 0 || batch == 0) return HYMT2_OK;
     HYMT2_REQUIRE(batch > 0 && tokens > 0 && nh > 0 && nkv > 0, "attention: bad sizes");
     HYMT2_REQUIRE(nh % nkv == 0, "attention: %d heads are not a multiple of %d kv heads", nh, nkv);
@@ -319,8 +363,11 @@ static int attention_simt_general(void* out, const void* q, const void* k_cache,
     p.scale = scale;
     p.status = status;
     p.sink = sink;
+    HYMT2_REQUIRE(maps >= 1 && (maps == 1 || v_cache) && softcap >= 0.f && temp_every > 0, "attention: %d maps, a cap of %g, a temperature every %d positions",
+                  maps, (double)softcap, temp_every);
+    p.maps = maps; p.softcap = softcap; p.temp_coef = temp_coef; p.temp_every = temp_every;
     const size_t smem = sizeof(float) * ((size_t)ROWS * d + (size_t)KEY_TILE * (d + 1) + (v_cache ? (size_t)KEY_TILE * dv : 0) + ROWS * KEY_TILE);
-    dim3 grid((max_new_tokens + p.tokens_per_tile - 1) / p.tokens_per_tile, nkv * p.head_chunks, batch * p.max_splits);
+    dim3 grid((max_new_tokens + p.tokens_per_tile - 1) / p.tokens_per_tile, nkv * p.head_chunks * maps, batch * p.max_splits);
     HYMT2_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "attention: grid too large (batch %d x splits %d)", batch, p.max_splits);
     int rc = HYMT2_OK;
     HYMT2_DISPATCH_DTYPE(dtype, T, {
@@ -332,7 +379,8 @@ static int attention_simt_general(void* out, const void* q, const void* k_cache,
         kernel<<<grid, ROWS * LANES_PER_ROW, smem, stream>>>(p);
         rc = hymt2_check_launch("attention_simt");
         if (rc == HYMT2_OK && split_keys > 0) {
-            attention_merge_kernel<T><<<tokens * nh, merge_threads(dv), 0, stream>>>(p, tokens);
+            auto merge = maps > 1 ? attention_merge_kernel<float> : attention_merge_kernel<T>;
+            merge<<<tokens * nh * maps, merge_threads(dv), 0, stream>>>(p, tokens);
             rc = hymt2_check_launch("attention_merge");
         }
     });
@@ -363,6 +411,20 @@ HYMT2_API int hymt2_attention_simt_kv(void* out, const void* q, const void* k_ca
     return attention_simt_general(out, q, k_cache, v_cache, dtype, block_table, table_stride, block_tokens, cu_seqlens, slot_ids,
                                   kv_lens, batch, tokens, max_new_tokens, nh, nkv, d, dv, scale, window, split_keys, max_splits,
                                   part_acc, part_ml, stream, status, sink);
+}
+
+// The general form with `maps` maps a head (out is float32 [tokens, nh, maps, dv] when there are several), a cap on the scores
+// (0: none) and a temperature of the queries (coef 0: none).  Keys' rows hold maps * d entries.
+HYMT2_API int hymt2_attention_simt_maps(void* out, const void* q, const void* k_cache, const void* v_cache, int dtype,
+                                        const int* block_table, int table_stride, int block_tokens,
+                                        const int* cu_seqlens, const int* slot_ids, const int* kv_lens,
+                                        int batch, int tokens, int max_new_tokens, int nh, int nkv, int maps, int d, int dv,
+                                        float scale, float softcap, float temp_coef, int temp_every, int split_keys, int max_splits,
+                                        float* part_acc, float* part_ml, cudaStream_t stream, int* status) {
+    HYMT2_REQUIRE(v_cache != nullptr, "attention: no values");
+    return attention_simt_general(out, q, k_cache, v_cache, dtype, block_table, table_stride, block_tokens, cu_seqlens, slot_ids,
+                                  kv_lens, batch, tokens, max_new_tokens, nh, nkv, d, dv, scale, 0, split_keys, max_splits,
+                                  part_acc, part_ml, stream, status, 0, maps, softcap, temp_coef, temp_every);
 }
 
 // Attention over a cache that holds ONE vector per token and layer, shared by all heads: the key of every head

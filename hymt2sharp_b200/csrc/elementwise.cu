@@ -74,6 +74,22 @@ __global__ void convert_kernel(TO* __restrict__ out, const TI* __restrict__ x, s
     if (i < total) out[i] = from_float<TO>(to_float(x[i]));
 }
 
+// The same for rows that go into a wider matrix: out[r, c] (leading dimension ldo) = x[r, c]
+template <typename TO, int V>
+__global__ void place_rows_kernel(TO* __restrict__ out, long ldo, const float* __restrict__ x, int cols, size_t total) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
+    if (i >= total) return;
+    const size_t r = i / cols;
+    const int c = (int)(i - r * cols);
+    const Pack<float, V> v = load_pack<float, V>(x + i);
+    Pack<TO, V> o;
+#pragma unroll
+    for (int k = 0; k < V; k++) o.v[k] = from_float<TO>(v.v[k]);
+    store_pack<TO, V>(out + r * ldo + c, o);
+}
+
 // x[t, h, v] <- x[t, h, v] * sigmoid(g[t, per_head ? h : h * vdim + v])
 template <typename T, int V>
 __global__ void sigmoid_gate_kernel(T* __restrict__ x, const T* __restrict__ g, int heads, int vdim, long ldg, int per_head,
@@ -184,6 +200,19 @@ HYMT2_API int hymt2_convert(void* out, int out_dtype, const void* x, int x_dtype
     HYMT2_DISPATCH_DTYPE(out_dtype, TO, HYMT2_DISPATCH_DTYPE(x_dtype, TI,
         (launch_pdl(convert_kernel<TO, TI>, dim3(blocks_for((size_t)total)), dim3(256), 0, stream, (TO*)out, (const TI*)x, (size_t)total))));
     return hymt2_check_launch("convert");
+}
+
+HYMT2_API int hymt2_place_rows(void* out, int out_dtype, long ldo, const float* x, int rows, int cols, cudaStream_t stream) {
+    if (rows == 0) return HYMT2_OK;
+    HYMT2_REQUIRE(rows > 0 && cols > 0 && ldo >= cols, "place_rows: bad sizes");
+    const size_t total = (size_t)rows * cols;
+    HYMT2_DISPATCH_DTYPE(out_dtype, TO, {
+        if (cols % 4 == 0 && ldo % 4 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)x % 16 == 0)
+            launch_pdl(place_rows_kernel<TO, 4>, dim3(blocks_for(total / 4)), dim3(256), 0, stream, (TO*)out, ldo, x, cols, total);
+        else
+            launch_pdl(place_rows_kernel<TO, 1>, dim3(blocks_for(total)), dim3(256), 0, stream, (TO*)out, ldo, x, cols, total);
+    });
+    return hymt2_check_launch("place_rows");
 }
 
 HYMT2_API int hymt2_sigmoid_gate(void* x, const void* g, int dtype, int rows, int heads, int vdim, long ldg, int per_head,

@@ -29,6 +29,59 @@ HYMT2_API int hymt2_embed(float* out, const void* table, int table_dtype, const 
     return hymt2_check_launch("embed");
 }
 
+// The same with a second table: out[t] = table[id] * scale + pairs[row], row = (previous token * mul_prev + id * mul_cur) mod
+// buckets, and row `buckets` for a sequence's first token (position 0).  The token in front of a step's first one is the
+// int32 at `state_offset` of the sequence's state row, which then receives the step's last token: the block of a sequence's
+// first token reads it and writes it, so nothing is read after it was overwritten.  Rows without a slot touch no state.
+template <typename T>
+__global__ void embed_pairs_kernel(float* __restrict__ out, const T* __restrict__ table, const T* __restrict__ pairs,
+                                   const int* __restrict__ ids, const int* __restrict__ token_seq, const int* __restrict__ token_pos,
+                                   const int* __restrict__ cu_seqlens, const int* __restrict__ slot_ids, uint8_t* state, long state_offset,
+                                   long state_stride, int hidden, int vocab, float scale, int buckets, long long mul_prev,
+                                   long long mul_cur, int* status) {
+    pdl_wait();
+    pdl_launch_dependents();
+    __shared__ int row_s;
+    const int t = blockIdx.x;
+    const int id = ids[t];
+    if (threadIdx.x == 0) {
+        const int seq = token_seq[t], slot = slot_ids[seq], first = cu_seqlens[seq];
+        int* kept = slot >= 0 ? reinterpret_cast<int*>(state + (size_t)slot * state_stride + state_offset) : nullptr;
+        long long row = buckets;
+        if (token_pos[t] > 0 && slot >= 0) {
+            const long long prev = t == first ? *kept : ids[t - 1];
+            row = (prev * mul_prev + (long long)id * mul_cur) % buckets;
+            if (row < 0) row += buckets;
+        }
+        if (t == first && kept) *kept = ids[cu_seqlens[seq + 1] - 1];
+        row_s = (int)row;
+    }
+    __syncthreads();
+    if (id < 0 || id >= vocab) {  // never read outside the table: flag it and give zeros
+        if (threadIdx.x == 0) atomicExch(status, 1);
+        for (int i = threadIdx.x; i < hidden; i += blockDim.x) out[(size_t)t * hidden + i] = 0.f;
+        return;
+    }
+    const T* row = table + (size_t)id * hidden;
+    const T* pair = pairs + (size_t)row_s * hidden;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x)
+        out[(size_t)t * hidden + i] = fmaf(to_float(row[i]), scale, to_float(pair[i]));
+}
+
+HYMT2_API int hymt2_embed_pairs(float* out, const void* table, const void* pairs, int table_dtype, const int* ids, const int* token_seq,
+                                const int* token_pos, const int* cu_seqlens, const int* slot_ids, void* state, long state_offset,
+                                long state_stride, int tokens, int hidden, int vocab, float scale, int buckets, long long mul_prev,
+                                long long mul_cur, int* status, cudaStream_t stream) {
+    if (tokens == 0) return HYMT2_OK;
+    HYMT2_REQUIRE(tokens > 0 && hidden > 0 && vocab > 0 && buckets > 0, "embed_pairs: bad sizes tokens=%d hidden=%d vocab=%d buckets=%d", tokens,
+                  hidden, vocab, buckets);
+    HYMT2_REQUIRE(state && state_offset % 4 == 0 && state_stride % 4 == 0, "embed_pairs: the state rows are not aligned");
+    HYMT2_DISPATCH_DTYPE(table_dtype, T,
+        launch_pdl(embed_pairs_kernel<T>, dim3(tokens), dim3(256), 0, stream, out, (const T*)table, (const T*)pairs, ids, token_seq, token_pos,
+                   cu_seqlens, slot_ids, (uint8_t*)state, state_offset, state_stride, hidden, vocab, scale, buckets, mul_prev, mul_cur, status));
+    return hymt2_check_launch("embed_pairs");
+}
+
 // After a decode step: every live row of the batch is one token longer.
 __global__ void advance_decode_kernel(int* token_pos, int* kv_lens, const int* slot_ids, int rows) {
     pdl_launch_dependents();

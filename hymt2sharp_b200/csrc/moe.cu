@@ -3,9 +3,11 @@
 // Everything here is float32 and integer arithmetic; nothing depends on the order in which blocks run (no atomics), so a
 // token's result does not depend on what else is in the step.
 //
-//   route    scores s = softmax(z + bias) over ALL router outputs (bias: optional); the `top` largest of s + correction are
-//            chosen (ties: the lower index); a chosen output's weight is its s, without the correction, either as it is or
-//            (`renorm`) divided by the sum over the chosen ones, which is the softmax over the chosen outputs alone
+//   route    scores s = softmax(z + bias) over ALL router outputs, or sigmoid(z + bias) of each (bias: optional); the `top`
+//            largest of s + correction are chosen (ties: the lower index), with several groups of neighbouring outputs only
+//            from the `keep` groups whose two largest have the largest sums; a chosen output's weight is its s, without the
+//            correction, either as it is or (`renorm`) divided by the sum over the chosen ones (for softmax scores that is
+//            the softmax over the chosen outputs alone)
 //   count    how many (token, choice) pairs name each expert that has tensors (outputs from `experts` on name identity
 //            experts, which need no product)
 //   place    every expert's pairs, in token order, get consecutive rows of a sorted list; an expert's segment is padded to
@@ -19,31 +21,64 @@ namespace {
 
 constexpr int ROUTE_WARPS = 4;
 
-__global__ void __launch_bounds__(ROUTE_WARPS * 32)
-moe_route_kernel(int* __restrict__ chosen, float* __restrict__ weight, const float* __restrict__ logits,
-                 const float* __restrict__ correction, const float* __restrict__ bias, int renorm, int tokens, int outputs, int top) {
-    extern __shared__ float smem[];   // [ROUTE_WARPS][2 * outputs]: scores, choice scores
-    pdl_wait();
-    pdl_launch_dependents();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int t = blockIdx.x * ROUTE_WARPS + warp;
-    if (t >= tokens) return;
-    float* s = smem + (size_t)warp * 2 * outputs;
-    float* c = s + outputs;
-    const float* z = logits + (size_t)t * outputs;
-    float m = -INFINITY;
-    for (int i = lane; i < outputs; i += 32) m = fmaxf(m, z[i] + (bias ? bias[i] : 0.f));
-    m = warp_max(m);
-    float sum = 0.f;
-    for (int i = lane; i < outputs; i += 32) { const float e = expf(z[i] + (bias ? bias[i] : 0.f) - m); s[i] = e; sum += e; }
-    sum = warp_sum(sum);
-    const float inv = 1.0f / sum;
-    for (int i = lane; i < outputs; i += 32) {
-        s[i] *= inv;
-        c[i] = s[i] + (correction ? correction[i] : 0.f);
+enum { SCORES_SOFTMAX = 0, SCORES_SIGMOID = 1 };
+
+// How outputs become scores and scores a choice.
+struct RouteRule {
+    const float* correction;   // [outputs] or null
+    const float* bias;         // [outputs] or null
+    int scores;                // SCORES_SOFTMAX over all outputs, or SCORES_SIGMOID of each
+    int renorm;                // weights: divided by (the sum over the chosen ones + share_eps)
+    float share_eps;
+    int groups, keep;          // equal groups of neighbouring outputs, of which the best `keep` take part (groups 1: all)
+    int outputs, top;
+    long ldz;                  // row stride of the router's outputs
+};
+
+// floats of shared memory that a warp's routing needs
+__host__ __device__ inline int route_floats(int outputs, int groups) { return 2 * outputs + groups; }
+
+// One token by one warp; s [outputs], c [outputs], worth [groups] are the warp's shared memory.  `also` (may be null) receives
+// the choice a second time.
+__device__ __forceinline__ void route_token(const RouteRule& r, const float* __restrict__ z, float* s, float* c, float* worth, int lane,
+                                            int* __restrict__ chosen, float* __restrict__ weight, int* also) {
+    const int outputs = r.outputs;
+    if (r.scores == SCORES_SIGMOID) {
+        for (int i = lane; i < outputs; i += 32) s[i] = 1.0f / (1.0f + expf(-(z[i] + (r.bias ? r.bias[i] : 0.f))));
+    } else {
+        float m = -INFINITY;
+        for (int i = lane; i < outputs; i += 32) m = fmaxf(m, z[i] + (r.bias ? r.bias[i] : 0.f));
+        m = warp_max(m);
+        float sum = 0.f;
+        for (int i = lane; i < outputs; i += 32) { const float e = expf(z[i] + (r.bias ? r.bias[i] : 0.f) - m); s[i] = e; sum += e; }
+        sum = warp_sum(sum);
+        const float inv = 1.0f / sum;
+        for (int i = lane; i < outputs; i += 32) s[i] *= inv;
     }
+    for (int i = lane; i < outputs; i += 32) c[i] = s[i] + (r.correction ? r.correction[i] : 0.f);   // (a lane's own entries)
     __syncwarp();
-    for (int k = 0; k < top; k++) {
+    if (r.groups > 1) {
+        // a group's worth is the sum of its two largest scores; a group stays if fewer than `keep` are worth more (of equals
+        // the lower number counts as more)
+        const int per = outputs / r.groups;
+        for (int g = lane; g < r.groups; g += 32) {
+            float first = -INFINITY, second = -INFINITY;
+            for (int i = g * per; i < (g + 1) * per; i++) {
+                if (c[i] > first) { second = first; first = c[i]; }
+                else if (c[i] > second) second = c[i];
+            }
+            worth[g] = per > 1 ? first + second : first;
+        }
+        __syncwarp();
+        for (int g = lane; g < r.groups; g += 32) {
+            int above = 0;
+            for (int o = 0; o < r.groups; o++) above += worth[o] > worth[g] || (worth[o] == worth[g] && o < g);
+            if (above >= r.keep)
+                for (int i = g * per; i < (g + 1) * per; i++) c[i] = -INFINITY;
+        }
+        __syncwarp();
+    }
+    for (int k = 0; k < r.top; k++) {
         float best = -INFINITY;
         int at = 0x7fffffff;
         for (int i = lane; i < outputs; i += 32)
@@ -54,18 +89,33 @@ moe_route_kernel(int* __restrict__ chosen, float* __restrict__ weight, const flo
             const int oa = __shfl_xor_sync(0xffffffffu, at, o);
             if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
         }
+        at = min(at, outputs - 1);   // (scores that are no numbers name nobody: stay inside the tables)
         if (lane == 0) {
-            chosen[(size_t)t * top + k] = at;
-            weight[(size_t)t * top + k] = s[at];
+            chosen[k] = at;
+            weight[k] = s[at];
+            if (also) also[k] = at;
             c[at] = -INFINITY;
         }
         __syncwarp();
     }
-    if (renorm && lane == 0) {   // the weights become the softmax over the chosen outputs alone: the same exponentials, another sum
+    if (r.renorm && lane == 0) {
         float chosen_sum = 0.f;
-        for (int k = 0; k < top; k++) chosen_sum += weight[(size_t)t * top + k];
-        for (int k = 0; k < top; k++) weight[(size_t)t * top + k] /= chosen_sum;
+        for (int k = 0; k < r.top; k++) chosen_sum += weight[k];
+        for (int k = 0; k < r.top; k++) weight[k] /= chosen_sum + r.share_eps;
     }
+}
+
+__global__ void __launch_bounds__(ROUTE_WARPS * 32)
+moe_route_kernel(int* __restrict__ chosen, float* __restrict__ weight, const float* __restrict__ logits, RouteRule r, int tokens) {
+    extern __shared__ float smem[];   // [ROUTE_WARPS][route_floats]: scores, choice scores, groups
+    pdl_wait();
+    pdl_launch_dependents();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t = blockIdx.x * ROUTE_WARPS + warp;
+    if (t >= tokens) return;
+    float* s = smem + (size_t)warp * route_floats(r.outputs, r.groups);
+    route_token(r, logits + (size_t)t * r.ldz, s, s + r.outputs, s + 2 * r.outputs, lane, chosen + (size_t)t * r.top,
+                weight + (size_t)t * r.top, nullptr);
 }
 
 constexpr int PLACE_THREADS = 256;
@@ -189,55 +239,18 @@ constexpr int SMALL_PAIRS = 1024, SMALL_THREADS = 256;
 
 __global__ void __launch_bounds__(SMALL_THREADS)
 moe_route_place_small_kernel(int* __restrict__ chosen, float* __restrict__ weight, int* __restrict__ pair_row, int* __restrict__ row_token,
-                             int* __restrict__ tile_group, const float* __restrict__ logits, const float* __restrict__ correction,
-                             const float* __restrict__ bias, int renorm, int tokens, int outputs, int top, int experts, int tile, int max_tiles) {
-    extern __shared__ float smem[];   // [warps][2 * outputs] scores and choice scores, then [experts + 1] segment starts
+                             int* __restrict__ tile_group, const float* __restrict__ logits, RouteRule r, int tokens, int experts, int tile,
+                             int max_tiles) {
+    extern __shared__ float smem[];   // [warps][route_floats] scores, choice scores, groups; then [experts + 1] segment starts
     __shared__ int pairs_s[SMALL_PAIRS];
     pdl_wait();
     pdl_launch_dependents();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = SMALL_THREADS / 32;
-    float* s = smem + (size_t)warp * 2 * outputs;
-    float* c = s + outputs;
-    int* start = reinterpret_cast<int*>(smem + (size_t)warps * 2 * outputs);
-    for (int t = warp; t < tokens; t += warps) {
-        const float* z = logits + (size_t)t * outputs;
-        float m = -INFINITY;
-        for (int i = lane; i < outputs; i += 32) m = fmaxf(m, z[i] + (bias ? bias[i] : 0.f));
-        m = warp_max(m);
-        float sum = 0.f;
-        for (int i = lane; i < outputs; i += 32) { const float e = expf(z[i] + (bias ? bias[i] : 0.f) - m); s[i] = e; sum += e; }
-        sum = warp_sum(sum);
-        const float inv = 1.0f / sum;
-        for (int i = lane; i < outputs; i += 32) {
-            s[i] *= inv;
-            c[i] = s[i] + (correction ? correction[i] : 0.f);
-        }
-        __syncwarp();
-        for (int k = 0; k < top; k++) {
-            float best = -INFINITY;
-            int at = 0x7fffffff;
-            for (int i = lane; i < outputs; i += 32)
-                if (c[i] > best) { best = c[i]; at = i; }
-#pragma unroll
-            for (int o = 16; o > 0; o >>= 1) {
-                const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-                const int oa = __shfl_xor_sync(0xffffffffu, at, o);
-                if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
-            }
-            if (lane == 0) {
-                chosen[(size_t)t * top + k] = at;
-                weight[(size_t)t * top + k] = s[at];
-                pairs_s[t * top + k] = at;
-                c[at] = -INFINITY;
-            }
-            __syncwarp();
-        }
-        if (renorm && lane == 0) {
-            float chosen_sum = 0.f;
-            for (int k = 0; k < top; k++) chosen_sum += weight[(size_t)t * top + k];
-            for (int k = 0; k < top; k++) weight[(size_t)t * top + k] /= chosen_sum;
-        }
-    }
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = SMALL_THREADS / 32, top = r.top;
+    float* s = smem + (size_t)warp * route_floats(r.outputs, r.groups);
+    int* start = reinterpret_cast<int*>(smem + (size_t)warps * route_floats(r.outputs, r.groups));
+    for (int t = warp; t < tokens; t += warps)
+        route_token(r, logits + (size_t)t * r.ldz, s, s + r.outputs, s + 2 * r.outputs, lane, chosen + (size_t)t * top,
+                    weight + (size_t)t * top, pairs_s + t * top);
     __syncthreads();
     const int pairs = tokens * top;
     for (int e = threadIdx.x; e < experts; e += SMALL_THREADS) {
@@ -339,14 +352,25 @@ HYMT2_API int hymt2_moe_gather(void* xs, const void* x, int dtype, const int* ro
     return hymt2_check_launch("moe_gather");
 }
 
-HYMT2_API int hymt2_moe_route(int* chosen, float* weight, const float* logits, const float* correction, const float* bias, int renorm,
-                              int tokens, int outputs, int top, cudaStream_t stream) {
+static int check_rule(const char* what, const RouteRule& r, int tokens) {
+    HYMT2_REQUIRE(tokens > 0 && r.outputs > 0 && r.top > 0 && r.top <= r.outputs && r.ldz >= r.outputs, "%s: bad sizes tokens=%d outputs=%d top=%d", what,
+                  tokens, r.outputs, r.top);
+    HYMT2_REQUIRE(r.scores == SCORES_SOFTMAX || r.scores == SCORES_SIGMOID, "%s: unknown kind of scores %d", what, r.scores);
+    HYMT2_REQUIRE(r.groups > 0 && r.outputs % r.groups == 0 && r.keep > 0 && r.keep <= r.groups && (r.groups == 1 || r.top <= r.keep * (r.outputs / r.groups)),
+                  "%s: %d of %d groups hold fewer than %d of %d outputs", what, r.keep, r.groups, r.top, r.outputs);
+    return HYMT2_OK;
+}
+
+HYMT2_API int hymt2_moe_route(int* chosen, float* weight, const float* logits, long ldz, const float* correction, const float* bias, int scores,
+                              int renorm, float share_eps, int groups, int keep, int tokens, int outputs, int top, cudaStream_t stream) {
     if (tokens == 0) return HYMT2_OK;
-    HYMT2_REQUIRE(tokens > 0 && outputs > 0 && top > 0 && top <= outputs, "moe_route: bad sizes tokens=%d outputs=%d top=%d", tokens, outputs, top);
-    const size_t smem = (size_t)ROUTE_WARPS * 2 * outputs * sizeof(float);
+    const RouteRule r{correction, bias, scores, renorm, share_eps, groups, keep, outputs, top, ldz};
+    const int rc = check_rule("moe_route", r, tokens);
+    if (rc != HYMT2_OK) return rc;
+    const size_t smem = (size_t)ROUTE_WARPS * route_floats(outputs, groups) * sizeof(float);
     HYMT2_REQUIRE(smem <= 48 * 1024, "moe_route: %d router outputs are too many", outputs);
     launch_pdl(moe_route_kernel, dim3((tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem, stream, chosen, weight,
-               logits, correction, bias, renorm, tokens, outputs, top);
+               logits, r, tokens);
     return hymt2_check_launch("moe_route");
 }
 
@@ -377,16 +401,20 @@ HYMT2_API int hymt2_moe_combine(float* out, const float* y, const void* x, int x
 
 // moe_route and moe_place in one launch for a step of few tokens (tokens * top <= 1024, experts <= 4096).
 HYMT2_API int hymt2_moe_route_place_small(int* chosen, float* weight, int* pair_row, int* row_token, int* tile_group, const float* logits,
-                                          const float* correction, const float* bias, int renorm, int tokens, int outputs, int top, int experts,
-                                          int tile, int max_tiles, cudaStream_t stream) {
+                                          long ldz, const float* correction, const float* bias, int scores, int renorm, float share_eps,
+                                          int groups, int keep, int tokens, int outputs, int top, int experts, int tile, int max_tiles,
+                                          cudaStream_t stream) {
     if (tokens == 0) return HYMT2_OK;
-    HYMT2_REQUIRE(tokens > 0 && outputs > 0 && top > 0 && top <= outputs && experts >= 0 && experts <= outputs && tile > 0, "moe_route_place_small: bad sizes");
+    const RouteRule r{correction, bias, scores, renorm, share_eps, groups, keep, outputs, top, ldz};
+    const int rc = check_rule("moe_route_place_small", r, tokens);
+    if (rc != HYMT2_OK) return rc;
+    HYMT2_REQUIRE(experts >= 0 && experts <= outputs && tile > 0, "moe_route_place_small: bad sizes");
     HYMT2_REQUIRE((long)tokens * top <= SMALL_PAIRS, "moe_route_place_small: %d pairs are too many", tokens * top);
     HYMT2_REQUIRE(experts == 0 || (long)max_tiles * tile >= (long)tokens * top + (long)experts * (tile - 1), "moe_route_place_small: too few tiles");
-    const size_t smem = ((size_t)(SMALL_THREADS / 32) * 2 * outputs + experts + 1) * sizeof(float);
+    const size_t smem = ((size_t)(SMALL_THREADS / 32) * route_floats(outputs, groups) + experts + 1) * sizeof(float);
     HYMT2_REQUIRE(smem <= 40 * 1024, "moe_route_place_small: %d router outputs are too many", outputs);
     launch_pdl(moe_route_place_small_kernel, dim3(1), dim3(SMALL_THREADS), smem, stream, chosen, weight, pair_row, row_token, tile_group,
-               logits, correction, bias, renorm, tokens, outputs, top, experts, tile, max_tiles);
+               logits, r, tokens, experts, tile, max_tiles);
     return hymt2_check_launch("moe_route_place");
 }
 

@@ -24,6 +24,8 @@ class DecoderModel:
         self.slots: list[list[MixerSlot]] = []   # per entry of the order: one MixerSlot for each mixer of its block
         self.state_bytes = 0
         self._ones = None
+        self.pairs = self.join = None            # the bigram table; the product that joins the residual with the embedding's output
+        self.pair_state_offset = 0
         # a step can be captured into a CUDA graph only if every part launches kernels and nothing else
         self.graph_safe = all(getattr(b, "graph_safe", False) for b in self.blocks)
         self._plan_memory()
@@ -32,6 +34,10 @@ class DecoderModel:
     def tensors(self) -> dict[str, TensorSpec]:
         s = self.spec
         t = {s.embedding: TensorSpec((s.vocab, s.hidden))}
+        if s.bigram is not None:
+            t[s.bigram.table] = TensorSpec((s.bigram.buckets + 1, s.hidden))
+        if s.join is not None:
+            t[s.join] = TensorSpec((s.hidden, 2 * s.hidden))
         for b in self.blocks:
             t.update(b.tensors())
         t.update(self.final_norm.tensors())
@@ -50,6 +56,8 @@ class DecoderModel:
         planes: list[int] = []
         specs: list[GroupSpec] = []
         offset = 0
+        if self.spec.bigram is not None:
+            self.pair_state_offset, offset = offset, offset + 4     # the token in front of the next one
         for i, run in enumerate(self.spec.order):
             block = self.blocks[run.layer]
             needs, states = list(block.cache_needs()), list(block.state_bytes())
@@ -86,6 +94,12 @@ class DecoderModel:
     def load(self, weights: dict, device, dtype: torch.dtype) -> None:
         s = self.spec
         self.embedding = compute_form(weights[s.embedding], device, dtype)
+        if s.bigram is not None:
+            self.pairs = compute_form(weights[s.bigram.table], device, dtype)
+            if self.pairs.dtype != self.embedding.dtype:
+                self.pairs = self.pairs.to(self.embedding.dtype)
+        if s.join is not None:
+            self.join = Linear(compute_form(weights[s.join], device, dtype), role="join")
         for b in self.blocks:
             b.load(weights, device, dtype)
         self.final_norm.load(weights, device, dtype)
@@ -127,7 +141,17 @@ class DecoderModel:
             visit(self.blocks[layer])
         visit(self.final_norm)
         visit(self.head)
+        visit(self.join)
         return total
+
+    def _embed(self, out: torch.Tensor, ctx) -> None:
+        s = self.spec
+        if s.bigram is None:
+            ops.embed(out, self.embedding, ctx.tokens, ctx.status, s.embed_scale or 1.0)
+        else:
+            ops.embed_pairs(out, self.embedding, self.pairs, ctx.tokens, ctx.token_seq, ctx.token_pos, ctx.cu_seqlens, ctx.slot_ids,
+                            ctx.cache.state, self.pair_state_offset, 1.0 if s.embed_scale is None else s.embed_scale, s.bigram.mul_prev,
+                            s.bigram.mul_cur, ctx.status)
 
     # -- one step -----------------------------------------------------------------
     def forward(self, ctx, want_rows: torch.Tensor | None, num_want: int) -> torch.Tensor:
@@ -137,15 +161,22 @@ class DecoderModel:
         streams = self.spec.residual_streams
         if streams is None:
             residual = torch.empty((T, self.spec.hidden), dtype=torch.float32, device=ctx.device)
-            ops.embed(residual, self.embedding, ctx.tokens, ctx.status, self.spec.embed_scale or 1.0)
+            self._embed(residual, ctx)
         else:
             residual = torch.empty((streams, T, self.spec.hidden), dtype=torch.float32, device=ctx.device)
-            ops.embed(residual[0], self.embedding, ctx.tokens, ctx.status, self.spec.embed_scale or 1.0)
+            self._embed(residual[0], ctx)
             ops.streams_fill(residual)
         order = self.spec.order
+        joined = None
+        if self.join is not None:     # [x | x0] side by side in the compute type; the right half is the embedding's output throughout
+            joined = torch.empty((T, 2 * self.spec.hidden), dtype=ctx.dtype, device=ctx.device)
+            ops.place_rows(joined[:, self.spec.hidden:], residual)
         for i, (run, slots) in enumerate(zip(order, self.slots)):
             # the first norm of the block that runs next, for a block whose last product can prepare it (parts.base.Prenormed)
-            nxt = self.blocks[order[i + 1].layer] if i + 1 < len(order) else None
+            nxt = self.blocks[order[i + 1].layer] if i + 1 < len(order) and not order[i + 1].joins else None
+            if run.joins:
+                ops.place_rows(joined[:, :self.spec.hidden], residual)
+                self.join(joined, out=residual)
             ctx.next_first_norm = getattr(nxt, "first_norm", lambda: None)() if nxt is not None else None
             ctx.block_ahead = nxt
             self.blocks[run.layer].forward(residual, ctx, slots)

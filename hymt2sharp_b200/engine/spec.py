@@ -10,13 +10,26 @@ from ..parts.base import PartSpec
 
 
 @dataclass
+class Bigram:
+    """A second table that the embedding adds a row of: row (previous token * mul_prev + token * mul_cur) mod buckets, and for a
+    sequence's first token row number `buckets`, the last one.  The previous token is state of the sequence."""
+    table: str                        # checkpoint name of the [buckets + 1, hidden] table
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+
+
+@dataclass
 class Run:
     """One entry of the order in which layers run.  A layer may be named by several
     entries (it then runs several times with the same weights, each run with a cache
     plane of its own), and an entry may read the cache plane that an earlier entry
-    wrote (`cache_from` = that entry's index in the order) instead of writing one."""
+    wrote (`cache_from` = that entry's index in the order) instead of writing one.
+    With `joins` the residual x becomes W [x; x0] before the layer runs, x0 being the
+    embedding's output and W the matrix that the spec's `join` names."""
     layer: int
     cache_from: int | None = None
+    joins: bool = False
 
 
 @dataclass
@@ -38,10 +51,14 @@ class ModelSpec:
     # None: the residual is one matrix [T, hidden].  n >= 1: it is kept as n streams [n, T, hidden] (parts.block.StreamsBlock),
     # all equal to the embedding's output at the start and added up in front of the final norm
     residual_streams: int | None = None
+    bigram: Bigram | None = None      # (None: the embedding's rows alone)
+    join: str | None = None           # checkpoint name of the [hidden, 2 hidden] matrix of the runs that say `joins`
 
     def __post_init__(self):
         if not self.order:
             self.order = [Run(i) for i in range(len(self.layers))]
+        if any(run.joins for run in self.order) and (self.join is None or self.residual_streams is not None):
+            raise ValueError("a run that joins the residual with the embedding's output needs the matrix's name and one residual stream")
         for i, run in enumerate(self.order):
             if not (0 <= run.layer < len(self.layers)):
                 raise ValueError(f"order[{i}] names layer {run.layer}, the model has {len(self.layers)}")

@@ -6,6 +6,7 @@ from __future__ import annotations
 
 import ctypes
 from ctypes import c_float, c_int, c_long, c_void_p
+from dataclasses import dataclass
 
 import torch
 
@@ -191,6 +192,27 @@ def embed(out: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, status: tor
         raise KernelError(f"embed: shapes out {tuple(out.shape)} table {tuple(table.shape)} ids {tuple(ids.shape)}")
     _check(_lib().hymt2_embed(_ptr(out), _ptr(table), c_int(dtype_code(table.dtype)), _ptr(ids), c_int(T),
                               c_int(H), c_int(table.shape[0]), c_float(scale), _ptr(status), _stream()), "embed")
+
+
+def embed_pairs(out: torch.Tensor, table: torch.Tensor, pairs: torch.Tensor, ids: torch.Tensor, token_seq: torch.Tensor, token_pos: torch.Tensor,
+                cu_seqlens: torch.Tensor, slot_ids: torch.Tensor, state: torch.Tensor, state_offset: int, scale: float, mul_prev: int,
+                mul_cur: int, status: torch.Tensor) -> None:
+    """out[t] = float32(table[ids[t]]) * scale + pairs[row], row = (previous token * mul_prev + ids[t] * mul_cur) mod (rows of `pairs`
+    less one), the last row for a sequence's first token.  The token before a step's first one is the int32 at byte
+    `state_offset` of the sequence's state row, which receives the step's last token."""
+    _need(out, "out", torch.float32, 2); _need(table, "table", None, 2); _need(pairs, "pairs", table.dtype, 2)
+    T, H = out.shape
+    for t, n in ((ids, "ids"), (token_seq, "token_seq"), (token_pos, "token_pos"), (cu_seqlens, "cu_seqlens"), (slot_ids, "slot_ids")):
+        _need(t, n, torch.int32, 1)
+    if table.shape[1] != H or pairs.shape[1] != H or pairs.shape[0] < 2 or min(ids.shape[0], token_seq.shape[0], token_pos.shape[0]) < T:
+        raise KernelError(f"embed_pairs: shapes out {tuple(out.shape)} table {tuple(table.shape)} pairs {tuple(pairs.shape)}")
+    if state.dtype != torch.uint8 or state.dim() != 2 or state_offset % 4 or state.stride(0) % 4 or state_offset + 4 > state.shape[1]:
+        raise KernelError("embed_pairs: the state rows are too short or not aligned")
+    _check(_lib().hymt2_embed_pairs(_ptr(out), _ptr(table), _ptr(pairs), c_int(dtype_code(table.dtype)), _ptr(ids), _ptr(token_seq),
+                                    _ptr(token_pos), _ptr(cu_seqlens), _ptr(slot_ids), _ptr(state), c_long(state_offset),
+                                    c_long(state.stride(0)), c_int(T), c_int(H), c_int(table.shape[0]), c_float(scale),
+                                    c_int(pairs.shape[0] - 1), ctypes.c_longlong(mul_prev), ctypes.c_longlong(mul_cur), _ptr(status), _stream()),
+           "embed_pairs")
 
 
 def advance_decode(token_pos: torch.Tensor, kv_lens: torch.Tensor, slot_ids: torch.Tensor) -> None:
@@ -1191,6 +1213,48 @@ def attention_simt_kv(out: torch.Tensor, q: torch.Tensor, k_plane: torch.Tensor,
            "attention_simt", 2 if split_keys > 0 else 1)
 
 
+def attention_simt_maps(out: torch.Tensor, q: torch.Tensor, k_plane: torch.Tensor, v_plane: torch.Tensor, block_table: torch.Tensor,
+                        cu_seqlens: torch.Tensor, slot_ids: torch.Tensor, kv_lens: torch.Tensor, batch: int, max_new_tokens: int, nh: int,
+                        nkv: int, maps: int, d: int, dv: int, scale: float, softcap: float = 0.0, temp_coef: float = 0.0, temp_every: int = 1,
+                        split_keys: int = 0, max_splits: int = 0, part_acc: torch.Tensor | None = None, part_ml: torch.Tensor | None = None,
+                        status: torch.Tensor | None = None) -> None:
+    """Causal attention with `maps` softmax maps a head over the same values: q [T, nh * maps * d], keys' rows of maps * d entries,
+    out [T, nh * maps * dv] (float32 when there are several maps).  score = (q . k) * scale * (1 + temp_coef * ln(floor((p + 1) /
+    temp_every) + 1)) at the query's position p, then softcap * tanh(score / softcap) with softcap > 0.  Scratch of a split run:
+    attention_simt_scratch with nh * maps heads of dv."""
+    if status is None:
+        status = device_status(out.device)
+    _need(q, "q", None, 2); _need(out, "out", torch.float32 if maps > 1 else q.dtype, 2)
+    _need(k_plane, "k_plane", q.dtype, 4); _need(v_plane, "v_plane", q.dtype, 4)
+    T = out.shape[0]
+    if out.shape[1] != nh * maps * dv or q.shape[1] != nh * maps * d or q.shape[0] < T or k_plane.shape[1] != nkv or k_plane.shape[3] != maps * d \
+            or v_plane.shape != (*k_plane.shape[:3], dv):
+        raise KernelError(f"attention: shapes out {tuple(out.shape)} q {tuple(q.shape)} k {tuple(k_plane.shape)} v {tuple(v_plane.shape)}")
+    _need(block_table, "block_table", torch.int32, 2)
+    for t, n in ((cu_seqlens, "cu_seqlens"), (slot_ids, "slot_ids"), (kv_lens, "kv_lens")):
+        _need(t, n, torch.int32, 1)
+    if split_keys > 0:
+        need_acc, need_ml = attention_simt_scratch(T, nh * maps, dv, max_splits)
+        _need(part_acc, "part_acc", torch.float32); _need(part_ml, "part_ml", torch.float32)
+        if part_acc.numel() < need_acc or part_ml.numel() < need_ml:
+            raise KernelError("attention: the split scratch is too small")
+    _check(_lib().hymt2_attention_simt_maps(_ptr(out), _ptr(q), _ptr(k_plane), _ptr(v_plane), c_int(dtype_code(q.dtype)), _ptr(block_table),
+                                            c_int(block_table.stride(0)), c_int(k_plane.shape[2]), _ptr(cu_seqlens), _ptr(slot_ids),
+                                            _ptr(kv_lens), c_int(batch), c_int(T), c_int(max_new_tokens), c_int(nh), c_int(nkv), c_int(maps),
+                                            c_int(d), c_int(dv), c_float(scale), c_float(softcap), c_float(temp_coef), c_int(temp_every),
+                                            c_int(split_keys), c_int(max_splits), _ptr(part_acc), _ptr(part_ml), _stream(), _ptr(status)),
+           "attention_simt", 2 if split_keys > 0 else 1)
+
+
+def diff_combine(out: torch.Tensor, maps: torch.Tensor, nh: int, dv: int, lam: float, eps: float, factor: float) -> None:
+    """out [T, nh * dv] = unit_rms(maps[t, h, 0] - lam * maps[t, h, 1]) * factor over the dv entries; maps [T, nh * 2 * dv] float32."""
+    _need(out, "out", None, 2); _need(maps, "maps", torch.float32, 2)
+    if out.shape[1] != nh * dv or maps.shape != (out.shape[0], 2 * nh * dv):
+        raise KernelError(f"diff_combine: shapes out {tuple(out.shape)} maps {tuple(maps.shape)}")
+    _check(_lib().hymt2_diff_combine(_ptr(out), c_int(dtype_code(out.dtype)), _ptr(maps), c_int(out.shape[0]), c_int(nh), c_int(dv),
+                                     c_float(lam), c_float(eps), c_float(factor), _stream()), "diff_combine")
+
+
 # -- small steps ---------------------------------------------------------------------------------------------------------------
 def relu_squared(out: torch.Tensor, x: torch.Tensor) -> None:
     """out = max(x, 0)^2."""
@@ -1207,6 +1271,16 @@ def convert(out: torch.Tensor, x: torch.Tensor) -> None:
         raise KernelError("convert: shapes differ")
     _check(_lib().hymt2_convert(_ptr(out), c_int(dtype_code(out.dtype)), _ptr(x), c_int(dtype_code(x.dtype)), c_long(x.numel()), _stream()),
            "convert")
+
+
+def place_rows(out: torch.Tensor, x: torch.Tensor) -> None:
+    """out[r, c] = x[r, c] in out's type, `out` being a range of columns of a wider matrix."""
+    ldo = _rows_view(out, "out")
+    _need(x, "x", torch.float32, 2)
+    if out.shape != x.shape:
+        raise KernelError("place_rows: shapes differ")
+    _check(_lib().hymt2_place_rows(_ptr(out), c_int(dtype_code(out.dtype)), c_long(ldo), _ptr(x), c_int(x.shape[0]), c_int(x.shape[1]),
+                                   _stream()), "place_rows")
 
 
 def rmsnorm_add_then_rows(residual: torch.Tensor, x: torch.Tensor, gain: torch.Tensor, eps: float, out: torch.Tensor, groups: int = 1) -> None:
@@ -1226,19 +1300,44 @@ EPILOGUE_RELU_SQUARED = 3
 _group_tiles: dict = {}
 
 
-def moe_route(chosen: torch.Tensor, weight: torch.Tensor, logits: torch.Tensor, correction: torch.Tensor | None,
-              bias: torch.Tensor | None = None, renormalise: bool = False) -> None:
-    """From router outputs logits [T, R] (float32), plus `bias` [R] where one is given: scores = softmax over all R; chosen [T, top]
-    (int32) = the `top` largest of score + correction, best first, ties to the lower index; weight [T, top] (float32) = their
-    scores, as they are, or (`renormalise`) divided by their sum: the softmax over the chosen outputs alone."""
-    _need(logits, "logits", torch.float32, 2); _need(chosen, "chosen", torch.int32, 2); _need(weight, "weight", torch.float32, 2)
-    T, R = logits.shape
+SCORES = {"softmax": 0, "sigmoid": 1}
+
+
+@dataclass(frozen=True)
+class RouteRule:
+    """How a router's outputs become scores, and scores a choice: `scores` "softmax" (over all outputs) or "sigmoid" (of each);
+    `renormalise`: the chosen scores are divided by their sum + share_eps; with groups > 1 only the outputs of the `keep`
+    groups (equal ones, of neighbours) whose two largest scores have the largest sums can be chosen."""
+    scores: str = "softmax"
+    renormalise: bool = False
+    share_eps: float = 0.0
+    groups: int = 1
+    keep: int = 1
+
+
+def _rule_arguments(what: str, logits, correction, bias, rule: RouteRule, outputs: int | None, chosen, weight):
+    ldz = _rows_view(logits, "logits", torch.float32)
+    _need(chosen, "chosen", torch.int32, 2); _need(weight, "weight", torch.float32, 2)
+    T, R = logits.shape[0], outputs or logits.shape[1]
     top = chosen.shape[1]
-    if chosen.shape[0] != T or weight.shape != chosen.shape or not (0 < top <= R):
-        raise KernelError(f"moe_route: shapes logits {tuple(logits.shape)} chosen {tuple(chosen.shape)} weight {tuple(weight.shape)}")
+    if chosen.shape[0] != T or weight.shape != chosen.shape or not (0 < top <= R <= logits.shape[1]):
+        raise KernelError(f"{what}: shapes logits {tuple(logits.shape)} chosen {tuple(chosen.shape)} weight {tuple(weight.shape)}")
     _f32(correction, "correction", R); _f32(bias, "bias", R)
-    _check(_lib().hymt2_moe_route(_ptr(chosen), _ptr(weight), _ptr(logits), _ptr(correction), _ptr(bias), c_int(1 if renormalise else 0),
-                                  c_int(T), c_int(R), c_int(top), _stream()), "moe_route")
+    if rule.scores not in SCORES:
+        raise KernelError(f"{what}: scores '{rule.scores}' are not known (known: {', '.join(SCORES)})")
+    return T, R, top, (c_long(ldz), _ptr(correction), _ptr(bias), c_int(SCORES[rule.scores]), c_int(1 if rule.renormalise else 0),
+                       c_float(rule.share_eps), c_int(rule.groups), c_int(rule.keep))
+
+
+def moe_route(chosen: torch.Tensor, weight: torch.Tensor, logits: torch.Tensor, correction: torch.Tensor | None,
+              bias: torch.Tensor | None = None, renormalise: bool = False, rule: RouteRule | None = None, outputs: int | None = None) -> None:
+    """From router outputs logits [T, R] (float32), plus `bias` [R] where one is given: scores (softmax over all R unless the rule
+    says otherwise); chosen [T, top] (int32) = the `top` largest of score + correction, best first, ties to the lower index;
+    weight [T, top] (float32) = their scores, as they are, or (`renormalise`) divided by their sum: for softmax scores the
+    softmax over the chosen outputs alone.  `outputs`: how many of the columns are the router's (the first ones)."""
+    rule = rule or RouteRule(renormalise=renormalise)
+    T, R, top, args = _rule_arguments("moe_route", logits, correction, bias, rule, outputs, chosen, weight)
+    _check(_lib().hymt2_moe_route(_ptr(chosen), _ptr(weight), _ptr(logits), *args, c_int(T), c_int(R), c_int(top), _stream()), "moe_route")
 
 
 def moe_tiles(tokens: int, top: int, experts: int, tile: int) -> int:
@@ -1383,20 +1482,17 @@ MOE_SMALL_PAIRS = 64   # up to this many (token, choice) pairs one block routes 
 
 def moe_route_place(chosen: torch.Tensor, weight: torch.Tensor, pair_row: torch.Tensor, row_token: torch.Tensor, tile_group: torch.Tensor,
                     logits: torch.Tensor, correction: torch.Tensor | None, experts: int, tile: int, bias: torch.Tensor | None = None,
-                    renormalise: bool = False) -> None:
+                    renormalise: bool = False, rule: RouteRule | None = None, outputs: int | None = None) -> None:
     """moe_route and moe_place in one launch, for a step of at most MOE_SMALL_PAIRS (token, choice) pairs."""
-    _need(logits, "logits", torch.float32, 2); _need(chosen, "chosen", torch.int32, 2); _need(weight, "weight", torch.float32, 2)
     for t, n in ((pair_row, "pair_row"), (row_token, "row_token"), (tile_group, "tile_group")):
         _need(t, n, torch.int32)
-    T, R = logits.shape
-    top, tiles = chosen.shape[1], tile_group.numel() - 1
-    if chosen.shape[0] != T or weight.shape != chosen.shape or pair_row.shape != chosen.shape or not (0 < top <= R) or T * top > MOE_SMALL_PAIRS \
-            or row_token.numel() < tiles * tile or tiles < moe_tiles(T, top, experts, tile):
+    rule = rule or RouteRule(renormalise=renormalise)
+    T, R, top, args = _rule_arguments("moe_route_place", logits, correction, bias, rule, outputs, chosen, weight)
+    tiles = tile_group.numel() - 1
+    if pair_row.shape != chosen.shape or T * top > MOE_SMALL_PAIRS or row_token.numel() < tiles * tile or tiles < moe_tiles(T, top, experts, tile):
         raise KernelError("moe_route_place: shapes do not fit, or a buffer is too small")
-    _f32(correction, "correction", R); _f32(bias, "bias", R)
-    _check(_lib().hymt2_moe_route_place_small(_ptr(chosen), _ptr(weight), _ptr(pair_row), _ptr(row_token), _ptr(tile_group), _ptr(logits),
-                                              _ptr(correction), _ptr(bias), c_int(1 if renormalise else 0), c_int(T), c_int(R), c_int(top),
-                                              c_int(experts), c_int(tile), c_int(tiles), _stream()), "moe_route_place")
+    _check(_lib().hymt2_moe_route_place_small(_ptr(chosen), _ptr(weight), _ptr(pair_row), _ptr(row_token), _ptr(tile_group), _ptr(logits), *args,
+                                              c_int(T), c_int(R), c_int(top), c_int(experts), c_int(tile), c_int(tiles), _stream()), "moe_route_place")
 
 
 MOE_COMBINE_NORM_MAX_WIDTH = 12000   # a row of the fused combine-and-norm kernel lies in shared memory
@@ -1424,6 +1520,53 @@ def moe_combine_norm(residual: torch.Tensor, rows: torch.Tensor | None, branch: 
                                          _ptr(y), _ptr(x), c_int(dtype_code(x.dtype)), _ptr(pair_row), _ptr(weight), _ptr(gain),
                                          c_int(dtype_code(gain.dtype)), c_int(T), c_int(H), c_int(pair_row.shape[1]), c_float(eps), _stream()),
            "moe_combine_norm")
+
+
+JOIN_MAX_TOP = 32
+
+
+def join_branches(x: torch.Tensor, branches: list, mixture: tuple | None = None, norm: tuple | None = None) -> torch.Tensor | None:
+    """x (float32 [T, W]) += sum over `branches` (at most two (y, gain) pairs, float32 [T, W] and [W]) of gain * y, plus, with `mixture`
+    = (y, pair_row, weight, gain, shared, z): gain * (sum_k weight[t, k] * y[pair_row[t, k]] + sigmoid(z[t]) * shared[t]), shared
+    float32 [T, W] or None, z a float32 column [T, 1] or None (factor 1).  `norm` = (gain, eps, out): out = the RMS norm of the new
+    rows, which is also returned.  One kernel, one block a token."""
+    _need(x, "x", torch.float32, 2)
+    T, W = x.shape
+    if len(branches) > 2:
+        raise KernelError("join_branches: at most two plain branches")
+    for y, g in branches:
+        _need(y, "branch", torch.float32, 2); _f32(g, "gain", W)
+        if y.shape != x.shape or g is None:
+            raise KernelError(f"join_branches: a branch of {tuple(y.shape)} for rows {tuple(x.shape)}")
+    pad = list(branches) + [(None, None)] * (2 - len(branches))
+    y = pair_row = weight = gain = shared = z = h = ngain = None
+    top, ldz, eps = 0, 0, 0.0
+    if mixture is not None:
+        y, pair_row, weight, gain, shared, z = mixture
+        _need(y, "routed", torch.float32, 2); _need(pair_row, "pair_row", torch.int32, 2); _need(weight, "weight", torch.float32, 2)
+        _f32(gain, "gain", W)
+        top = pair_row.shape[1]
+        if y.shape[1] != W or pair_row.shape[0] != T or weight.shape != pair_row.shape or gain is None or top > JOIN_MAX_TOP:
+            raise KernelError(f"join_branches: routed rows {tuple(y.shape)}, pairs {tuple(pair_row.shape)} for rows {tuple(x.shape)}")
+        if shared is not None:
+            _need(shared, "shared", torch.float32, 2)
+            if shared.shape != x.shape:
+                raise KernelError("join_branches: the shared expert's rows differ in shape")
+        if z is not None:
+            if z.dtype != torch.float32 or z.shape != (T, 1):
+                raise KernelError("join_branches: the shared expert's gate is one float32 a token")
+            ldz = z.stride(0)
+    if norm is not None:
+        ngain, eps, h = norm
+        _need(ngain, "norm gain", None, 1); _need(h, "normed rows", None, 2)
+        if ngain.shape[0] != W or h.shape != x.shape:
+            raise KernelError("join_branches: the norm does not fit the rows")
+    _check(_lib().hymt2_join_branches(_ptr(x), _ptr(pad[0][0]), _ptr(pad[0][1]), _ptr(pad[1][0]), _ptr(pad[1][1]), _ptr(y), _ptr(pair_row),
+                                      _ptr(weight), c_int(top), _ptr(gain), _ptr(shared), _ptr(z), c_long(ldz), _ptr(h),
+                                      c_int(dtype_code(h.dtype) if h is not None else F32), _ptr(ngain),
+                                      c_int(dtype_code(ngain.dtype) if ngain is not None else F32), c_float(eps), c_int(T), c_int(W), _stream()),
+           "join_branches")
+    return h
 
 
 # -- a residual kept as several streams --------------------------------------------------------------------------------------------

@@ -221,6 +221,98 @@ class SandwichBlock:
 register_part("block", "sandwich", SandwichBlock)
 
 
+class ParallelBlock:
+    """A block whose sublayers read the same rows, the output of one norm, and join the residual together:
+
+        h = norm(x);   x <- x + gain_m * mixer(h) + gain_f * ff(h)          (no feed-forward: the last term is absent)
+
+    gain_m and gain_f are stored vectors of the model's width (`mixer_gain`, `ff_gain`: their names), applied entry by entry in
+    float32.  The sublayers store into float32 buffers of their own; one kernel adds them to the residual, a mixture of
+    experts from its experts' rows (a feed-forward that offers `pieces`), and norms the new rows for the block that runs next
+    when that is a parallel block too (`ctx.block_ahead`); those rows wait in `ctx.shared["parallel_rows"]`."""
+
+    def __init__(self, norm: PartSpec, mixer: PartSpec, mixer_gain: str, feed_forward: PartSpec | None = None, ff_gain: str | None = None):
+        if (feed_forward is None) != (ff_gain is None):
+            raise ValueError("a feed-forward comes with the name of its gain")
+        self.norm = build_part("norm", norm)
+        self.mixer = build_part("mixer", mixer)
+        self.feed_forward = build_part("feed_forward", feed_forward) if feed_forward is not None else None
+        self.names = [mixer_gain, ff_gain]
+        self.gains = [None, None]
+
+    def parts(self):
+        return tuple(p for p in (self.norm, self.mixer, self.feed_forward) if p is not None)
+
+    def cache_needs(self) -> list:
+        return [self.mixer.cache_need()]
+
+    def state_bytes(self) -> list:
+        return [int(self.mixer.state_bytes())]
+
+    @property
+    def graph_safe(self) -> bool:
+        return all(getattr(p, "graph_safe", False) for p in self.parts())
+
+    def tensors(self):
+        from ..weights.loader import TensorSpec
+        t = {}
+        for p in self.parts():
+            t.update(p.tensors())
+        for name in self.names:
+            if name is not None:
+                t[name] = TensorSpec((self.norm.dim,), init="gain")
+        return t
+
+    def load(self, weights, device, dtype):
+        for p in self.parts():
+            p.load(weights, device, dtype)
+        self.gains = [None if name is None else weights[name].to(device).float().contiguous() for name in self.names]
+
+    def first_norm(self):
+        return None   # (its rows come from the sum at the end of the block in front, not from a product)
+
+    @staticmethod
+    def _stored(part, h, like, ctx, *slot):
+        import torch
+        y = torch.empty(like.shape, dtype=torch.float32, device=like.device)
+        if getattr(part, "can_store", False):
+            part.forward(h, y, ctx, *slot, store=True)
+        else:
+            y.zero_()
+            part.forward(h, y, ctx, *slot)
+        return y
+
+    def forward(self, residual, ctx, slots) -> None:
+        import torch
+        ctx.weights_ahead = ctx.norm_ahead = ctx.prenormed = None
+        left = ctx.shared.pop("parallel_rows", None)
+        if left is not None and left[0] is residual and left[1] is self:
+            h = left[2]
+        else:
+            h = self.norm.forward(residual, ctx, ctx.dtype, fresh=True)
+        ff = self.feed_forward
+        branches = [(self._stored(self.mixer, h, residual, ctx, slots[0]), self.gains[0])]
+        mixture = None
+        if ff is not None:
+            pieces = ff.pieces(h, ctx) if hasattr(ff, "pieces") else None
+            if pieces is not None:
+                y, pair_row, weight, shared, z = pieces
+                mixture = (y, pair_row, weight, self.gains[1], shared, z)
+            else:
+                branches.append((self._stored(ff, h, residual, ctx), self.gains[1]))
+        ctx.prenormed = None
+        nxt = ctx.block_ahead
+        if not isinstance(nxt, ParallelBlock) or getattr(nxt.norm, "groups", 0) != 1:
+            ops.join_branches(residual, branches, mixture)
+            return
+        rows = torch.empty(residual.shape, dtype=ctx.dtype, device=residual.device)
+        ops.join_branches(residual, branches, mixture, (nxt.norm.gain, nxt.norm.eps, rows))
+        ctx.shared["parallel_rows"] = (residual, nxt, rows)
+
+
+register_part("block", "parallel", ParallelBlock)
+
+
 class StreamsBlock:
     """A pre-norm block over a residual that is kept as several streams (hyper-connections), with any number of mixers side
     by side.  X is float32 [streams, T, hidden]; for sublayer q (1: the mixers, 2: the feed-forward) with the stored vectors

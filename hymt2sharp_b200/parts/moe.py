@@ -9,7 +9,12 @@ the correction and not renormalised.  A shared expert (any feed-forward part) ru
 Chosen by parameters beyond that: a bias of the router (`router_bias`, a stored vector added to z); weights that are the
 softmax over the CHOSEN outputs only (`weights="chosen_softmax"`; the choice by score is then the choice by z); and gated
 experts, expert(x) = W_down (act(W_gate x) * (W_up x)) (`gate_proj` given; act "silu"): gate and up are one grouped product
-over the stacked matrices, and a small kernel applies the activation.
+over the stacked matrices, and a small kernel applies the activation.  The scores may be the sigmoid of each output
+(`scores="sigmoid"`), the weights the chosen scores' shares of their sum (`weights="chosen_share"`, `share_eps` added to the
+sum), and the choice limited to groups: the outputs form `groups` equal groups of neighbours, and only those of the `keep`
+groups whose two largest scores have the largest sums can be chosen.  The shared expert may have a gate per token
+(`shared_gate`, a stored [1, hidden] matrix): its output is multiplied by sigmoid(W x); that product is one more row of the
+router's.
 
 How a step runs: router product; `moe_route` (softmax, choice); `moe_place` sorts the (token, choice) pairs by expert, each
 expert's rows padded to whole row tiles; one grouped product per projection over the sorted rows (the first gathers its
@@ -27,7 +32,7 @@ from .linear import Linear, compute_form
 
 ACTIVATIONS = {"relu2": ops.EPILOGUE_RELU_SQUARED}      # experts without a gate: an epilogue of the grouped product
 GATED_ACTIVATIONS = {"silu": ops.GATED_SILU, "gelu_tanh": ops.GATED_GELU_TANH}
-WEIGHTS = ("scores", "chosen_softmax")
+WEIGHTS = ("scores", "chosen_softmax", "chosen_share")
 SKINNY_MAX_PAIRS = 512        # up to this many (token, choice) pairs in a step the kernel for few rows runs the experts,
 SKINNY_PAIRS_BESIDE_TC = 64   # where the tensor cores take the operands only up to this many: beyond, most experts meet several
                               # rows, and a row tile of 128 on the tensor cores, mostly empty, still reads each expert once
@@ -39,7 +44,8 @@ class RoutedExperts:
 
     def __init__(self, hidden: int, experts: int, identity: int, top: int, intermediate: int, activation: str, router: str,
                  up_proj: str, down_proj: str, correction: str | None = None, shared: PartSpec | None = None,
-                 gate_proj: str | None = None, router_bias: str | None = None, weights: str = "scores"):
+                 gate_proj: str | None = None, router_bias: str | None = None, weights: str = "scores", scores: str = "softmax",
+                 share_eps: float = 0.0, groups: int = 1, keep: int = 1, shared_gate: str | None = None):
         """`up_proj` / `down_proj` / `gate_proj`: the tensor names of expert e with `{}` in place of e."""
         known = GATED_ACTIVATIONS if gate_proj is not None else ACTIVATIONS
         if activation not in known:
@@ -47,13 +53,22 @@ class RoutedExperts:
                              f"(known: {', '.join(known)})")
         if weights not in WEIGHTS:
             raise ValueError(f"weights '{weights}' is not known (known: {', '.join(WEIGHTS)})")
-        self.gated, self.renormalise = gate_proj is not None, weights == "chosen_softmax"
+        if scores not in ops.SCORES or (weights == "chosen_softmax" and scores != "softmax"):
+            raise ValueError(f"scores '{scores}' with weights '{weights}': known scores are {', '.join(ops.SCORES)}, and the softmax over the "
+                             f"chosen outputs comes from softmax scores")
+        outputs = experts + identity
+        if groups < 1 or outputs % groups or not (0 < keep <= groups) or (groups > 1 and top > keep * (outputs // groups)):
+            raise ValueError(f"{outputs} outputs in {groups} groups of which {keep} are kept cannot give {top} choices")
+        if shared_gate is not None and shared is None:
+            raise ValueError("a gate of the shared expert needs a shared expert")
+        self.gated = gate_proj is not None
+        self.rule = ops.RouteRule(scores=scores, renormalise=weights != "scores", share_eps=float(share_eps), groups=int(groups), keep=int(keep))
         if experts < 0 or identity < 0 or not (0 < top <= experts + identity):
             raise ValueError(f"{top} of {experts} + {identity} experts cannot be chosen")
         self.hidden, self.experts, self.identity, self.top = int(hidden), int(experts), int(identity), int(top)
         self.intermediate, self.activation = int(intermediate), activation
-        self.names = dict(r=router, c=correction, u=up_proj, d=down_proj, g=gate_proj, b=router_bias)
-        self.bias = None
+        self.names = dict(r=router, c=correction, u=up_proj, d=down_proj, g=gate_proj, b=router_bias, sg=shared_gate)
+        self.bias = self.unit_gain = None
         self.shared = build_part("feed_forward", shared) if shared is not None else None
         self.router = self.correction = self.up = self.down = None
 
@@ -75,11 +90,16 @@ class RoutedExperts:
             t[n["d"].format(e)] = TensorSpec((self.hidden, self.intermediate))
         if self.shared is not None:
             t.update(self.shared.tensors())
+        if n["sg"] is not None:
+            t[n["sg"]] = TensorSpec((1, self.hidden))
         return t
 
     def load(self, weights, device, dtype):
         n = self.names
-        self.router = Linear(compute_form(weights[n["r"]], device, dtype), role="router")
+        rows = weights[n["r"]]
+        if n["sg"] is not None:    # the shared expert's gate is one more row of the router's product
+            rows = torch.cat([rows, weights[n["sg"]].to(rows.dtype)], dim=0)
+        self.router = Linear(compute_form(rows, device, dtype), role="router")
         self.correction = weights[n["c"]].to(device).float().contiguous() if n["c"] is not None else None
         self.bias = weights[n["b"]].to(device).float().contiguous() if n["b"] is not None else None
         if self.experts:
@@ -107,9 +127,11 @@ class RoutedExperts:
         return "tc" if tensor_cores else "simt"
 
     def _experts(self, x: torch.Tensor, ctx):
-        """Routing, the sorted rows and the experts' products: (y, pair_row, weight), y float32 [sorted rows, hidden]."""
+        """Routing, the sorted rows and the experts' products: (y, pair_row, weight, z), y float32 [sorted rows, hidden], z float32
+        [T, 1] the shared expert's gate in front of its sigmoid (None without one)."""
         T, dev = x.shape[0], x.device
         logits = self.router(x, out_dtype=torch.float32, ctx=ctx)
+        z = logits[:, self.outputs:] if self.names["sg"] is not None else None
         chosen = torch.empty((T, self.top), dtype=torch.int32, device=dev)
         weight = torch.empty((T, self.top), dtype=torch.float32, device=dev)
         kernel = self._grouped_kernel(x, T)
@@ -122,12 +144,12 @@ class RoutedExperts:
         counts = ints[T * self.top + tiles * tile + tiles + 1:]
         if T * self.top <= ops.MOE_SMALL_PAIRS and self.outputs <= 512:
             ops.moe_route_place(chosen, weight, pair_row, row_token, tile_group, logits, self.correction, self.experts, tile,
-                                self.bias, self.renormalise)
+                                self.bias, rule=self.rule, outputs=self.outputs)
         else:
-            ops.moe_route(chosen, weight, logits, self.correction, self.bias, self.renormalise)
+            ops.moe_route(chosen, weight, logits, self.correction, self.bias, rule=self.rule, outputs=self.outputs)
             ops.moe_place(pair_row, row_token, tile_group, counts, chosen, self.experts, tile)
         if not self.experts:
-            return torch.empty((1, self.hidden), dtype=torch.float32, device=dev), pair_row, weight   # y is never read
+            return torch.empty((1, self.hidden), dtype=torch.float32, device=dev), pair_row, weight, z   # y is never read
         rows, gather = x, True
         if kernel == "tc":     # its tiles come by TMA, which reads rows side by side
             rows, gather = torch.empty((tiles * tile, self.hidden), dtype=x.dtype, device=dev), False
@@ -145,14 +167,49 @@ class RoutedExperts:
         ops.tag = "experts_down"
         ops.gemm_grouped(kernel, y, act, self.down, tile_group, row_token, False, ops.EPILOGUE_STORE)
         ops.tag = None
-        return y, pair_row, weight
+        return y, pair_row, weight, z
+
+    def _shared_rows(self, x: torch.Tensor, ctx):
+        """The shared expert's output as float32 rows of its own."""
+        rows = torch.empty((x.shape[0], self.hidden), dtype=torch.float32, device=x.device)
+        if getattr(self.shared, "can_store", False):
+            self.shared.forward(x, rows, ctx, store=True)
+        else:
+            rows.zero_()
+            self.shared.forward(x, rows, ctx)
+        return rows
+
+    def pieces(self, x: torch.Tensor, ctx):
+        """What is left to add up: (y, pair_row, weight, shared, z) for ops.join_branches, a block's own sum.  None: this mixture has
+        outputs that are no rows of y (identity experts), or more choices than that kernel takes."""
+        if self.identity or self.top > ops.JOIN_MAX_TOP or not self.experts:
+            return None
+        y, pair_row, weight, z = self._experts(x, ctx)
+        shared = self._shared_rows(x, ctx) if self.shared is not None else None
+        ctx.prenormed = None
+        return y, pair_row, weight, shared, z
 
     def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, store: bool = False) -> None:
-        y, pair_row, weight = self._experts(x, ctx)
+        if self.names["sg"] is not None:
+            # the gated shared expert's rows are added up with the experts' by the kernel that a block uses for its own sum
+            pieces = self.pieces(x, ctx)
+            if pieces is None:
+                raise ValueError("a gate of the shared expert beside identity experts, or beside this many choices, is not built")
+            if store:
+                residual.zero_()
+            y, pair_row, weight, shared, z = pieces
+            ops.join_branches(residual, [], (y, pair_row, weight, self._ones(x.device), shared, z))
+            return
+        y, pair_row, weight, _ = self._experts(x, ctx)
         ops.moe_combine(residual, y, x, pair_row, weight, add=not store)
         if self.shared is not None:
             self.shared.forward(x, residual, ctx)
         ctx.prenormed = None
+
+    def _ones(self, device) -> torch.Tensor:
+        if self.unit_gain is None:
+            self.unit_gain = torch.ones(self.hidden, dtype=torch.float32, device=device)
+        return self.unit_gain
 
     def forward_then_norm(self, x: torch.Tensor, residual: torch.Tensor, norm, ctx, rows_dtype=None):
         """residual += norm(mixture(x)) for a block whose norm stands behind the sublayer: the experts' rows are added up,
@@ -160,15 +217,10 @@ class RoutedExperts:
         wanted), or False when this part cannot do it for this norm (the block then goes the long way)."""
         if getattr(norm, "groups", 1) != 1 or self.hidden > ops.MOE_COMBINE_NORM_MAX_WIDTH or norm.dim != self.hidden:
             return False
-        branch = None
-        if self.shared is not None:
-            branch = torch.empty_like(residual)
-            if getattr(self.shared, "can_store", False):
-                self.shared.forward(x, branch, ctx, store=True)
-            else:
-                branch.zero_()
-                self.shared.forward(x, branch, ctx)
-        y, pair_row, weight = self._experts(x, ctx)
+        if self.names["sg"] is not None:
+            return False
+        branch = self._shared_rows(x, ctx) if self.shared is not None else None
+        y, pair_row, weight, _ = self._experts(x, ctx)
         rows = torch.empty(residual.shape, dtype=rows_dtype, device=residual.device) if rows_dtype is not None else None
         ops.moe_combine_norm(residual, rows, branch, y, x, pair_row, weight, norm.gain, norm.eps)
         ctx.prenormed = None
