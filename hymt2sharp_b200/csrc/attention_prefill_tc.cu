@@ -26,6 +26,17 @@
 // more term in its denominator, of score 0 and without a value, added to a row's sum at the end.
 // Takes key and value sizes of 64 and 128 (in any pairing) and cache blocks of 64 tokens; other shapes stay with the
 // general kernel.
+//
+// Differential attention (FORM_MAPS, FORM_MAPS_CAPPED) has two softmax maps a head over the same values: o = a1 - lambda * a2,
+// then o / sqrt(mean(o^2) + eps) * factor over the head's DV entries.  A CTA takes one map, a cluster of two CTAs the head;
+// each reads its half of the head's query and key rows (2 D entries: map 1's, then map 2's), and behind the last tile the two
+// exchange half of their outputs through shared memory, so that each combines, norms and writes half of the head's columns.
+// A query's scores are multiplied by a temperature of its position.  With a cap C on the scores, C * tanh(s / C), a softmax
+// needs no running maximum: for C up to MAX_FIXED_CAP every exp(score) lies within float32's (and bfloat16's) range and
+// so do the sums, the numerators are taken as they are, and O is never rescaled.  tanh is the kernel's scarcest resource: while every
+// |s / C| of a warp's rows in a tile stays below 1 it is an odd polynomial on pairs of scores (two-wide float32 fused
+// multiply-adds), coefficients fitted for the smallest largest error over that range (2e-8, of an error of 1e-7 with float32's
+// own rounding); else it is 1 - 2 / (exp(2 x) + 1).  d = 32 (two maps side by side in one 128-byte row), 64 and 128 are taken.
 #include "tc_common.cuh"
 
 namespace {
@@ -50,7 +61,37 @@ struct PrefillParams {
     float scale_log2;          // scale * log2(e)
     int* status;
     int sink;
+    // differential attention
+    float scale, softcap, temp_coef;
+    int temp_every;
+    float lambda, eps, factor;
 };
+
+enum { FORM_CLASSIC = 0, FORM_MAPS = 1, FORM_MAPS_CAPPED = 2 };
+constexpr float MAX_FIXED_CAP = 60.f;
+
+// Two float32 side by side in a 64-bit register.
+__device__ __forceinline__ uint64_t pack2(float a, float b) {
+    uint64_t r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ void unpack2(uint64_t v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+    uint64_t r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
+    uint64_t r;
+    asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
 
 __device__ __forceinline__ float ex2_approx(float x) {
     float y;
@@ -68,12 +109,14 @@ __device__ __forceinline__ void tmem_store16(uint32_t taddr, const float* v) {
 }
 
 
-template <int D, int DV>
+template <int D, int DV, int FORM = FORM_CLASSIC>
 __global__ void __launch_bounds__(NUM_THREADS, 2)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, PrefillParams p) {
-    constexpr int D_BOXES = D / 64, DV_BOXES = DV / 64;     // TMA boxes of 64 elements along d and along dv
-    constexpr int Q_BYTES = Q_ROWS * D * 2, K_TILE_BYTES = KEY_TILE * D * 2, V_TILE_BYTES = KEY_TILE * DV * 2, P_BYTES = Q_ROWS * KEY_TILE * 2;
+    constexpr bool MAPS = FORM != FORM_CLASSIC;
+    constexpr int KD = D < 64 ? 64 : D;                     // entries of a query or key row that are loaded
+    constexpr int D_BOXES = KD / 64, DV_BOXES = DV / 64;    // TMA boxes of 64 elements along d and along dv
+    constexpr int Q_BYTES = Q_ROWS * KD * 2, K_TILE_BYTES = KEY_TILE * KD * 2, V_TILE_BYTES = KEY_TILE * DV * 2, P_BYTES = Q_ROWS * KEY_TILE * 2;
     // P of a tile (16 KB) takes the place of the tile's K (free once S is computed): a K slot holds the larger of the two
     constexpr int K_SLOT_BYTES = K_TILE_BYTES >= P_BYTES ? K_TILE_BYTES : P_BYTES;
     constexpr int BARS_OFFSET = Q_BYTES + K_SLOTS * K_SLOT_BYTES + KV_STAGES * V_TILE_BYTES;
@@ -94,9 +137,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     // ones start first and the short ones fill the gaps.  When all CTAs fit on the SMs at once (two each), the
     // ones beyond the first per SM are numbered by RISING length instead: the SM that got the longest tile also
     // gets the shortest.
-    int n = blockIdx.x;
-    const int total = gridDim.x, per_qtile = p.nh * p.batch;
-    if (total <= 2 * p.sm_count && n >= p.sm_count) n = p.sm_count + (total - 1 - n);
+    const int map = MAPS ? blockIdx.x & 1 : 0;             // (the two maps of a head are neighbours: one cluster)
+    int n = MAPS ? blockIdx.x >> 1 : blockIdx.x;
+    const int total = MAPS ? gridDim.x >> 1 : gridDim.x, per_qtile = p.nh * p.batch, first_wave = MAPS ? p.sm_count >> 1 : p.sm_count;
+    if (total <= 2 * first_wave && n >= first_wave) n = first_wave + (total - 1 - n);
     const int qtile = p.qtiles - 1 - n / per_qtile, head = (n % per_qtile) % p.nh, b = (n % per_qtile) / p.nh;
     const int slot = p.slot_ids[b];
     const int tok0 = p.cu_seqlens[b], T_b = p.cu_seqlens[b + 1] - tok0;
@@ -150,15 +194,18 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     __syncthreads();
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const uint32_t tmem_base = tmem_base_s;
+    bool ok = true;             // softmax threads: no wait gave up
+    float l = 0.f;              // and the sum of their row's numerators
 
     if (warp == 0 && lane == 0) {
         // ---- producer: Q with K(0), then K(i + 1) with V(i) ---------------------------------------
         const int* table = p.block_table + (size_t)slot * p.table_stride;
         auto cache_row = [&](int tile) { return (table[tile_begin + tile] * p.nkv + kvh) * KEY_TILE; };
         mbar_expect_tx(q_full, Q_BYTES + K_TILE_BYTES);
+        const int k_col = MAPS && D >= 64 ? map * D : 0, q_col = head * (MAPS ? 2 * D : D) + k_col;
         for (int x = 0; x < D_BOXES; x++) {
-            tma_load_2d(q_smem + x * (Q_ROWS * 128), &map_q, q_full, head * D + x * 64, tok0 + qtile * Q_ROWS);
-            tma_load_2d(k_of(0) + x * (KEY_TILE * 128), &map_k, q_full, x * 64, cache_row(0));
+            tma_load_2d(q_smem + x * (Q_ROWS * 128), &map_q, q_full, q_col + x * 64, tok0 + qtile * Q_ROWS);
+            tma_load_2d(k_of(0) + x * (KEY_TILE * 128), &map_k, q_full, k_col + x * 64, cache_row(0));
         }
         int issued = 0;
         for (int i = 0; i < num_tiles; i++) {
@@ -170,7 +217,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             const int v_row = cache_row(i), k_row = more ? cache_row(i + 1) : 0;
             const uint32_t k_dst = k_of(i + 1), v_dst = v_of(i);
             for (int x = 0; x < D_BOXES; x++)
-                if (more) tma_load_2d(k_dst + x * (KEY_TILE * 128), &map_k, kv_full + 8 * s, x * 64, k_row);
+                if (more) tma_load_2d(k_dst + x * (KEY_TILE * 128), &map_k, kv_full + 8 * s, k_col + x * 64, k_row);
             for (int x = 0; x < DV_BOXES; x++) tma_load_2d(v_dst + x * (KEY_TILE * 128), &map_v, kv_full + 8 * s, x * 64, v_row);
             issued = i + 1;
         }
@@ -185,7 +232,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         // the slowest link of the chain.
         // The descriptors of slot 0 once; per instruction only constants are added (the address sits in the
         // low bits in units of 16 bytes, and shared memory is too small to carry out of them).
-        const uint64_t q_desc = desc_k_major(q_smem), k_desc0 = desc_k_major(k_smem);
+        const int in_row = MAPS && D < 64 ? map * D * 2 : 0;   // bytes: where the map's entries begin in a loaded row
+        const uint64_t q_desc = desc_k_major(q_smem) + (in_row >> 4), k_desc0 = desc_k_major(k_smem) + (in_row >> 4);
         constexpr uint64_t K_STEP = K_SLOT_BYTES >> 4;
         // S(i) = Q K(i)^T over d in steps of 16, into the S buffer of i's parity.  K(i) has landed; the buffer's
         // last scores, those of tile i - 2, have been read: the softmax warps read a tile's scores before they
@@ -199,12 +247,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             }
             umma_commit(s_full + 8 * (i & 1));
         };
-        bool ok = mbar_wait(q_full, 0, abort_flag, p.status, 112);
-        if (ok) {
+        const bool landed = mbar_wait(q_full, 0, abort_flag, p.status, 112);
+        if (landed) {
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             issue_scores(0);
         }
-        for (int i = 0; ok && i + 1 < num_tiles; i++) {
+        for (int i = 0; landed && i + 1 < num_tiles; i++) {
             // K(i + 1) has landed (with V(i))
             if (!mbar_wait(kv_full + 8 * (i % KV_STAGES), (i / KV_STAGES) & 1, abort_flag, p.status, 113)) break;
             mbar_arrive(kv_empty + 8 * (i % KV_STAGES));   // seen: the stage may be filled again once P·V of tile i is through too
@@ -239,8 +287,25 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const int pos = first_pos + r;                                  // position of this row's query
         const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
         const bool row_ok = r < rows_here;
-        float m = -INFINITY, l = 0.f;
-        bool ok = true;
+        float m = -INFINITY;
+        float scale_log2 = p.scale_log2, row_scale = p.scale;
+        if constexpr (MAPS) {
+            if (p.temp_coef != 0.f) {
+                const float temp = 1.0f + p.temp_coef * logf((float)((pos + 1) / p.temp_every + 1));
+                scale_log2 *= temp;
+                row_scale *= temp;
+            }
+        }
+        // capped scores: exp(C tanh(x)) = 2^(x * (a polynomial in x^2)) with the factor C log2(e) in the coefficients
+        const float cap_log2 = p.softcap * 1.4426950408889634f, to_x = FORM == FORM_MAPS_CAPPED ? row_scale / p.softcap : 0.f;
+        uint64_t c2[7], x2 = 0, lsum[2] = {0, 0};
+        if constexpr (FORM == FORM_MAPS_CAPPED) {
+            constexpr float c[7] = {0.9999997019767761f, -0.33332130312919617f, 0.13319583237171173f, -0.05326583608984947f,
+                                    0.019973281770944595f, -0.005951280705630779f, 0.0009637721814215183f};
+#pragma unroll
+            for (int k = 0; k < 7; k++) c2[k] = pack2(c[k] * cap_log2, c[k] * cap_log2);
+            x2 = pack2(to_x, to_x);
+        }
         for (int i = 0; i < num_tiles; i++) {
             if (!(ok = mbar_wait(s_full + 8 * (i & 1), (i >> 1) & 1, abort_flag, p.status, 115))) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -248,6 +313,58 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             float s[KEY_TILE];
             tmem_load32(lane_addr + S_COL + 64 * (i & 1), s);
             tmem_load32(lane_addr + S_COL + 64 * (i & 1) + 32, s + 32);
+            const uint32_t p_dst = k_of(i);
+            if constexpr (FORM == FORM_MAPS_CAPPED) {
+                const bool edge = __any_sync(0xffffffffu, !row_ok || key0 + KEY_TILE - 1 > pos);
+                if (edge) {   // (what lies behind a row's position, or was never written, counts as 0 until its numerator is dropped)
+#pragma unroll
+                    for (int c = 0; c < KEY_TILE; c++) s[c] = (row_ok && key0 + c <= pos) ? s[c] : 0.f;
+                }
+                float mx[2] = {0.f, 0.f};
+#pragma unroll
+                for (int c = 0; c < KEY_TILE; c += 2) mx[(c >> 1) & 1] = fmaxf(mx[(c >> 1) & 1], fmaxf(fabsf(s[c]), fabsf(s[c + 1])));
+                const bool wide = __any_sync(0xffffffffu, !(fmaxf(mx[0], mx[1]) * fabsf(to_x) <= 1.0f));
+                auto numerators = [&](auto of_pair) {
+#pragma unroll
+                    for (int c8 = 0; c8 < KEY_TILE / 8; c8++) {
+                        uint32_t packed[4];
+#pragma unroll
+                        for (int j = 0; j < 4; j++) {
+                            const int c = c8 * 8 + 2 * j;
+                            float p0, p1;
+                            of_pair(s[c], s[c + 1], p0, p1);
+                            if (edge) {
+                                p0 = (row_ok && key0 + c <= pos) ? p0 : 0.f;
+                                p1 = (row_ok && key0 + c + 1 <= pos) ? p1 : 0.f;
+                            }
+                            lsum[j & 1] = add2(lsum[j & 1], pack2(p0, p1));
+                            const __nv_bfloat162 h = __floats2bfloat162_rn(p0, p1);
+                            packed[j] = *reinterpret_cast<const uint32_t*>(&h);
+                        }
+                        const uint32_t dst = p_dst + r * 128 + ((c8 ^ (r & 7)) << 4);
+                        asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(dst), "r"(packed[0]), "r"(packed[1]),
+                                     "r"(packed[2]), "r"(packed[3]) : "memory");
+                    }
+                };
+                if (!wide) {
+                    numerators([&](float s0, float s1, float& p0, float& p1) {
+                        const uint64_t x = mul2(pack2(s0, s1), x2), u = mul2(x, x);
+                        uint64_t q = c2[6];
+#pragma unroll
+                        for (int k = 5; k >= 0; k--) q = fma2(q, u, c2[k]);
+                        float e0, e1;
+                        unpack2(mul2(q, x), e0, e1);
+                        p0 = ex2_approx(e0);
+                        p1 = ex2_approx(e1);
+                    });
+                } else {
+                    const float twice = 2.0f * 1.4426950408889634f * to_x;
+                    numerators([&](float s0, float s1, float& p0, float& p1) {   // exp(2x) = inf and 0 give tanh 1 and -1
+                        p0 = ex2_approx(fmaf(__fdividef(1.0f, ex2_approx(s0 * twice) + 1.0f), -2.0f * cap_log2, cap_log2));
+                        p1 = ex2_approx(fmaf(__fdividef(1.0f, ex2_approx(s1 * twice) + 1.0f), -2.0f * cap_log2, cap_log2));
+                    });
+                }
+            } else {
             // s stays unscaled: the scale (> 0) goes into the exponent's multiply-add; most tiles lie wholly
             // inside the row's visible range and need no mask
             // four running maxima (and four sums below): one chain of 64 dependent operations would leave
@@ -264,7 +381,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     mx[c & 3] = fmaxf(mx[c & 3], s[c]);
                 }
             }
-            float tile_max = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * p.scale_log2;
+            float tile_max = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * scale_log2;
             // raise the row's maximum only when it grows by more than 2^8 (or at its first visible key)
             const bool raise = tile_max > m + 8.0f || (m == -INFINITY && tile_max > -INFINITY);
             const float corr = raise ? exp2f(m - tile_max) : 1.f;   // m = -inf: 0
@@ -287,7 +404,6 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             // a row that has seen no key yet (m = -inf) has only masked scores: -inf * scale + 0 = -inf, exp2 gives 0
             const float neg_m = m == -INFINITY ? 0.f : -m;
             // P as bfloat16 into the swizzled K-major tile: row r, 16-byte chunk c8 at chunk (c8 ^ (r & 7))
-            const uint32_t p_dst = k_of(i);
 #pragma unroll
             for (int c8 = 0; c8 < KEY_TILE / 8; c8++) {
                 uint32_t packed[4];
@@ -295,8 +411,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 for (int j = 0; j < 4; j++) {
                     // the special-function unit is this kernel's scarcest resource: one instruction an element
                     // (exp2f brings a range fix-up of several more; -inf gives 0 either way, and P has 8 bits)
-                    const float p0 = ex2_approx(fmaf(s[c8 * 8 + 2 * j], p.scale_log2, neg_m));
-                    const float p1 = ex2_approx(fmaf(s[c8 * 8 + 2 * j + 1], p.scale_log2, neg_m));
+                    const float p0 = ex2_approx(fmaf(s[c8 * 8 + 2 * j], scale_log2, neg_m));
+                    const float p1 = ex2_approx(fmaf(s[c8 * 8 + 2 * j + 1], scale_log2, neg_m));
                     const __nv_bfloat162 h = __floats2bfloat162_rn(p0, p1);
                     psum[j] += p0 + p1;
                     packed[j] = *reinterpret_cast<const uint32_t*>(&h);
@@ -306,6 +422,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                              "r"(packed[2]), "r"(packed[3]) : "memory");
             }
             l += (psum[0] + psum[1]) + (psum[2] + psum[3]);
+            }
             // rows of V at and past the sequence's length were never written by this sequence: their
             // weight is 0, but 0 x (whatever bits lie there) must stay 0.  Only a sequence's last tile has
             // such rows; V of the tile must have landed before they are overwritten.
@@ -326,7 +443,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         }
         if (ok) ok = mbar_wait(o_full + 8 * ((num_tiles - 1) % O_BARS), ((num_tiles - 1) / O_BARS) & 1, abort_flag, p.status, 117);
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        if (ok) {
+        if constexpr (FORM == FORM_MAPS_CAPPED) {
+            float a, b, c, d;
+            unpack2(lsum[0], a, b);
+            unpack2(lsum[1], c, d);
+            l = (a + b) + (c + d);
+        }
+        if (!MAPS && ok) {
             // the sink: a term exp2(0 - m) in the sum (m is the offset that every numerator of the row was taken against; a row
             // that sees a key has a finite one)
             if (p.sink && m > -INFINITY) l += exp2f(-m);
@@ -349,6 +472,62 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         }
     }
 
+    if constexpr (MAPS) {
+        // ---- the two maps of the head meet: every thread of both CTAs takes part in the three cluster barriers, whether or not a
+        // wait gave up above.  Shared memory of Q and of the keys is free: every product of this CTA is through.
+        constexpr int HALF = DV / 2;
+        static_assert(HALF * Q_ROWS * 4 <= K_SLOTS * K_SLOT_BYTES, "half of the outputs takes the keys' place");
+        asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+        __syncthreads();
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        const bool softmax_warp = warp >= 4;
+        const int quarter = warp & 3, r = quarter * 32 + lane;
+        const uint32_t lane_addr = tmem_base + ((uint32_t)(quarter * 32) << 16) + O_COL;
+        float* given = reinterpret_cast<float*>(smem_raw + Q_BYTES);          // [HALF columns][Q_ROWS]: the half that the other CTA writes out
+        float* squares = reinterpret_cast<float*>(smem_raw);                  // [Q_ROWS]
+        const float inv = ok && l > 0.f ? 1.0f / l : 0.f;
+        if (softmax_warp) {
+#pragma unroll
+            for (int c = 0; c < HALF; c += 32) {
+                float o[32];
+                tmem_load32(lane_addr + (map ^ 1) * HALF + c, o);
+#pragma unroll
+                for (int j = 0; j < 32; j++) given[(c + j) * Q_ROWS + r] = o[j] * inv;
+            }
+        }
+        __syncwarp();
+        cluster_sync_all();
+        float o[HALF], ss = 0.f;
+        if (softmax_warp) {
+#pragma unroll
+            for (int c = 0; c < HALF; c += 32) {
+                tmem_load32(lane_addr + map * HALF + c, o + c);
+#pragma unroll
+                for (int j = 0; j < 32; j++) {
+                    const float other = ld_cluster_f32(smem_u32(given + (c + j) * Q_ROWS + r), map ^ 1), own = o[c + j] * inv;
+                    o[c + j] = map == 0 ? fmaf(-p.lambda, other, own) : fmaf(-p.lambda, own, other);
+                    ss = fmaf(o[c + j], o[c + j], ss);
+                }
+            }
+            squares[r] = ss;
+        }
+        __syncwarp();
+        cluster_sync_all();
+        if (softmax_warp && ok && r < rows_here) {
+            const float scale = p.factor / sqrtf((ss + ld_cluster_f32(smem_u32(squares + r), map ^ 1)) / (float)DV + p.eps);
+            __nv_bfloat16* dst = p.out + ((size_t)(tok0 + qtile * Q_ROWS + r) * p.nh + head) * DV + map * HALF;
+#pragma unroll
+            for (int j = 0; j < HALF; j += 8) {
+                __nv_bfloat162 h[4];
+#pragma unroll
+                for (int q = 0; q < 4; q++) h[q] = __floats2bfloat162_rn(o[j + 2 * q] * scale, o[j + 2 * q + 1] * scale);
+                *reinterpret_cast<uint4*>(dst + j) = *reinterpret_cast<uint4*>(h);
+            }
+        }
+        __syncwarp();
+        cluster_sync_all();   // a CTA keeps its shared memory until the other has read it
+    }
+
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
     __syncthreads();
     if (warp == 1) {
@@ -357,13 +536,14 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     }
 }
 
-template <int D, int DV>
+template <int D, int DV, int FORM = FORM_CLASSIC>
 int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const PrefillParams& p, dim3 grid,
            cudaStream_t stream) {
-    constexpr size_t k_tile = KEY_TILE * D * 2, v_tile = KEY_TILE * DV * 2, p_tile = Q_ROWS * KEY_TILE * 2;
-    constexpr size_t smem = Q_ROWS * D * 2 + K_SLOTS * (k_tile >= p_tile ? k_tile : p_tile) + KV_STAGES * v_tile +
+    constexpr int kd = D < 64 ? 64 : D;
+    constexpr size_t k_tile = KEY_TILE * kd * 2, v_tile = KEY_TILE * DV * 2, p_tile = Q_ROWS * KEY_TILE * 2;
+    constexpr size_t smem = Q_ROWS * kd * 2 + K_SLOTS * (k_tile >= p_tile ? k_tile : p_tile) + KV_STAGES * v_tile +
                             NUM_BARS * 8 + 8;   // tiles, barriers, two words
-    auto kernel = attention_prefill_tc_kernel<D, DV>;
+    auto kernel = attention_prefill_tc_kernel<D, DV, FORM>;
     static bool configured = false;
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -371,8 +551,31 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
         cudaFuncSetAttribute(kernel, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);   // two CTAs an SM
         configured = true;
     }
-    kernel<<<grid, NUM_THREADS, smem, stream>>>(mq, mk, mv, p);
-    return hymt2_check_launch("attention_prefill_tc");
+    if constexpr (FORM != FORM_CLASSIC) {   // the two maps of a head are a cluster
+        cudaLaunchConfig_t cfg = {};
+        cfg.gridDim = grid;
+        cfg.blockDim = dim3(NUM_THREADS);
+        cfg.dynamicSmemBytes = smem;
+        cfg.stream = stream;
+        cudaLaunchAttribute attr[1];
+        attr[0].id = cudaLaunchAttributeClusterDimension;
+        attr[0].val.clusterDim.x = 2;
+        attr[0].val.clusterDim.y = 1;
+        attr[0].val.clusterDim.z = 1;
+        cfg.attrs = attr;
+        cfg.numAttrs = 1;
+        const cudaError_t e = cudaLaunchKernelEx(&cfg, kernel, mq, mk, mv, p);
+        if (e != cudaSuccess) { hymt2_set_error("attention_prefill_tc: %s", cudaGetErrorString(e)); return HYMT2_ERR_LAUNCH; }
+        return HYMT2_OK;
+    } else {
+        kernel<<<grid, NUM_THREADS, smem, stream>>>(mq, mk, mv, p);
+        return hymt2_check_launch("attention_prefill_tc");
+    }
+}
+
+template <int D, int DV>
+int launch_maps(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const PrefillParams& p, dim3 grid, cudaStream_t stream) {
+    return p.softcap > 0.f ? launch<D, DV, FORM_MAPS_CAPPED>(mq, mk, mv, p, grid, stream) : launch<D, DV, FORM_MAPS>(mq, mk, mv, p, grid, stream);
 }
 
 }  // namespace
@@ -409,7 +612,7 @@ HYMT2_API int hymt2_attention_prefill_tc_kv(void* out, const void* q, const void
     cudaGetDevice(&dev);
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
     PrefillParams p{(__nv_bfloat16*)out, block_table, cu_seqlens, slot_ids, kv_lens, table_stride, nh, nkv, window,
-                    batch, qtiles, sms, scale * 1.4426950408889634f, status, sink};
+                    batch, qtiles, sms, scale * 1.4426950408889634f, status, sink, scale};
     dim3 grid((unsigned)(qtiles * nh * batch), 1, 1);
     if (d == 128) return dv == 128 ? launch<128, 128>(mq, mk, mv, p, grid, stream) : launch<128, 64>(mq, mk, mv, p, grid, stream);
     return dv == 128 ? launch<64, 128>(mq, mk, mv, p, grid, stream) : launch<64, 64>(mq, mk, mv, p, grid, stream);
@@ -423,4 +626,37 @@ HYMT2_API int hymt2_attention_prefill_tc(void* out, const void* q, const void* k
                                          int* status, cudaStream_t stream) {
     return hymt2_attention_prefill_tc_kv(out, q, k_cache, v_cache, cache_blocks, block_table, table_stride, block_tokens, cu_seqlens,
                                          slot_ids, kv_lens, batch, tokens, max_new_tokens, nh, nkv, d, d, scale, window, 0, status, stream);
+}
+
+// Differential attention: q rows of nh * 2 * d entries (row stride ldq), keys' rows of 2 * d, out [tokens, nh * dv].  softcap 0: scores
+// as they are; else at most MAX_FIXED_CAP.
+HYMT2_API int hymt2_attention_prefill_tc_maps(void* out, const void* q, long ldq, const void* k_cache, const void* v_cache, long cache_blocks,
+                                              const int* block_table, int table_stride, int block_tokens, const int* cu_seqlens,
+                                              const int* slot_ids, const int* kv_lens, int batch, int tokens, int max_new_tokens, int nh,
+                                              int nkv, int d, int dv, float scale, float softcap, float temp_coef, int temp_every,
+                                              float lambda, float eps, float factor, int* status, cudaStream_t stream) {
+    if (tokens == 0 || batch == 0) return HYMT2_OK;
+    HYMT2_REQUIRE((d == 32 || d == 64 || d == 128) && (dv == 64 || dv == 128), "attention_prefill_tc: maps of %d and values of %d are not taken", d, dv);
+    HYMT2_REQUIRE(block_tokens == KEY_TILE, "attention_prefill_tc: cache blocks must hold %d tokens", KEY_TILE);
+    HYMT2_REQUIRE(nh > 0 && nkv > 0 && nh % nkv == 0 && batch <= 65535 && nh <= 65535 && ldq >= (long)nh * 2 * d && ldq % 8 == 0, "attention_prefill_tc: bad sizes");
+    HYMT2_REQUIRE(softcap >= 0.f && softcap <= MAX_FIXED_CAP && scale > 0.f && temp_every > 0, "attention_prefill_tc: a cap of %g is not taken", (double)softcap);
+    HYMT2_REQUIRE(((uintptr_t)q % 16 == 0) && ((uintptr_t)k_cache % 16 == 0) && ((uintptr_t)v_cache % 16 == 0) &&
+                  ((uintptr_t)out % 16 == 0), "attention_prefill_tc: tensors must be 16-byte aligned");
+    HYMT2_REQUIRE(status != nullptr, "attention_prefill_tc: a status word is needed");
+    CUtensorMap mq, mk, mv;
+    const long cache_rows = cache_blocks * nkv * KEY_TILE;
+    const bool ok = make_map(&mq, q, tokens, (long)nh * 2 * d, ldq, Q_ROWS) &&
+                    make_map(&mk, k_cache, cache_rows, 2 * d, 2 * d, KEY_TILE) && make_map(&mv, v_cache, cache_rows, dv, dv, KEY_TILE);
+    HYMT2_REQUIRE(ok, "attention_prefill_tc: cuTensorMapEncodeTiled refused the operands");
+    const int qtiles = (max_new_tokens + Q_ROWS - 1) / Q_ROWS;
+    HYMT2_REQUIRE((long)qtiles * nh * batch * 2 <= 2147483647L, "attention_prefill_tc: too many tiles");
+    int dev = 0, sms = 148;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+    PrefillParams p{(__nv_bfloat16*)out, block_table, cu_seqlens, slot_ids, kv_lens, table_stride, nh, nkv, 0,
+                    batch, qtiles, sms, scale * 1.4426950408889634f, status, 0, scale, softcap, temp_coef, temp_every, lambda, eps, factor};
+    dim3 grid((unsigned)(qtiles * nh * batch * 2), 1, 1);
+    if (d == 128) return dv == 128 ? launch_maps<128, 128>(mq, mk, mv, p, grid, stream) : launch_maps<128, 64>(mq, mk, mv, p, grid, stream);
+    if (d == 64) return dv == 128 ? launch_maps<64, 128>(mq, mk, mv, p, grid, stream) : launch_maps<64, 64>(mq, mk, mv, p, grid, stream);
+    return dv == 128 ? launch_maps<32, 128>(mq, mk, mv, p, grid, stream) : launch_maps<32, 64>(mq, mk, mv, p, grid, stream);
 }

@@ -124,3 +124,19 @@ def try_attention_kv(out, q, k_plane, v_plane, block_table, ctx, nh, nkv, d, dv,
                                     ctx.max_new_tokens, nh, nkv, d, dv, scale, window, sink, ops.device_status(out.device))
         return True
     return False
+
+
+def try_diff_attention(out, q, k_plane, v_plane, block_table, ctx, nh, nkv, d, dv, scale, softcap, temp_coef, temp_every, lam, eps, factor) -> bool:
+    """Differential attention with its two maps combined, in bfloat16 with cache blocks of 64 tokens: steps with pieces of several
+    tokens go to the tcgen05 kernel for maps of 32, 64 or 128 entries and values of 64 or 128.  False: the caller runs the
+    general kernel."""
+    if out.dtype != torch.bfloat16 or k_plane.shape[2] != 64 or scale <= 0 or not (0 <= softcap <= ops.DIFF_MAX_FIXED_CAP):
+        return False
+    if softcap == 0 and temp_coef < 0:      # (a running maximum wants scores that grow with the products)
+        return False
+    if ctx.decode or d not in (32, 64, 128) or dv not in (64, 128) or q.stride(0) % 8 or q.data_ptr() % 16:
+        return False
+    ops.attention_prefill_tc_maps(out, q, k_plane, v_plane, block_table, ctx.cu_seqlens, ctx.slot_ids, ctx.kv_lens, ctx.num_seqs,
+                                  ctx.max_new_tokens, nh, nkv, d, dv, scale, softcap, temp_coef, temp_every, lam, eps, factor,
+                                  ops.device_status(out.device))
+    return True

@@ -1246,6 +1246,32 @@ def attention_simt_maps(out: torch.Tensor, q: torch.Tensor, k_plane: torch.Tenso
            "attention_simt", 2 if split_keys > 0 else 1)
 
 
+DIFF_MAX_FIXED_CAP = 60.0   # up to this cap a score's exponential needs no offset in float32 (the tensor-core kernels' form of capped scores)
+
+
+def attention_prefill_tc_maps(out: torch.Tensor, q: torch.Tensor, k_plane: torch.Tensor, v_plane: torch.Tensor, block_table: torch.Tensor,
+                              cu_seqlens: torch.Tensor, slot_ids: torch.Tensor, kv_lens: torch.Tensor, batch: int, max_new_tokens: int, nh: int,
+                              nkv: int, d: int, dv: int, scale: float, softcap: float, temp_coef: float, temp_every: int, lam: float, eps: float,
+                              factor: float, status: torch.Tensor) -> None:
+    """Differential attention of a prompt's tokens on the tcgen05 tensor cores: attention_simt_maps with two maps and diff_combine behind it
+    in one kernel, bfloat16, maps of 32, 64 or 128 entries, values of 64 or 128, cache blocks of 64 tokens.  q may be the first
+    columns of wider rows."""
+    ldq = _rows_view(q, "q", torch.bfloat16)
+    _need(out, "out", torch.bfloat16, 2); _need(k_plane, "k_plane", torch.bfloat16, 4); _need(v_plane, "v_plane", torch.bfloat16, 4)
+    if out.shape[1] != nh * dv or q.shape[1] != nh * 2 * d or q.shape[0] < out.shape[0] or k_plane.shape[1] != nkv or k_plane.shape[3] != 2 * d \
+            or v_plane.shape != (*k_plane.shape[:3], dv):
+        raise KernelError(f"attention_prefill_tc: shapes out {tuple(out.shape)} q {tuple(q.shape)} k {tuple(k_plane.shape)} v {tuple(v_plane.shape)}")
+    _need(block_table, "block_table", torch.int32, 2)
+    for t, n in ((cu_seqlens, "cu_seqlens"), (slot_ids, "slot_ids"), (kv_lens, "kv_lens")):
+        _need(t, n, torch.int32, 1)
+    _check(_lib().hymt2_attention_prefill_tc_maps(_ptr(out), _ptr(q), c_long(ldq), _ptr(k_plane), _ptr(v_plane), c_long(k_plane.shape[0]),
+                                                  _ptr(block_table), c_int(block_table.stride(0)), c_int(k_plane.shape[2]), _ptr(cu_seqlens),
+                                                  _ptr(slot_ids), _ptr(kv_lens), c_int(batch), c_int(out.shape[0]), c_int(max_new_tokens),
+                                                  c_int(nh), c_int(nkv), c_int(d), c_int(dv), c_float(scale), c_float(softcap), c_float(temp_coef),
+                                                  c_int(temp_every), c_float(lam), c_float(eps), c_float(factor), _ptr(status), _stream()),
+           "attention_prefill_tc")
+
+
 def diff_combine(out: torch.Tensor, maps: torch.Tensor, nh: int, dv: int, lam: float, eps: float, factor: float) -> None:
     """out [T, nh * dv] = unit_rms(maps[t, h, 0] - lam * maps[t, h, 1]) * factor over the dv entries; maps [T, nh * 2 * dv] float32."""
     _need(out, "out", None, 2); _need(maps, "maps", torch.float32, 2)

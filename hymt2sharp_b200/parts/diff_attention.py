@@ -20,7 +20,7 @@ import math
 import torch
 
 from ..cache.allocator import GroupSpec
-from ..kernels import ops
+from ..kernels import fast, ops
 from ..weights.loader import TensorSpec
 from .attention import SPLIT_KEYS
 from .base import MixerSlot, register_part
@@ -91,6 +91,9 @@ class DiffAttention:
 
     def attend(self, out, q, k_plane, v_plane, table, ctx) -> None:
         T, H, G, d, dv = ctx.num_tokens, self.heads, self.kv_heads, self.dim, self.vdim
+        if fast.try_diff_attention(out, q, k_plane, v_plane, table, ctx, H, G, d, dv, self.scale, self.softcap, self.temp_coef, self.temp_every,
+                                   self.lam, self.eps, 1.0 - self.diff):
+            return
         split, max_splits, acc, ml = 0, 0, None, None
         if ctx.decode and ctx.max_kv_len > SPLIT_KEYS:
             split, max_splits = SPLIT_KEYS, -(-ctx.max_kv_len // SPLIT_KEYS)
