@@ -15,6 +15,13 @@
 // cache once per kv head (all heads of the group share it).  The warps that computed a
 // row's last chunk fold all chunks of the row in chunk order, each for its quarter of d.
 // Formulas: src/HyMT2Sharp/Ops.cs:462-532 (the reference's fused decode attention).
+//
+// MAPS 2 is differential attention: a head's query and key rows hold two maps of 64 entries, and its output is
+// o = a1 - lambda * a2, then o / sqrt(mean(o^2) + eps) * factor over the head's 128 entries.  The scores of a map are a
+// product over its 64 columns of the same tiles (accumulator columns 0 and 16), the numerators of both maps stand in one
+// operand of 16 rows (at most 8 heads per kv head), and one product makes both maps' sums.  A query's scores are multiplied by a temperature of its position
+// and may be capped, C * tanh(s / C).  Whoever folds a row has both maps' sums, combines them and norms them: the four warps
+// of the folding group exchange their quarters' sums of squares.
 #include "tc_common.cuh"
 
 namespace {
@@ -33,6 +40,10 @@ struct DecodeTcParams {
     int table_stride, nh, nkv, window, max_splits, rows;
     float scale_log2;
     int* status;
+    // differential attention
+    float softcap, temp_coef;
+    int temp_every;
+    float lambda, eps, factor;
 };
 
 constexpr int STAGES = 3;        // chunks whose keys and values are in shared memory or on their way
@@ -42,26 +53,29 @@ constexpr int MAX_CHUNKS = 2048; // chunks of one sequence (262,144 positions); 
 static_assert(MAX_CHUNKS <= 32767, "an item keeps chunk numbers in 16 bits");
 constexpr int FOLD_BATCH = 20;   // chunks whose partials are loaded together when a row is folded
 
-template <int G>   // query heads per kv head that the softmax loops cover (the group size rounded up)
+template <int G, int MAPS>   // query heads per kv head that the softmax loops cover (the group size rounded up); maps a head
 __global__ void __launch_bounds__(NUM_THREADS, 1)
 attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                            const __grid_constant__ CUtensorMap map_v, DecodeTcParams p) {
     // Persistent: a CTA takes the work items (sequence, kv head, chunk) w = blockIdx.x, + gridDim.x, ...
     // Per stage of shared memory: K [d half][128 keys x 128 B], V [key block][d half][64 keys x 128 B],
-    // Q [d half][16 x 128 B], P^T [key block][16 x 128 B].  Two (S^T, O^T) pairs alternate in tensor memory,
+    // Q [d half][16 x 128 B]; per group of softmax warps: P^T [key block][16 x 128 B] (a group writes its next P^T
+    // only after the sums of its last one are through).  Two (S^T, O^T) pairs alternate in tensor memory,
     // so the tensor core computes the next chunk's scores while the softmax warps work on this one.
-    constexpr int K_BYTES = CHUNK * D * 2, V_BYTES = CHUNK * D * 2, Q_BYTES = NQ * D * 2, P_BYTES = 2 * NQ * 128;
-    constexpr int STAGE_BYTES = K_BYTES + V_BYTES + Q_BYTES + P_BYTES;
+    constexpr int NP = NQ, MAP_ROWS = NP / MAPS, VG = G * MAPS;   // rows of P^T, and of one map; (map, head) pairs that a thread keeps
+    static_assert(G <= MAP_ROWS, "a map's heads fill its rows of P^T at most");
+    constexpr int K_BYTES = CHUNK * D * 2, V_BYTES = CHUNK * D * 2, Q_BYTES = NQ * D * 2, P_BYTES = 2 * NP * 128;
+    constexpr int STAGE_BYTES = K_BYTES + V_BYTES + Q_BYTES;
     constexpr int HALF_K = CHUNK * 128, BOX = BLOCK_KEYS * 128;
-    constexpr uint32_t TMEM_COLS = 64;   // buffer t: S^T at 32 t, O^T at 32 t + 16
+    constexpr uint32_t TMEM_COLS = 64 * MAPS, T_STEP = 32 * MAPS, O_AT = NQ * MAPS;   // buffer t: S^T at T_STEP t (16 columns a map), O^T at T_STEP t + O_AT
     constexpr uint32_t IDESC_S = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(NQ >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
-    constexpr uint32_t IDESC_O = IDESC_S | (1u << 15);
+    constexpr uint32_t IDESC_O = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 15) | ((uint32_t)(NP >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
 
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t bars[3 * STAGES + 8];
     __shared__ uint32_t tmem_base_s;
     __shared__ int abort_s;
-    __shared__ float red_max[2][4][NQ], red_sum[2][4][NQ];
+    __shared__ float red_max[2][4][VG], red_sum[2][4][VG];
     __shared__ int n_items_s;
 
     pdl_launch_dependents();
@@ -70,7 +84,7 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
     auto k_of = [&](int s) { return base + s * STAGE_BYTES; };
     auto v_of = [&](int s) { return base + s * STAGE_BYTES + K_BYTES; };
     auto q_of = [&](int s) { return base + s * STAGE_BYTES + K_BYTES + V_BYTES; };
-    auto p_of = [&](int s) { return base + s * STAGE_BYTES + K_BYTES + V_BYTES + Q_BYTES; };
+    auto p_of = [&](int t) { return base + STAGES * STAGE_BYTES + t * P_BYTES; };
     const uint32_t kq_full = smem_u32(&bars[0]), v_full = kq_full + 8 * STAGES, stage_free = kq_full + 16 * STAGES;
     const uint32_t s_done = smem_u32(&bars[3 * STAGES]), p_ready = s_done + 16, o_done = s_done + 32, tmem_free = s_done + 48;
     volatile int* abort_flag = &abort_s;
@@ -250,7 +264,8 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
                 for (int k = 0; k < D / 16; k++) {
                     constexpr int HALF_Q = NQ * 128;
                     const uint64_t k_off = ((k / 4) * HALF_K + (k % 4) * 32) >> 4, q_off = ((k / 4) * HALF_Q + (k % 4) * 32) >> 4;
-                    umma_bf16(tmem_base + 32 * t, kd + k_off, qd + q_off, IDESC_S, k > 0 ? 1u : 0u);
+                    if constexpr (MAPS == 1) umma_bf16(tmem_base + T_STEP * t, kd + k_off, qd + q_off, IDESC_S, k > 0 ? 1u : 0u);
+                    else umma_bf16(tmem_base + T_STEP * t + (k / 4) * NQ, kd + k_off, qd + q_off, IDESC_S, k % 4 > 0 ? 1u : 0u);   // a half of the columns a map
                 }
                 umma_commit(s_done + 8 * t);
             }
@@ -264,15 +279,15 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
                 if (!mbar_wait(p_ready + 8 * t, (uint32_t)((n >> 1) & 1), abort_flag, p.status, 127)) break;
                 if (!mbar_wait(v_full + 8 * s, (uint32_t)((n / STAGES) & 1), abort_flag, p.status, 129)) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                const uint64_t vd = v_desc0 + s * STAGE_STEP, pd = p_desc0 + s * STAGE_STEP;
+                const uint64_t vd = v_desc0 + s * STAGE_STEP, pd = p_desc0 + t * (P_BYTES >> 4);
                 const int blocks_here = items[n].blocks_here;
     #pragma unroll
                 for (int kb = 0; kb < 2; kb++) {
                     if (kb < blocks_here) {
     #pragma unroll
                         for (int k = 0; k < BLOCK_KEYS / 16; k++)
-                            umma_bf16(tmem_base + 32 * t + 16, vd + ((kb * 2 * BOX + k * (16 * 128)) >> 4),
-                                      pd + ((kb * (NQ * 128) + k * 32) >> 4), IDESC_O, (kb > 0 || k > 0) ? 1u : 0u);
+                            umma_bf16(tmem_base + T_STEP * t + O_AT, vd + ((kb * 2 * BOX + k * (16 * 128)) >> 4),
+                                      pd + ((kb * (NP * 128) + k * 32) >> 4), IDESC_O, (kb > 0 || k > 0) ? 1u : 0u);
                     }
                 }
                 umma_commit(o_done + 8 * t);
@@ -285,7 +300,7 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
             // ---- softmax (thread = key), then partial output (thread = d).  Two groups of four warps take turns:
             // group 0 the even items of this CTA with accumulator pair 0, group 1 the odd ones with pair 1.
             const int grp = (warp - 2) >> 2, quarter = warp & 3, t = quarter * 32 + lane;
-            const uint32_t lane_base = tmem_base + ((uint32_t)(quarter * 32) << 16) + 32 * grp;
+            const uint32_t lane_base = tmem_base + ((uint32_t)(quarter * 32) << 16) + T_STEP * grp;
             auto group_sync = [&]() {
                 if (grp == 0) asm volatile("bar.sync 1, 128;" ::: "memory");
                 else asm volatile("bar.sync 2, 128;" ::: "memory");
@@ -294,7 +309,7 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
             // The rows of P^T beyond the group are zero for good: their columns of O^T are never read, but must be
             // finite.  Nothing else writes there, so they are cleared once, before the first P^T of this CTA.
             if (round == 0) {
-                for (int i = threadIdx.x - 64; i < STAGES * P_BYTES / 16; i += 256)
+                for (int i = threadIdx.x - 64; i < 2 * P_BYTES / 16; i += 256)
                     asm volatile("st.shared.v4.b32 [%0], {%1, %1, %1, %1};" ::"r"(p_of(i / (P_BYTES / 16)) + (i % (P_BYTES / 16)) * 16), "r"(0) : "memory");
                 asm volatile("bar.sync 4, 256;" ::: "memory");
             }
@@ -305,39 +320,56 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
                 const int key = it.chunk_begin + t;
                 const bool visible = key >= it.lo && key <= it.pos;
                 const int head0 = it.kvh * g;
-                float sc[NQ];
+                float sc[VG], scale_log2 = p.scale_log2, capped = 0.f, twice = 0.f;
+                if constexpr (MAPS > 1) {
+                    if (p.temp_coef != 0.f) scale_log2 *= 1.0f + p.temp_coef * logf((float)((it.pos + 1) / p.temp_every + 1));
+                    if (p.softcap > 0.f) {
+                        capped = p.softcap * 1.4426950408889634f;
+                        twice = 2.0f * scale_log2 / p.softcap;    // exp(2 s / C) as a power of two
+                    }
+                }
                 if (!(ok = mbar_wait(s_done + 8 * grp, (uint32_t)(use & 1), abort_flag, p.status, 124))) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                tmem_load16(lane_base, sc);
     #pragma unroll
-                for (int h = 0; h < G; h++) sc[h] = (visible && h < g) ? sc[h] * p.scale_log2 : -INFINITY;
-                float mx[G];
+                for (int m = 0; m < MAPS; m++) {
+                    float raw[NQ];
+                    tmem_load16(lane_base + m * NQ, raw);
     #pragma unroll
-                for (int h = 0; h < G; h++) {
+                    for (int h = 0; h < G; h++) {
+                        float v = raw[h] * scale_log2;
+                        if (MAPS > 1 && capped > 0.f)   // C tanh(s / C) = C - 2 C / (exp(2 s / C) + 1)
+                            v = fmaf(__fdividef(1.0f, exp2f(raw[h] * twice) + 1.0f), -2.0f * capped, capped);
+                        sc[m * G + h] = (visible && h < g) ? v : -INFINITY;
+                    }
+                }
+                float mx[VG];
+    #pragma unroll
+                for (int h = 0; h < VG; h++) {
                     mx[h] = sc[h];
     #pragma unroll
                     for (int o = 16; o > 0; o >>= 1) mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], o));
                 }
                 group_sync();   // red_max and red_sum of this group's item before are read
-                if (lane < G) {
+                if (lane < VG) {
                     float mine = mx[0];
     #pragma unroll
-                    for (int h = 1; h < G; h++) mine = lane == h ? mx[h] : mine;
+                    for (int h = 1; h < VG; h++) mine = lane == h ? mx[h] : mine;
                     red_max[grp][quarter][lane] = mine;
                 }
                 group_sync();
-                float psum[G];
+                float psum[VG];
                 const int kb = t / BLOCK_KEYS, kin = t % BLOCK_KEYS;
-                const uint32_t p_dst = p_of(s);
+                const uint32_t p_dst = p_of(grp);
     #pragma unroll
-                for (int h = 0; h < G; h++) {
+                for (int h = 0; h < VG; h++) {
                     const float M = fmaxf(fmaxf(red_max[grp][0][h], red_max[grp][1][h]), fmaxf(red_max[grp][2][h], red_max[grp][3][h]));
                     const float pj = (M == -INFINITY || sc[h] == -INFINITY) ? 0.f : exp2f(sc[h] - M);
                     const __nv_bfloat16 pb = __float2bfloat16_rn(pj);
                     psum[h] = __bfloat162float(pb);   // the sum uses what the tensor core multiplies with
                     mx[h] = M;
-                    // P^T[h][key]: row h of the block's 16 x 128 B tile, 16-byte chunk (kin / 8) ^ (h & 7)
-                    const uint32_t dst = p_dst + kb * (NQ * 128) + h * 128 + ((((uint32_t)kin >> 3) ^ (h & 7)) << 4) + (kin & 7) * 2;
+                    // P^T[row][key], row = head, behind the map's first row: 16-byte chunk (kin / 8) ^ (row & 7) of the row's 128 bytes in the block's tile
+                    const int row = (h / G) * MAP_ROWS + h % G;
+                    const uint32_t dst = p_dst + kb * (NP * 128) + row * 128 + ((((uint32_t)kin >> 3) ^ (row & 7)) << 4) + (kin & 7) * 2;
                     asm volatile("st.shared.b16 [%0], %1;" ::"r"(dst), "h"(*reinterpret_cast<const unsigned short*>(&pb)) : "memory");
                 }
                 // rows of V at and past the sequence's length have never been written by this sequence, and the rows of
@@ -353,13 +385,13 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
                     }
                 }
     #pragma unroll
-                for (int h = 0; h < G; h++)
+                for (int h = 0; h < VG; h++)
     #pragma unroll
                     for (int o = 16; o > 0; o >>= 1) psum[h] += __shfl_xor_sync(0xffffffffu, psum[h], o);
-                if (lane < G) {
+                if (lane < VG) {
                     float mine = psum[0];
     #pragma unroll
-                    for (int h = 1; h < G; h++) mine = lane == h ? psum[h] : mine;
+                    for (int h = 1; h < VG; h++) mine = lane == h ? psum[h] : mine;
                     red_sum[grp][quarter][lane] = mine;
                 }
                 asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
@@ -368,23 +400,24 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
                 // partial output: thread = d
                 if (!(ok = mbar_wait(o_done + 8 * grp, (uint32_t)(use & 1), abort_flag, p.status, 126))) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                float o[NQ];
-                tmem_load16(lane_base + 16, o);
+                float o[NP];
+    #pragma unroll
+                for (int c = 0; c < NP; c += 16) tmem_load16(lane_base + O_AT + c, o + c);
                 asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
                 mbar_arrive(tmem_free + 8 * grp);   // this pair of accumulators may be filled again
                 group_sync();                       // red_sum of all four warps is written
     #pragma unroll
-                for (int h = 0; h < G; h++) {
-                    if (h < g) {
-                        const size_t row = ((size_t)it.b * p.nh + head0 + h) * p.max_splits + it.split;
-                        p.part_acc[row * D + t] = o[h];
+                for (int h = 0; h < VG; h++) {
+                    if (h % G < g) {
+                        const size_t row = (((size_t)it.b * p.nh + head0 + h % G) * MAPS + h / G) * p.max_splits + it.split;
+                        p.part_acc[row * D + t] = o[(h / G) * MAP_ROWS + h % G];
                     }
                 }
-                if (lane < g) {   // every warp keeps its own copy of (maximum, sum): a warp folds what warps of its quarter wrote
+                if (lane < VG && lane % G < g) {   // every warp keeps its own copy of (maximum, sum): a warp folds what warps of its quarter wrote
                     float mine = mx[0];
     #pragma unroll
-                    for (int h = 1; h < G; h++) mine = lane == h ? mx[h] : mine;
-                    const size_t row = ((size_t)it.b * p.nh + head0 + lane) * p.max_splits + it.split;
+                    for (int h = 1; h < VG; h++) mine = lane == h ? mx[h] : mine;
+                    const size_t row = (((size_t)it.b * p.nh + head0 + lane % G) * MAPS + lane / G) * p.max_splits + it.split;
                     *reinterpret_cast<float2*>(p.part_ml + (row * 4 + quarter) * 2) =
                         make_float2(mine, red_sum[grp][0][lane] + red_sum[grp][1][lane] + red_sum[grp][2][lane] + red_sum[grp][3][lane]);
                 }
@@ -400,26 +433,26 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
                 const Item& it = items[grp + 2 * lane];
                 atomicAdd(p.counters + ((size_t)it.b * p.nkv + it.kvh) * 4 + quarter, 1);
             }
-            for (int i = grp; ok && i < n_items; i += 2) {
+            // (with two maps the four warps of the group meet at a barrier for every row they fold: they all walk the same items, and a
+            // warp that gave up walks them too)
+            for (int i = grp; (ok || MAPS > 1) && i < n_items; i += 2) {
                 const Item& it = items[i];
                 const int s_begin = it.lo / CHUNK, n_chunks = it.pos / CHUNK + 1 - s_begin;
                 if (it.split != it.folder) continue;          // another CTA folds this row
                 int* counter = p.counters + ((size_t)it.b * p.nkv + it.kvh) * 4 + quarter;
                 int seen = 0;
-                if (lane == 0) {
+                if (lane == 0 && ok) {
                     uint32_t spins = 0;
                     while ((seen = *reinterpret_cast<volatile int*>(counter)) < n_chunks && ++spins < (1u << 22)) __nanosleep(20);
                     if (seen >= n_chunks) *counter = 0;          // ready for the next launch
                     else atomicExch(p.status, 128);              // a chunk never arrived: flag it, leave the row
                 }
                 seen = __shfl_sync(0xffffffffu, seen, 0);
-                if (seen < n_chunks) continue;
+                if (seen < n_chunks && MAPS == 1) continue;
                 __threadfence();
                 // a lane takes four neighbouring d of one head: 8 lanes per head, 4 heads per round
                 const int head0 = it.kvh * g;
-                for (int unit = lane; unit < g * 8; unit += 32) {
-                    const int h = unit >> 3, dd = quarter * 32 + (unit & 7) * 4;
-                    const size_t row = ((size_t)it.b * p.nh + head0 + h) * p.max_splits + s_begin;
+                auto fold = [&](size_t row, int dd) -> float4 {   // the quotient of one (map of a) head's four entries
                     float M = -INFINITY, L = 0.f;
                     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
                     for (int cb = 0; cb < n_chunks; cb += FOLD_BATCH) {
@@ -448,8 +481,50 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
                         M = Mb;
                     }
                     const float inv = L > 0.f ? 1.0f / L : 0.f;
-                    __nv_bfloat162 o2[2] = {__floats2bfloat162_rn(a.x * inv, a.y * inv), __floats2bfloat162_rn(a.z * inv, a.w * inv)};
+                    return make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv);
+                };
+                auto write = [&](int h, int dd, const float4& a) {
+                    __nv_bfloat162 o2[2] = {__floats2bfloat162_rn(a.x, a.y), __floats2bfloat162_rn(a.z, a.w)};
                     *reinterpret_cast<uint2*>(p.out + ((size_t)it.b * p.nh + head0 + h) * D + dd) = *reinterpret_cast<uint2*>(o2);
+                };
+                if constexpr (MAPS == 1) {
+                    for (int unit = lane; unit < g * 8; unit += 32) {
+                        const int h = unit >> 3, dd = quarter * 32 + (unit & 7) * 4;
+                        write(h, dd, fold(((size_t)it.b * p.nh + head0 + h) * p.max_splits + s_begin, dd));
+                    }
+                } else {
+                    constexpr int UNITS = (G * 8 + 31) / 32;
+                    const bool whole = seen >= n_chunks;
+                    float4 o[UNITS];
+    #pragma unroll
+                    for (int k = 0; k < UNITS; k++) {
+                        const int unit = lane + 32 * k, h = unit >> 3, dd = quarter * 32 + (unit & 7) * 4;
+                        o[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+                        if (whole && unit < g * 8) {
+                            const size_t row = ((size_t)it.b * p.nh + head0 + h) * 2 * p.max_splits + s_begin;
+                            const float4 a1 = fold(row, dd), a2 = fold(row + p.max_splits, dd);
+                            o[k] = make_float4(fmaf(-p.lambda, a2.x, a1.x), fmaf(-p.lambda, a2.y, a1.y), fmaf(-p.lambda, a2.z, a1.z), fmaf(-p.lambda, a2.w, a1.w));
+                        }
+                        float ss = fmaf(o[k].x, o[k].x, fmaf(o[k].y, o[k].y, fmaf(o[k].z, o[k].z, o[k].w * o[k].w)));
+    #pragma unroll
+                        for (int x = 1; x < 8; x <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+                        if ((lane & 7) == 0 && unit < g * 8) red_sum[grp][quarter][h] = ss;
+                    }
+                    auto fold_sync = [&]() {
+                        if (grp == 0) asm volatile("bar.sync 5, 128;" ::: "memory");
+                        else asm volatile("bar.sync 6, 128;" ::: "memory");
+                    };
+                    fold_sync();
+    #pragma unroll
+                    for (int k = 0; k < UNITS; k++) {
+                        const int unit = lane + 32 * k, h = unit >> 3, dd = quarter * 32 + (unit & 7) * 4;
+                        if (whole && unit < g * 8) {
+                            const float ss = red_sum[grp][0][h] + red_sum[grp][1][h] + red_sum[grp][2][h] + red_sum[grp][3][h];
+                            const float f = p.factor / sqrtf(ss / (float)D + p.eps);
+                            write(h, dd, make_float4(o[k].x * f, o[k].y * f, o[k].z * f, o[k].w * f));
+                        }
+                    }
+                    fold_sync();   // the sums have been read: the next row's may take their place
                 }
             }
         }
@@ -476,33 +551,31 @@ HYMT2_API int hymt2_attention_decode_tc_protocol(int* out) {
     return HYMT2_OK;
 }
 
-// out, q: [rows, nh * 128] bfloat16, one new token per row; k_cache, v_cache: one layer's planes
-// [blocks][nkv][64][128].  max_splits >= ceil(longest kv_len / 128); part_acc holds
-// rows*nh*max_splits*128 floats, part_ml rows*nh*max_splits*8, counters rows*nkv*4 zeroed ints.
-HYMT2_API int hymt2_attention_decode_tc(void* out, const void* q, const void* k_cache, const void* v_cache,
-                                        long cache_blocks, const int* block_table, int table_stride, int block_tokens,
-                                        const int* slot_ids, const int* kv_lens, int rows, int nh, int nkv, int d,
-                                        float scale, int window, int max_splits, float* part_acc, float* part_ml,
-                                        int* counters, int* status, cudaStream_t stream) {
+template <int MAPS>
+static int decode_tc_run(void* out, const void* q, const void* k_cache, const void* v_cache, long cache_blocks, const int* block_table,
+                         int table_stride, int block_tokens, const int* slot_ids, const int* kv_lens, int rows, int nh, int nkv, int d,
+                         float scale, int window, int max_splits, float* part_acc, float* part_ml, int* counters, int* status,
+                         float softcap, float temp_coef, int temp_every, float lambda, float eps, float factor, cudaStream_t stream) {
     if (rows == 0) return HYMT2_OK;
-    HYMT2_REQUIRE(d == D, "attention_decode_tc: head_dim %d is not taken (128 is)", d);
+    HYMT2_REQUIRE(d == D, "attention_decode_tc: rows of %d entries are not taken (128 are)", d);
     HYMT2_REQUIRE(block_tokens == BLOCK_KEYS, "attention_decode_tc: cache blocks must hold %d tokens", BLOCK_KEYS);
-    HYMT2_REQUIRE(nh > 0 && nkv > 0 && nh % nkv == 0 && nh / nkv <= NQ, "attention_decode_tc: at most %d heads per kv head", NQ);
+    HYMT2_REQUIRE(nh > 0 && nkv > 0 && nh % nkv == 0 && nh / nkv <= NQ / MAPS, "attention_decode_tc: at most %d heads per kv head", NQ / MAPS);
     HYMT2_REQUIRE(max_splits > 0 && max_splits <= MAX_CHUNKS, "attention_decode_tc: at most %d chunks of 128 keys are taken, got %d", MAX_CHUNKS, max_splits);
     HYMT2_REQUIRE(part_acc && part_ml && counters && status, "attention_decode_tc: scratch is needed");
     HYMT2_REQUIRE(rows <= MAX_ROWS, "attention_decode_tc: at most %d sequences in one launch, got %d", MAX_ROWS, rows);
+    HYMT2_REQUIRE(softcap >= 0.f && temp_every > 0, "attention_decode_tc: a cap of %g, a temperature every %d positions", (double)softcap, temp_every);
     CUtensorMap mq, mk, mv;
     const long cache_rows = cache_blocks * nkv * BLOCK_KEYS;
     const bool ok = make_map(&mq, q, (long)rows * nh, d, d, NQ) && make_map(&mk, k_cache, cache_rows, d, d, BLOCK_KEYS) &&
                     make_map(&mv, v_cache, cache_rows, d, d, BLOCK_KEYS);
     HYMT2_REQUIRE(ok, "attention_decode_tc: cuTensorMapEncodeTiled refused the operands");
     DecodeTcParams p{(__nv_bfloat16*)out, block_table, slot_ids, kv_lens, part_acc, part_ml, counters, table_stride, nh, nkv,
-                     window, max_splits, rows, scale * 1.4426950408889634f, status};
-    constexpr size_t smem = (size_t)STAGES * (2 * CHUNK * D * 2 + NQ * D * 2 + 2 * NQ * 128) + 1024;
+                     window, max_splits, rows, scale * 1.4426950408889634f, status, softcap, temp_coef, temp_every, lambda, eps, factor};
+    constexpr size_t smem = (size_t)STAGES * (2 * CHUNK * D * 2 + NQ * D * 2) + 2 * (2 * NQ * 128) + 1024;
     const int g = nh / nkv;
-    auto kernel = g <= 1 ? attention_decode_tc_kernel<1> : g <= 2 ? attention_decode_tc_kernel<2>
-                : g <= 4 ? attention_decode_tc_kernel<4> : g <= 8 ? attention_decode_tc_kernel<8>
-                : attention_decode_tc_kernel<16>;
+    auto kernel = g <= 1 ? attention_decode_tc_kernel<1, MAPS> : g <= 2 ? attention_decode_tc_kernel<2, MAPS>
+                : g <= 4 ? attention_decode_tc_kernel<4, MAPS> : g <= 8 ? attention_decode_tc_kernel<8, MAPS>
+                : attention_decode_tc_kernel<MAPS == 1 ? 16 : 8, MAPS>;
     static bool configured[5] = {};
     const int which = g <= 1 ? 0 : g <= 2 ? 1 : g <= 4 ? 2 : g <= 8 ? 3 : 4;
     if (!configured[which]) {
@@ -527,4 +600,26 @@ HYMT2_API int hymt2_attention_decode_tc(void* out, const void* q, const void* k_
     cudaError_t e = launch_pdl(kernel, dim3((unsigned)ctas), dim3(NUM_THREADS), smem, stream, mq, mk, mv, p);
     if (e != cudaSuccess) { hymt2_set_error("attention_decode_tc: %s", cudaGetErrorString(e)); return HYMT2_ERR_LAUNCH; }
     return hymt2_check_launch("attention_decode_tc");
+}
+
+// out, q: [rows, nh * 128] bfloat16, one new token per row; k_cache, v_cache: one layer's planes
+// [blocks][nkv][64][128].  max_splits >= ceil(longest kv_len / 128); part_acc holds
+// rows*nh*max_splits*128 floats, part_ml rows*nh*max_splits*8, counters rows*nkv*4 zeroed ints.
+HYMT2_API int hymt2_attention_decode_tc(void* out, const void* q, const void* k_cache, const void* v_cache,
+                                        long cache_blocks, const int* block_table, int table_stride, int block_tokens,
+                                        const int* slot_ids, const int* kv_lens, int rows, int nh, int nkv, int d,
+                                        float scale, int window, int max_splits, float* part_acc, float* part_ml,
+                                        int* counters, int* status, cudaStream_t stream) {
+    return decode_tc_run<1>(out, q, k_cache, v_cache, cache_blocks, block_table, table_stride, block_tokens, slot_ids, kv_lens, rows, nh, nkv, d,
+                            scale, window, max_splits, part_acc, part_ml, counters, status, 0.f, 0.f, 1, 0.f, 0.f, 1.f, stream);
+}
+
+// Differential attention with maps of 64 and values of 128 entries; the scratch is that of nh * 2 heads.
+HYMT2_API int hymt2_attention_decode_tc_maps(void* out, const void* q, const void* k_cache, const void* v_cache,
+                                             long cache_blocks, const int* block_table, int table_stride, int block_tokens,
+                                             const int* slot_ids, const int* kv_lens, int rows, int nh, int nkv, float scale, float softcap,
+                                             float temp_coef, int temp_every, float lambda, float eps, float factor, int max_splits,
+                                             float* part_acc, float* part_ml, int* counters, int* status, cudaStream_t stream) {
+    return decode_tc_run<2>(out, q, k_cache, v_cache, cache_blocks, block_table, table_stride, block_tokens, slot_ids, kv_lens, rows, nh, nkv, D,
+                            scale, 0, max_splits, part_acc, part_ml, counters, status, softcap, temp_coef, temp_every, lambda, eps, factor, stream);
 }

@@ -127,14 +127,25 @@ def try_attention_kv(out, q, k_plane, v_plane, block_table, ctx, nh, nkv, d, dv,
 
 
 def try_diff_attention(out, q, k_plane, v_plane, block_table, ctx, nh, nkv, d, dv, scale, softcap, temp_coef, temp_every, lam, eps, factor) -> bool:
-    """Differential attention with its two maps combined, in bfloat16 with cache blocks of 64 tokens: steps with pieces of several
-    tokens go to the tcgen05 kernel for maps of 32, 64 or 128 entries and values of 64 or 128.  False: the caller runs the
-    general kernel."""
-    if out.dtype != torch.bfloat16 or k_plane.shape[2] != 64 or scale <= 0 or not (0 <= softcap <= ops.DIFF_MAX_FIXED_CAP):
+    """Differential attention with its two maps combined, in bfloat16 with cache blocks of 64 tokens: decode steps go to the
+    tcgen05 decode kernel (maps of 64 entries, values of 128, at most 8 heads per kv head), steps with pieces of several tokens to
+    the tcgen05 prompt kernel (maps of 32, 64 or 128 entries, values of 64 or 128).  False: the caller runs the general kernel."""
+    if out.dtype != torch.bfloat16 or k_plane.shape[2] != 64:
         return False
-    if softcap == 0 and temp_coef < 0:      # (a running maximum wants scores that grow with the products)
+    if ctx.decode:
+        if (d, dv) != (64, 128) or nh // nkv > 8 or ctx.num_tokens > DECODE_TC_MAX_ROWS or ctx.max_kv_len > DECODE_TC_MAX_CHUNKS * DECODE_TC_CHUNK_KEYS:
+            return False
+        splits = max(1, -(-ctx.max_kv_len // DECODE_TC_CHUNK_KEYS))
+        na, nm, nc = ops.attention_decode_tc_scratch(ctx.num_tokens, 2 * nh, nkv, 128, splits)
+        acc = torch.empty(na, dtype=torch.float32, device=out.device)
+        ml = torch.empty(nm, dtype=torch.float32, device=out.device)
+        ops.attention_decode_tc_maps(out, q, k_plane, v_plane, block_table, ctx.slot_ids, ctx.kv_lens, nh, nkv, scale, softcap, temp_coef,
+                                     temp_every, lam, eps, factor, splits, acc, ml, ops.zeroed_counters(out.device, nc),
+                                     ops.device_status(out.device))
+        return True
+    if d not in (32, 64, 128) or dv not in (64, 128) or q.stride(0) % 8 or q.data_ptr() % 16 or scale <= 0 or not (0 <= softcap <= ops.DIFF_MAX_FIXED_CAP):
         return False
-    if ctx.decode or d not in (32, 64, 128) or dv not in (64, 128) or q.stride(0) % 8 or q.data_ptr() % 16:
+    if softcap == 0 and temp_coef < 0:      # (its running maximum wants scores that grow with the products)
         return False
     ops.attention_prefill_tc_maps(out, q, k_plane, v_plane, block_table, ctx.cu_seqlens, ctx.slot_ids, ctx.kv_lens, ctx.num_seqs,
                                   ctx.max_new_tokens, nh, nkv, d, dv, scale, softcap, temp_coef, temp_every, lam, eps, factor,

@@ -1246,6 +1246,30 @@ def attention_simt_maps(out: torch.Tensor, q: torch.Tensor, k_plane: torch.Tenso
            "attention_simt", 2 if split_keys > 0 else 1)
 
 
+def attention_decode_tc_maps(out: torch.Tensor, q: torch.Tensor, k_plane: torch.Tensor, v_plane: torch.Tensor, block_table: torch.Tensor,
+                             slot_ids: torch.Tensor, kv_lens: torch.Tensor, nh: int, nkv: int, scale: float, softcap: float, temp_coef: float,
+                             temp_every: int, lam: float, eps: float, factor: float, max_splits: int, part_acc: torch.Tensor, part_ml: torch.Tensor,
+                             counters: torch.Tensor, status: torch.Tensor) -> None:
+    """Differential attention of a decode step (one new token a row) on the tcgen05 tensor cores: attention_decode_tc with two maps of 64
+    entries a head over values of 128, at most 8 heads per kv head.  Scratch: attention_decode_tc_scratch with nh * 2 heads."""
+    d = 128
+    _need(out, "out", torch.bfloat16, 2); _need(q, "q", torch.bfloat16, 2)
+    _need(k_plane, "k_plane", torch.bfloat16, 4); _need(v_plane, "v_plane", torch.bfloat16, 4)
+    rows = out.shape[0]
+    if out.shape[1] != nh * d or q.shape != out.shape or k_plane.shape[1] != nkv or k_plane.shape[3] != d or v_plane.shape != k_plane.shape:
+        raise KernelError(f"attention_decode_tc: shapes out {tuple(out.shape)} q {tuple(q.shape)} k {tuple(k_plane.shape)}")
+    _need(block_table, "block_table", torch.int32, 2); _need(slot_ids, "slot_ids", torch.int32, 1); _need(kv_lens, "kv_lens", torch.int32, 1)
+    na, nm, nc = attention_decode_tc_scratch(rows, nh * 2, nkv, d, max_splits)
+    _need(part_acc, "part_acc", torch.float32); _need(part_ml, "part_ml", torch.float32); _need(counters, "counters", torch.int32, 1)
+    if part_acc.numel() < na or part_ml.numel() < nm or counters.numel() < nc:
+        raise KernelError("attention_decode_tc: the scratch is too small")
+    _check(_lib().hymt2_attention_decode_tc_maps(_ptr(out), _ptr(q), _ptr(k_plane), _ptr(v_plane), c_long(k_plane.shape[0]), _ptr(block_table),
+                                                 c_int(block_table.stride(0)), c_int(k_plane.shape[2]), _ptr(slot_ids), _ptr(kv_lens),
+                                                 c_int(rows), c_int(nh), c_int(nkv), c_float(scale), c_float(softcap), c_float(temp_coef),
+                                                 c_int(temp_every), c_float(lam), c_float(eps), c_float(factor), c_int(max_splits),
+                                                 _ptr(part_acc), _ptr(part_ml), _ptr(counters), _ptr(status), _stream()), "attention_decode_tc")
+
+
 DIFF_MAX_FIXED_CAP = 60.0   # up to this cap a score's exponential needs no offset in float32 (the tensor-core kernels' form of capped scores)
 
 
