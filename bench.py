@@ -258,7 +258,35 @@ def pulenex_config(size: str, layers: int):
                                         logit_scale=0.25))
 
 
-DESIGN_TABLES = {"pemezen": DESIGN_SIZES, "novunex": NOVUNEX_SIZES, "rutetar": RUTETAR_SIZES, "pulenex": PULENEX_SIZES}
+# Sosepel: differential attention with two maps of 64 entries over values of 128; the first of every four layers has a dense
+# feed-forward, the others a mixture of `experts` gated experts of width `ff` in `groups` groups, `top` chosen out of `keep` groups,
+# and a gated shared expert; layers 1 and 2 run twice, so that as many layers run as the models beside it have
+SOSEPEL_SIZES = {
+    "s": dict(width=1024, vocab=32768, heads=8, kv_heads=2, dim=64, vdim=128, dense_ff=5632, experts=16, top=4, groups=4, keep=2, ff=512,
+              shared=1024, buckets=20011, dense=DESIGN_SIZES["s"]["dense"]),
+    "m": dict(width=2048, vocab=65536, heads=16, kv_heads=4, dim=64, vdim=128, dense_ff=11264, experts=32, top=4, groups=8, keep=4, ff=1024,
+              shared=2048, buckets=50021, dense=DESIGN_SIZES["m"]["dense"]),
+}
+
+
+def sosepel_config(size: str, layers: int):
+    from hymt2sharp_b200.config import SosepelConfig
+    z = SOSEPEL_SIZES[size]
+    entries = []
+    for i in range(max(3, layers - 2)):
+        mixer = dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=z["dim"], vdim=z["vdim"], scale=z["dim"] ** -0.5, diff=0.35, softcap=40.0,
+                     q_temp=dict(coef=0.1, every=2048))
+        mlp = dict(kind="dense", ff=z["dense_ff"]) if i % 4 == 0 else \
+            dict(kind="moe", expert=dict(ff=z["ff"]), router=dict(experts=z["experts"], top=z["top"], groups=dict(count=z["groups"], keep=z["keep"])),
+                 shared=dict(ff=z["shared"]))
+        entries.append(dict(type="attention", mixer=mixer, mlp=mlp))
+    return SosepelConfig.from_dict(dict(architecture="Sosepel", vocab=z["vocab"], width=z["width"], layers=entries, norm=dict(eps=1e-6),
+                                        loop=dict(start=1, stop=3, times=2), logit_softcap=25.0,
+                                        embedding=dict(scale=6.0, bigram=dict(buckets=z["buckets"], mul_prev=4099, mul_cur=61))))
+
+
+DESIGN_NEIGHBOURS = {"sosepel": "novunex"}   # a design whose closest model is another one than the dense: that one stands beside both
+DESIGN_TABLES = {"sosepel": SOSEPEL_SIZES, "pemezen": DESIGN_SIZES, "novunex": NOVUNEX_SIZES, "rutetar": RUTETAR_SIZES, "pulenex": PULENEX_SIZES}
 
 
 def make_design_models(size: str, layers: int, design: str = "pemezen") -> dict:
@@ -276,8 +304,9 @@ def make_design_models(size: str, layers: int, design: str = "pemezen") -> dict:
             mixer = dict(heads=z["heads"], dim=z["dim"], rot_dim=z["rot_dim"], vdim=z["vdim"], kv_rank=z["kv_rank"],
                          scale=(z["dim"] + z["rot_dim"]) ** -0.5, rot=rot)
         entries.append(dict(type=kind, mixer=mixer, mlp=dict(kind="dense", ff=z["ff"])))
-    if design == "novunex":
-        new = novunex_config(size, layers)
+    makers = {"novunex": novunex_config, "sosepel": sosepel_config}
+    if design in makers:
+        new = makers[design](size, layers)
     elif design == "rutetar":
         new = rutetar_config(size, layers)
     elif design == "pulenex":
@@ -290,7 +319,9 @@ def make_design_models(size: str, layers: int, design: str = "pemezen") -> dict:
                                             rope_scaling={"type": "dynamic", "alpha": 1000.0}, **z["dense"]))
     old_data = {k: v for k, v in old.to_dict().items()}
     folders = {}
-    for name, cfg in ((design, new), ("hunyuan_dense", HunyuanDenseConfig.from_dict(old_data))):
+    beside = DESIGN_NEIGHBOURS.get(design)
+    for name, cfg in ((design, new), *(((beside, makers[beside](size, layers)),) if beside else ()),
+                      ("hunyuan_dense", HunyuanDenseConfig.from_dict(old_data))):
         folders[name] = write_random_model(tempfile.mkdtemp(prefix=f"hymt2_bench_{name}_"), cfg, 7, 0.02)
     return folders
 
@@ -508,7 +539,7 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip decode at batch 1 and 64")
     ap.add_argument("--no-kernels", action="store_true", help="skip the kernels timed alone")
     ap.add_argument("--no-graph", action="store_true")
-    ap.add_argument("--design", default=None, choices=["pemezen", "novunex", "rutetar", "pulenex"],
+    ap.add_argument("--design", default=None, choices=sorted(DESIGN_TABLES),
                     help="instead of the flagship workload: prefill (--prefill tokens) and decode (--batch sequences of --prefill tokens, "
                          "--steps steps) of this design beside the Hunyuan-dense model of equal size, with per-kernel times")
     ap.add_argument("--design-size", default="s", choices=sorted(DESIGN_SIZES))

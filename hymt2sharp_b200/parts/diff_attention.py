@@ -23,7 +23,7 @@ from ..cache.allocator import GroupSpec
 from ..kernels import fast, ops
 from ..weights.loader import TensorSpec
 from .attention import SPLIT_KEYS
-from .base import MixerSlot, register_part
+from .base import MixerSlot, RotaryEpilogue, register_part
 from .linear import Linear, compute_form
 
 MAPS = 2
@@ -77,11 +77,16 @@ class DiffAttention:
         T, H, G, d, dv = ctx.num_tokens, self.heads, self.kv_heads, self.dim, self.vdim
         k_plane, v_plane = ctx.cache.plane(slot.group, slot.plane)
         table = ctx.cache.tables[slot.group]
-        proj = self.qkv(x, ctx=ctx)
-        q = torch.empty((T, H * MAPS * d), dtype=proj.dtype, device=proj.device)
-        ops.rope_kv_general(proj, q, k_plane if slot.writes else None, v_plane if slot.writes else None, table, ctx.cache.block_tokens,
-                            ctx.token_seq, ctx.token_pos, ctx.slot_ids, None, 0, None, None, ops.NORM_NONE, self.eps, H, G, MAPS * d, dv, True)
-        out = torch.empty((T, H * dv), dtype=proj.dtype, device=proj.device)
+        planes = (k_plane, v_plane) if slot.writes else (None, None)
+        q = None
+        if MAPS * d == dv:      # projection and cache append as one kernel, where the kernels have one for the shape
+            q = fast.try_project_rope_kv(x, self.qkv.weight, RotaryEpilogue.none(), ctx, planes, k_plane.dtype, table, None, None, self.eps, H, G, dv)
+        if q is None:
+            proj = self.qkv(x, ctx=ctx)
+            q = torch.empty((T, H * MAPS * d), dtype=proj.dtype, device=proj.device)
+            ops.rope_kv_general(proj, q, *planes, table, ctx.cache.block_tokens, ctx.token_seq, ctx.token_pos, ctx.slot_ids, None, 0, None, None,
+                                ops.NORM_NONE, self.eps, H, G, MAPS * d, dv, True)
+        out = torch.empty((T, H * dv), dtype=q.dtype, device=q.device)
         self.attend(out, q, k_plane, v_plane, table, ctx)
         if store:
             self.out_store(out, out=residual)
