@@ -35,13 +35,16 @@
 // needs no running maximum: for C up to MAX_FIXED_CAP every exp(score) lies within float32's (and bfloat16's) range and
 // so do the sums, the numerators are taken as they are, and O is never rescaled.  tanh is the kernel's scarcest resource: while every
 // |s / C| of a warp's rows in a tile stays below 1 it is an odd polynomial on pairs of scores (two-wide float32 fused
-// multiply-adds), coefficients fitted for the smallest largest error over that range (2e-8, of an error of 1e-7 with float32's
-// own rounding); else it is 1 - 2 / (exp(2 x) + 1).  d = 32 (two maps side by side in one 128-byte row), 64 and 128 are taken.
+// multiply-adds; two threads share a row there, half of the tile's scores each, so that four softmax warps a scheduler hide one
+// another's latency), coefficients fitted for the smallest largest error over that range (2.4e-7, about what
+// float32's own rounding of the sum costs); else it is 1 - 2 / (exp(2 x) + 1).  d = 32 (two maps side by side in one 128-byte row), 64 and 128 are taken.
 #include "tc_common.cuh"
+
+#include <type_traits>
 
 namespace {
 
-constexpr int Q_ROWS = 128, KEY_TILE = 64, NUM_THREADS = 256, KV_STAGES = 2, K_SLOTS = 3;
+constexpr int Q_ROWS = 128, KEY_TILE = 64, KV_STAGES = 2, K_SLOTS = 3;
 // The numbers of the barrier protocol (why these: see the kernel).  hymt2_attention_prefill_tc_protocol hands them to the
 // test that explores every interleaving of the roles, so that the protocol explored is the one compiled here.
 constexpr int P_BARS = K_SLOTS;      // "P of tile i is written": one barrier per K slot, tile mod P_BARS
@@ -69,7 +72,15 @@ struct PrefillParams {
 
 enum { FORM_CLASSIC = 0, FORM_MAPS = 1, FORM_MAPS_CAPPED = 2 };
 constexpr float MAX_FIXED_CAP = 60.f;
+__host__ __device__ constexpr int row_threads(int form) { return form == FORM_MAPS_CAPPED ? 2 : 1; }      // softmax threads a query row
+__host__ __device__ constexpr int num_threads(int form) { return 128 + Q_ROWS * row_threads(form); }      // warps 0 to 2: copies and MMAs
 
+// the largest of three absolute values
+__device__ __forceinline__ float max3_abs(float a, float b, float c) {
+    float r;
+    asm("max.abs.f32 %0, %1, %2, %3;" : "=f"(r) : "f"(a), "f"(b), "f"(c));
+    return r;
+}
 // Two float32 side by side in a 64-bit register.
 __device__ __forceinline__ uint64_t pack2(float a, float b) {
     uint64_t r;
@@ -110,10 +121,11 @@ __device__ __forceinline__ void tmem_store16(uint32_t taddr, const float* v) {
 
 
 template <int D, int DV, int FORM = FORM_CLASSIC>
-__global__ void __launch_bounds__(NUM_THREADS, 2)
+__global__ void __launch_bounds__(num_threads(FORM), 2)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, PrefillParams p) {
     constexpr bool MAPS = FORM != FORM_CLASSIC;
+    constexpr int ROW_THREADS = row_threads(FORM), COLS = KEY_TILE / ROW_THREADS;   // softmax threads a row, and scores of a tile that each takes
     constexpr int KD = D < 64 ? 64 : D;                     // entries of a query or key row that are loaded
     constexpr int D_BOXES = KD / 64, DV_BOXES = DV / 64;    // TMA boxes of 64 elements along d and along dv
     constexpr int Q_BYTES = Q_ROWS * KD * 2, K_TILE_BYTES = KEY_TILE * KD * 2, V_TILE_BYTES = KEY_TILE * DV * 2, P_BYTES = Q_ROWS * KEY_TILE * 2;
@@ -182,7 +194,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         mbar_init(q_full, 1);
         for (int t = 0; t < S_BUFFERS; t++) mbar_init(s_full + 8 * t, 1);
         for (int t = 0; t < O_BARS; t++) mbar_init(o_full + 8 * t, 1);
-        for (int t = 0; t < P_BARS; t++) mbar_init(p_full + 8 * t, 128);
+        for (int t = 0; t < P_BARS; t++) mbar_init(p_full + 8 * t, Q_ROWS * ROW_THREADS);
         abort_s = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
@@ -281,7 +293,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             umma_commit(o_full + 8 * (i % O_BARS));
         }
     } else if (warp >= 4) {
-        // ---- softmax: one thread per query row; O stays in TMEM ------------------------------------
+        // ---- softmax: one or two threads per query row; O stays in TMEM ----------------------------
+        const int part = ROW_THREADS == 1 ? 0 : (warp - 4) >> 2;        // which of the row's threads: its scores begin at part * COLS
         const int quarter = warp & 3, r = quarter * 32 + lane;
         const uint32_t lane_addr = tmem_base + ((uint32_t)(quarter * 32) << 16);
         const int pos = first_pos + r;                                  // position of this row's query
@@ -298,72 +311,76 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         }
         // capped scores: exp(C tanh(x)) = 2^(x * (a polynomial in x^2)) with the factor C log2(e) in the coefficients
         const float cap_log2 = p.softcap * 1.4426950408889634f, to_x = FORM == FORM_MAPS_CAPPED ? row_scale / p.softcap : 0.f;
-        uint64_t c2[7], x2 = 0, lsum[2] = {0, 0};
+        uint64_t c2[6], x2 = 0, lsum[2] = {0, 0};
         if constexpr (FORM == FORM_MAPS_CAPPED) {
-            constexpr float c[7] = {0.9999997019767761f, -0.33332130312919617f, 0.13319583237171173f, -0.05326583608984947f,
-                                    0.019973281770944595f, -0.005951280705630779f, 0.0009637721814215183f};
+            constexpr float c[6] = {0.9999968409538269f, -0.3332400321960449f, 0.13253524899482727f, -0.05097286403179169f,
+                                    0.016114182770252228f, -0.002839465858414769f};
 #pragma unroll
-            for (int k = 0; k < 7; k++) c2[k] = pack2(c[k] * cap_log2, c[k] * cap_log2);
+            for (int k = 0; k < 6; k++) c2[k] = pack2(c[k] * cap_log2, c[k] * cap_log2);
             x2 = pack2(to_x, to_x);
         }
         for (int i = 0; i < num_tiles; i++) {
             if (!(ok = mbar_wait(s_full + 8 * (i & 1), (i >> 1) & 1, abort_flag, p.status, 115))) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const int key0 = (tile_begin + i) * KEY_TILE;
-            float s[KEY_TILE];
-            tmem_load32(lane_addr + S_COL + 64 * (i & 1), s);
-            tmem_load32(lane_addr + S_COL + 64 * (i & 1) + 32, s + 32);
+            float s[COLS];
+#pragma unroll
+            for (int c = 0; c < COLS; c += 32) tmem_load32(lane_addr + S_COL + 64 * (i & 1) + part * COLS + c, s + c);
             const uint32_t p_dst = k_of(i);
             if constexpr (FORM == FORM_MAPS_CAPPED) {
-                const bool edge = __any_sync(0xffffffffu, !row_ok || key0 + KEY_TILE - 1 > pos);
+                // this thread's last visible score (a row without a query counts as the last one that has one: nobody reads it)
+                const int last = min(pos, last_pos) - key0 - part * COLS;
+                const bool edge = __any_sync(0xffffffffu, COLS - 1 > last);
                 if (edge) {   // (what lies behind a row's position, or was never written, counts as 0 until its numerator is dropped)
 #pragma unroll
-                    for (int c = 0; c < KEY_TILE; c++) s[c] = (row_ok && key0 + c <= pos) ? s[c] : 0.f;
+                    for (int c = 0; c < COLS; c++) s[c] = c <= last ? s[c] : 0.f;
                 }
                 float mx[2] = {0.f, 0.f};
 #pragma unroll
-                for (int c = 0; c < KEY_TILE; c += 2) mx[(c >> 1) & 1] = fmaxf(mx[(c >> 1) & 1], fmaxf(fabsf(s[c]), fabsf(s[c + 1])));
+                for (int c = 0; c < COLS; c += 2) mx[(c >> 1) & 1] = max3_abs(mx[(c >> 1) & 1], s[c], s[c + 1]);
                 const bool wide = __any_sync(0xffffffffu, !(fmaxf(mx[0], mx[1]) * fabsf(to_x) <= 1.0f));
-                auto numerators = [&](auto of_pair) {
+                // (the tiles at a row's edge have code of their own: tests of the position, even skipped ones, cost the others a fifth)
+                auto numerators = [&](auto at_edge, auto of_pair) {
 #pragma unroll
-                    for (int c8 = 0; c8 < KEY_TILE / 8; c8++) {
+                    for (int c8 = 0; c8 < COLS / 8; c8++) {
                         uint32_t packed[4];
 #pragma unroll
                         for (int j = 0; j < 4; j++) {
                             const int c = c8 * 8 + 2 * j;
                             float p0, p1;
                             of_pair(s[c], s[c + 1], p0, p1);
-                            if (edge) {
-                                p0 = (row_ok && key0 + c <= pos) ? p0 : 0.f;
-                                p1 = (row_ok && key0 + c + 1 <= pos) ? p1 : 0.f;
+                            if constexpr (decltype(at_edge)::value) {
+                                p0 = c <= last ? p0 : 0.f;
+                                p1 = c + 1 <= last ? p1 : 0.f;
                             }
                             lsum[j & 1] = add2(lsum[j & 1], pack2(p0, p1));
                             const __nv_bfloat162 h = __floats2bfloat162_rn(p0, p1);
                             packed[j] = *reinterpret_cast<const uint32_t*>(&h);
                         }
-                        const uint32_t dst = p_dst + r * 128 + ((c8 ^ (r & 7)) << 4);
+                        const uint32_t dst = p_dst + r * 128 + (((part * (COLS / 8) + c8) ^ (r & 7)) << 4);
                         asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(dst), "r"(packed[0]), "r"(packed[1]),
                                      "r"(packed[2]), "r"(packed[3]) : "memory");
                     }
                 };
-                if (!wide) {
-                    numerators([&](float s0, float s1, float& p0, float& p1) {
-                        const uint64_t x = mul2(pack2(s0, s1), x2), u = mul2(x, x);
-                        uint64_t q = c2[6];
+                auto narrow_pair = [&](float s0, float s1, float& p0, float& p1) {
+                    const uint64_t x = mul2(pack2(s0, s1), x2), u = mul2(x, x);
+                    uint64_t q = c2[5];
 #pragma unroll
-                        for (int k = 5; k >= 0; k--) q = fma2(q, u, c2[k]);
-                        float e0, e1;
-                        unpack2(mul2(q, x), e0, e1);
-                        p0 = ex2_approx(e0);
-                        p1 = ex2_approx(e1);
-                    });
-                } else {
-                    const float twice = 2.0f * 1.4426950408889634f * to_x;
-                    numerators([&](float s0, float s1, float& p0, float& p1) {   // exp(2x) = inf and 0 give tanh 1 and -1
-                        p0 = ex2_approx(fmaf(__fdividef(1.0f, ex2_approx(s0 * twice) + 1.0f), -2.0f * cap_log2, cap_log2));
-                        p1 = ex2_approx(fmaf(__fdividef(1.0f, ex2_approx(s1 * twice) + 1.0f), -2.0f * cap_log2, cap_log2));
-                    });
-                }
+                    for (int k = 4; k >= 0; k--) q = fma2(q, u, c2[k]);
+                    float e0, e1;
+                    unpack2(mul2(q, x), e0, e1);
+                    p0 = ex2_approx(e0);
+                    p1 = ex2_approx(e1);
+                };
+                const float twice = 2.0f * 1.4426950408889634f * to_x;
+                auto wide_pair = [&](float s0, float s1, float& p0, float& p1) {   // exp(2x) = inf and 0 give tanh 1 and -1
+                    p0 = ex2_approx(fmaf(__fdividef(1.0f, ex2_approx(s0 * twice) + 1.0f), -2.0f * cap_log2, cap_log2));
+                    p1 = ex2_approx(fmaf(__fdividef(1.0f, ex2_approx(s1 * twice) + 1.0f), -2.0f * cap_log2, cap_log2));
+                };
+                if (!edge && !wide) numerators(std::false_type{}, narrow_pair);
+                else if (!edge) numerators(std::false_type{}, wide_pair);
+                else if (!wide) numerators(std::true_type{}, narrow_pair);
+                else numerators(std::true_type{}, wide_pair);
             } else {
             // s stays unscaled: the scale (> 0) goes into the exponent's multiply-add; most tiles lie wholly
             // inside the row's visible range and need no mask
@@ -428,7 +445,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             // such rows; V of the tile must have landed before they are overwritten.
             if (key0 + KEY_TILE > kv_len &&
                 !(ok = mbar_wait(kv_full + 8 * (i % KV_STAGES), (i / KV_STAGES) & 1, abort_flag, p.status, 110))) break;
-            if (r < KEY_TILE && key0 + r >= kv_len) {
+            if (part == 0 && r < KEY_TILE && key0 + r >= kv_len) {
 #pragma unroll
                 for (int x = 0; x < DV_BOXES; x++) {
                     const uint32_t rowp = v_of(i) + x * (KEY_TILE * 128) + r * 128;
@@ -475,49 +492,65 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     if constexpr (MAPS) {
         // ---- the two maps of the head meet: every thread of both CTAs takes part in the three cluster barriers, whether or not a
         // wait gave up above.  Shared memory of Q and of the keys is free: every product of this CTA is through.
-        constexpr int HALF = DV / 2;
+        constexpr int HALF = DV / 2, TAKEN = HALF / ROW_THREADS;   // columns that this CTA writes out, and that a thread takes of them
         static_assert(HALF * Q_ROWS * 4 <= K_SLOTS * K_SLOT_BYTES, "half of the outputs takes the keys' place");
         asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
         __syncthreads();
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         const bool softmax_warp = warp >= 4;
+        const int part = ROW_THREADS == 1 ? 0 : (warp - 4) >> 2;
         const int quarter = warp & 3, r = quarter * 32 + lane;
         const uint32_t lane_addr = tmem_base + ((uint32_t)(quarter * 32) << 16) + O_COL;
         float* given = reinterpret_cast<float*>(smem_raw + Q_BYTES);          // [HALF columns][Q_ROWS]: the half that the other CTA writes out
-        float* squares = reinterpret_cast<float*>(smem_raw);                  // [Q_ROWS]
+        float* squares = reinterpret_cast<float*>(smem_raw);                  // [ROW_THREADS][Q_ROWS]
+        float* sums = squares + ROW_THREADS * Q_ROWS;                          // [ROW_THREADS][Q_ROWS]
+        if (ROW_THREADS > 1) {   // (in the order of the row's threads, so that both add alike)
+            if (softmax_warp) sums[part * Q_ROWS + r] = l;
+            __syncthreads();
+            l = sums[r] + sums[Q_ROWS + r];
+        }
         const float inv = ok && l > 0.f ? 1.0f / l : 0.f;
-        if (softmax_warp) {
+        auto load_taken = [&](uint32_t at, float* v) {
+            if constexpr (TAKEN >= 32) {
 #pragma unroll
-            for (int c = 0; c < HALF; c += 32) {
-                float o[32];
-                tmem_load32(lane_addr + (map ^ 1) * HALF + c, o);
-#pragma unroll
-                for (int j = 0; j < 32; j++) given[(c + j) * Q_ROWS + r] = o[j] * inv;
+                for (int c = 0; c < TAKEN; c += 32) tmem_load32(at + c, v + c);
+            } else {
+                tmem_load16(at, v);
             }
+        };
+        const int col0 = part * TAKEN;
+        if (softmax_warp) {
+            float o[TAKEN];
+            load_taken(lane_addr + (map ^ 1) * HALF + col0, o);
+#pragma unroll
+            for (int j = 0; j < TAKEN; j++) given[(col0 + j) * Q_ROWS + r] = o[j] * inv;
         }
         __syncwarp();
         cluster_sync_all();
-        float o[HALF], ss = 0.f;
+        float o[TAKEN], ss = 0.f;
         if (softmax_warp) {
+            load_taken(lane_addr + map * HALF + col0, o);
 #pragma unroll
-            for (int c = 0; c < HALF; c += 32) {
-                tmem_load32(lane_addr + map * HALF + c, o + c);
-#pragma unroll
-                for (int j = 0; j < 32; j++) {
-                    const float other = ld_cluster_f32(smem_u32(given + (c + j) * Q_ROWS + r), map ^ 1), own = o[c + j] * inv;
-                    o[c + j] = map == 0 ? fmaf(-p.lambda, other, own) : fmaf(-p.lambda, own, other);
-                    ss = fmaf(o[c + j], o[c + j], ss);
-                }
+            for (int j = 0; j < TAKEN; j++) {
+                const float other = ld_cluster_f32(smem_u32(given + (col0 + j) * Q_ROWS + r), map ^ 1), own = o[j] * inv;
+                o[j] = map == 0 ? fmaf(-p.lambda, other, own) : fmaf(-p.lambda, own, other);
+                ss = fmaf(o[j], o[j], ss);
             }
-            squares[r] = ss;
+            squares[part * Q_ROWS + r] = ss;
         }
         __syncwarp();
         cluster_sync_all();
         if (softmax_warp && ok && r < rows_here) {
-            const float scale = p.factor / sqrtf((ss + ld_cluster_f32(smem_u32(squares + r), map ^ 1)) / (float)DV + p.eps);
-            __nv_bfloat16* dst = p.out + ((size_t)(tok0 + qtile * Q_ROWS + r) * p.nh + head) * DV + map * HALF;
+            float mine = 0.f, others = 0.f;
 #pragma unroll
-            for (int j = 0; j < HALF; j += 8) {
+            for (int t = 0; t < ROW_THREADS; t++) {
+                mine += squares[t * Q_ROWS + r];
+                others += ld_cluster_f32(smem_u32(squares + t * Q_ROWS + r), map ^ 1);
+            }
+            const float scale = p.factor / sqrtf((mine + others) / (float)DV + p.eps);
+            __nv_bfloat16* dst = p.out + ((size_t)(tok0 + qtile * Q_ROWS + r) * p.nh + head) * DV + map * HALF + col0;
+#pragma unroll
+            for (int j = 0; j < TAKEN; j += 8) {
                 __nv_bfloat162 h[4];
 #pragma unroll
                 for (int q = 0; q < 4; q++) h[q] = __floats2bfloat162_rn(o[j + 2 * q] * scale, o[j + 2 * q + 1] * scale);
@@ -554,7 +587,7 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
     if constexpr (FORM != FORM_CLASSIC) {   // the two maps of a head are a cluster
         cudaLaunchConfig_t cfg = {};
         cfg.gridDim = grid;
-        cfg.blockDim = dim3(NUM_THREADS);
+        cfg.blockDim = dim3(num_threads(FORM));
         cfg.dynamicSmemBytes = smem;
         cfg.stream = stream;
         cudaLaunchAttribute attr[1];
@@ -568,7 +601,7 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
         if (e != cudaSuccess) { hymt2_set_error("attention_prefill_tc: %s", cudaGetErrorString(e)); return HYMT2_ERR_LAUNCH; }
         return HYMT2_OK;
     } else {
-        kernel<<<grid, NUM_THREADS, smem, stream>>>(mq, mk, mv, p);
+        kernel<<<grid, num_threads(FORM), smem, stream>>>(mq, mk, mv, p);
         return hymt2_check_launch("attention_prefill_tc");
     }
 }
