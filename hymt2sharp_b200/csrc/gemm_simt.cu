@@ -265,7 +265,8 @@ gemm_skinny_batched_kernel(TC* __restrict__ C, const T* __restrict__ A, const T*
 
 // The grouped product for few sorted rows (a decode step): row tiles of GROUP_SKINNY_ROWS rows, a warp per output column
 // reads its weight row once, 16 bytes a lane, and keeps a float32 sum for every row of the tile.  The time is that of
-// reading the matrices of the groups in use once.
+// reading the matrices of the groups in use once.  For gated experts (EPI_SWIGLU: a group's matrix holds N gate rows, then N up
+// rows) the warp's two weight rows are a gate row and its up row, and one column silu(gate) * up comes out.
 constexpr int GROUP_SKINNY_ROWS = 8, GROUP_SKINNY_COLS = 2;   // rows of a tile; output columns (weight rows) of a warp
 
 template <typename T, typename TC, int EPI>
@@ -278,7 +279,9 @@ gemm_skinny_grouped_kernel(TC* __restrict__ C, const T* __restrict__ A, const T*
     if (group < 0) return;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     constexpr int COLS = GROUP_SKINNY_COLS;
-    const int n0 = (blockIdx.x * SKINNY_WARPS + warp) * COLS;
+    constexpr bool GATED = EPI == EPI_SWIGLU;
+    static_assert(COLS == 2, "a gate row and its up row");
+    const int n0 = (blockIdx.x * SKINNY_WARPS + warp) * (GATED ? 1 : COLS);
     if (n0 >= N) return;
     const int m0 = blockIdx.y * GROUP_SKINNY_ROWS;
     const T* a_row[GROUP_SKINNY_ROWS];
@@ -291,7 +294,7 @@ gemm_skinny_grouped_kernel(TC* __restrict__ C, const T* __restrict__ A, const T*
     }
     const T* w[COLS];
 #pragma unroll
-    for (int c = 0; c < COLS; c++) w[c] = W + (size_t)group * w_gs + (size_t)(n0 + c < N ? n0 + c : n0) * K;
+    for (int c = 0; c < COLS; c++) w[c] = W + (size_t)group * w_gs + (size_t)(GATED ? c * N + n0 : (n0 + c < N ? n0 + c : n0)) * K;
     float acc[COLS][GROUP_SKINNY_ROWS];
 #pragma unroll
     for (int c = 0; c < COLS; c++)
@@ -353,6 +356,11 @@ gemm_skinny_grouped_kernel(TC* __restrict__ C, const T* __restrict__ A, const T*
 #pragma unroll
     for (int m = 0; m < GROUP_SKINNY_ROWS; m++) {
         if (ok[m]) {
+            if constexpr (GATED) {
+                const float gate = warp_sum(acc[0][m]), up = warp_sum(acc[1][m]);
+                if (lane == 0) C[(size_t)(m0 + m) * ldc + n0] = from_float<TC>(gate / (1.0f + expf(-gate)) * up);
+                continue;
+            }
 #pragma unroll
             for (int c = 0; c < COLS; c++) {
                 float v = warp_sum(acc[c][m]);
@@ -442,9 +450,9 @@ HYMT2_API int hymt2_gemm_skinny_grouped(void* C, int c_dtype, const void* A, con
                                         int epilogue, cudaStream_t stream) {
     if (tiles == 0 || N == 0) return HYMT2_OK;
     HYMT2_REQUIRE(tiles > 0 && tiles <= 65535 && N > 0 && K > 0, "gemm_skinny_grouped: bad sizes tiles=%d N=%d K=%d", tiles, N, K);
-    HYMT2_REQUIRE(epilogue == EPI_STORE || epilogue == EPI_RELU_SQUARED, "gemm_skinny_grouped: unknown epilogue %d", epilogue);
+    HYMT2_REQUIRE(epilogue == EPI_STORE || epilogue == EPI_RELU_SQUARED || epilogue == EPI_SWIGLU, "gemm_skinny_grouped: unknown epilogue %d", epilogue);
     HYMT2_REQUIRE(lda >= K && ldc >= N && tile_group && row_source, "gemm_skinny_grouped: bad arguments");
-    const int per_block = SKINNY_WARPS * GROUP_SKINNY_COLS;
+    const int per_block = SKINNY_WARPS * (epilogue == EPI_SWIGLU ? 1 : GROUP_SKINNY_COLS);
     const dim3 grid((N + per_block - 1) / per_block, tiles);
     HYMT2_DISPATCH_DTYPE(dtype, T, {
         const long v = 16 / sizeof(T);
@@ -452,6 +460,9 @@ HYMT2_API int hymt2_gemm_skinny_grouped(void* C, int c_dtype, const void* A, con
         HYMT2_DISPATCH_DTYPE(c_dtype, TC, {
             if (epilogue == EPI_STORE)
                 launch_pdl(gemm_skinny_grouped_kernel<T, TC, EPI_STORE>, grid, dim3(SKINNY_WARPS * 32), 0, stream, (TC*)C, (const T*)A,
+                           (const T*)W, tile_group, row_source, gather, N, K, lda, ldc, w_gs, vec);
+            else if (epilogue == EPI_SWIGLU)
+                launch_pdl(gemm_skinny_grouped_kernel<T, TC, EPI_SWIGLU>, grid, dim3(SKINNY_WARPS * 32), 0, stream, (TC*)C, (const T*)A,
                            (const T*)W, tile_group, row_source, gather, N, K, lda, ldc, w_gs, vec);
             else
                 launch_pdl(gemm_skinny_grouped_kernel<T, TC, EPI_RELU_SQUARED>, grid, dim3(SKINNY_WARPS * 32), 0, stream, (TC*)C,

@@ -1403,20 +1403,22 @@ HYMT2_API int hymt2_gemm_tc_grouped(void* C, int c_dtype, const void* X, const v
     HYMT2_REQUIRE(tiles > 0 && groups > 0 && N > 0 && K > 0 && tile_group, "gemm_tc_grouped: bad sizes tiles=%d groups=%d N=%d K=%d", tiles, groups, N, K);
     HYMT2_REQUIRE(K % 8 == 0 && lda % 8 == 0 && N % 8 == 0, "gemm_tc_grouped: K, lda and N must be multiples of 8 (K=%d lda=%ld N=%d)", K, lda, N);
     HYMT2_REQUIRE(((uintptr_t)X % 16 == 0) && ((uintptr_t)W % 16 == 0), "gemm_tc_grouped: operands must be 16-byte aligned");
-    HYMT2_REQUIRE(act == 0 || act == 1, "gemm_tc_grouped: unknown activation %d", act);
+    HYMT2_REQUIRE(act == 0 || act == 1 || act == 2, "gemm_tc_grouped: unknown activation %d", act);
+    const int epi = act == 2 ? EPI_SWIGLU : EPI_STORE;          // 2: a group's matrix holds N gate rows, then N up rows
+    const int rows_w = act == 2 ? 2 * N : N;
     HYMT2_REQUIRE(status != nullptr, "gemm_tc_grouped: a status word is needed");
-    HYMT2_REQUIRE((long)tiles * TILE_M <= 2147483647L && (long)groups * N <= 2147483647L, "gemm_tc_grouped: too many rows");
+    HYMT2_REQUIRE((long)tiles * TILE_M <= 2147483647L && (long)groups * rows_w <= 2147483647L, "gemm_tc_grouped: too many rows");
     const int T = tiles * TILE_M;
     Plan pl;
-    make_plan(T, N, K, EPI_STORE, sm_count_of_current_device(), &pl, true);
+    make_plan(T, N, K, epi, sm_count_of_current_device(), &pl, true);
     CUtensorMap ma, mb;
-    const bool ok = make_map(&ma, X, T, K, lda, TILE_M) && make_map(&mb, W, (long)groups * N, K, K, pl.bn);
+    const bool ok = make_map(&ma, X, T, K, lda, TILE_M) && make_map(&mb, W, (long)groups * rows_w, K, K, act == 2 ? pl.bn / 2 : pl.bn);
     HYMT2_REQUIRE(ok, "gemm_tc_grouped: cuTensorMapEncodeTiled refused the operands");
     GemmTcParams p{C, ldc, T, N, K, pl.stages, pl.bn, 1, pl.k_blocks_per_split, 0, nullptr, nullptr, status, RopeEpilogue{}, WAIT_LIMIT, -1, NormSide{}};
     p.tile_group = tile_group;
-    p.group_rows = N;
-    p.act = act;
-    return launch_persistent(ma, mb, p, pl, EPI_STORE, c_dtype, stream);
+    p.group_rows = rows_w;
+    p.act = act == 1 ? 1 : 0;
+    return launch_persistent(ma, mb, p, pl, epi, c_dtype, stream);
 }
 
 // hymt2_gemm_tc with an RMSNorm folded in (see NormSide).  As a consumer (ss_in): the activations X are bf16(x * gain) and the sums

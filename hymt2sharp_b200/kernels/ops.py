@@ -1427,13 +1427,17 @@ def gemm_grouped(kernel: str, out: torch.Tensor, a: torch.Tensor, w: torch.Tenso
                  gather: bool, epilogue: int = EPILOGUE_STORE) -> None:
     """out[r] = epilogue(a[source(r)] @ w[tile_group[r // tile]]^T) for the sorted rows r of moe_place: w [experts, N, K];
     source(r) = row_token[r] with `gather` (a holds one row per token), r itself otherwise (a holds sorted rows); padding
-    rows and unused tiles are skipped ("tc": computed and never read).  Epilogues: EPILOGUE_STORE, EPILOGUE_RELU_SQUARED.
+    rows and unused tiles are skipped ("tc": computed and never read).  Epilogues: EPILOGUE_STORE, EPILOGUE_RELU_SQUARED, and for "skinny"
+    and "tc" EPILOGUE_SWIGLU (w [experts, 2N, K] holds an expert's N gate rows, then its N up rows; out = silu(gate) * up).
     kernel "simt": CUDA cores, any sizes and types; "skinny": CUDA cores, tiles of 8 rows, a and w of one type, the time of
     reading the weights once; "tc": tcgen05, bfloat16, no gather (see moe_gather), K and N multiples of 8."""
     _need(out, "out", None, 2); _need(a, "a", None, 2); _need(w, "w", None, 3)
     _need(tile_group, "tile_group", torch.int32, 1); _need(row_token, "row_token", torch.int32, 1)
     tiles, tile = tile_group.numel() - 1, gemm_group_tile(kernel)
-    N, K = w.shape[1], w.shape[2]
+    gated = epilogue == EPILOGUE_SWIGLU
+    N, K = w.shape[1] // (2 if gated else 1), w.shape[2]
+    if gated and (w.shape[1] % 2 or kernel == "simt" or (kernel == "tc" and out.dtype != torch.bfloat16)):
+        raise KernelError(f"gemm_grouped: gated experts are not taken by '{kernel}' with w {tuple(w.shape)} and out {out.dtype}")
     if out.shape != (tiles * tile, N) or a.shape[1] != K or row_token.numel() < tiles * tile or (not gather and a.shape[0] < tiles * tile):
         raise KernelError(f"gemm_grouped: shapes out {tuple(out.shape)} a {tuple(a.shape)} w {tuple(w.shape)} tiles {tiles} of {tile}")
     if kernel == "simt":
@@ -1446,14 +1450,14 @@ def gemm_grouped(kernel: str, out: torch.Tensor, a: torch.Tensor, w: torch.Tenso
             raise KernelError("gemm_grouped: the kernel for few rows wants a and w of one type")
         _check(_lib().hymt2_gemm_skinny_grouped(_ptr(out), c_int(dtype_code(out.dtype)), _ptr(a), _ptr(w), c_int(dtype_code(w.dtype)),
                                                 _ptr(tile_group), _ptr(row_token), c_int(1 if gather else 0), c_int(tiles), c_int(N), c_int(K),
-                                                c_long(a.stride(0)), c_long(out.stride(0)), c_long(N * K), c_int(epilogue), _stream()),
+                                                c_long(a.stride(0)), c_long(out.stride(0)), c_long(w.shape[1] * K), c_int(epilogue), _stream()),
                "gemm_skinny_grouped")
     else:
         if gather or a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
             raise KernelError("gemm_grouped: the tensor-core kernel wants sorted bfloat16 rows")
         _check(_lib().hymt2_gemm_tc_grouped(_ptr(out), c_int(dtype_code(out.dtype)), _ptr(a), _ptr(w), _ptr(tile_group), c_int(tiles),
                                             c_int(w.shape[0]), c_int(N), c_int(K), c_long(a.stride(0)), c_long(out.stride(0)),
-                                            c_int(1 if epilogue == EPILOGUE_RELU_SQUARED else 0), _ptr(device_status(out.device)), _stream()),
+                                            c_int(2 if gated else 1 if epilogue == EPILOGUE_RELU_SQUARED else 0), _ptr(device_status(out.device)), _stream()),
                "gemm_tc_grouped")
 
 

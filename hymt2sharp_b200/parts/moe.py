@@ -9,7 +9,8 @@ the correction and not renormalised.  A shared expert (any feed-forward part) ru
 Chosen by parameters beyond that: a bias of the router (`router_bias`, a stored vector added to z); weights that are the
 softmax over the CHOSEN outputs only (`weights="chosen_softmax"`; the choice by score is then the choice by z); and gated
 experts, expert(x) = W_down (act(W_gate x) * (W_up x)) (`gate_proj` given; act "silu"): gate and up are one grouped product
-over the stacked matrices, and a small kernel applies the activation.  The scores may be the sigmoid of each output
+over the stacked matrices, whose epilogue applies SiLU and multiplies (the general CUDA-core kernel, and another activation:
+a small kernel behind it).  The scores may be the sigmoid of each output
 (`scores="sigmoid"`), the weights the chosen scores' shares of their sum (`weights="chosen_share"`, `share_eps` added to the
 sum), and the choice limited to groups: the outputs form `groups` equal groups of neighbours, and only those of the `keep`
 groups whose two largest scores have the largest sums can be chosen.  The shared expert may have a gate per token
@@ -155,7 +156,10 @@ class RoutedExperts:
             rows, gather = torch.empty((tiles * tile, self.hidden), dtype=x.dtype, device=dev), False
             ops.moe_gather(rows, x, row_token)
         ops.tag = "experts_up"
-        if self.gated:
+        if self.gated and self.activation == "silu" and kernel != "simt":
+            act = torch.empty((tiles * tile, self.intermediate), dtype=x.dtype, device=dev)
+            ops.gemm_grouped(kernel, act, rows, self.up, tile_group, row_token, gather, ops.EPILOGUE_SWIGLU)
+        elif self.gated:
             both = torch.empty((tiles * tile, 2 * self.intermediate), dtype=x.dtype, device=dev)
             ops.gemm_grouped(kernel, both, rows, self.up, tile_group, row_token, gather, ops.EPILOGUE_STORE)
             act = torch.empty((tiles * tile, self.intermediate), dtype=x.dtype, device=dev)
