@@ -58,8 +58,8 @@ __device__ __forceinline__ void route_token(const RouteRule& r, const float* __r
     for (int i = lane; i < outputs; i += 32) c[i] = s[i] + (r.correction ? r.correction[i] : 0.f);   // (a lane's own entries)
     __syncwarp();
     if (r.groups > 1) {
-        // a group's worth is the sum of its two largest scores; a group stays if fewer than `keep` are worth more (of equals
-        // the lower number counts as more)
+        // a group is worth what its two best scores add up to; it stays if fewer than `keep` are worth more (of equals the
+        // lower number counts as more)
         const int per = outputs / r.groups;
         for (int g = lane; g < r.groups; g += 32) {
             float first = -INFINITY, second = -INFINITY;

@@ -11,8 +11,9 @@ from ..parts.base import PartSpec
 
 @dataclass
 class Bigram:
-    """A second table that the embedding adds a row of: row (previous token * mul_prev + token * mul_cur) mod buckets, and for a
-    sequence's first token row number `buckets`, the last one.  The previous token is state of the sequence."""
+    """A second table whose rows belong to pairs of tokens: the embedding of `token` behind `previous` adds row
+    (previous * mul_prev + token * mul_cur) mod buckets.  Where nothing stands in front (position 0) it adds the row behind the
+    buckets.  Which token came last is kept with the sequence, in its state row."""
     table: str                        # checkpoint name of the [buckets + 1, hidden] table
     buckets: int
     mul_prev: int

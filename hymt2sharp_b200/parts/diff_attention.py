@@ -7,7 +7,7 @@ tau(p) = 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1) (temp_coef 0: tau =
     s_m(i, j) = cap(tau(i) * scale * q_m(i) . k_m(j)),   cap(s) = softcap * tanh(s / softcap)      (no softcap: s itself)
     a_m(i)    = sum_{j <= i} softmax_j(s_m(i, .)) v(j)                                             m = 1, 2
     o         = a_1 - lambda * a_2,   y = o / sqrt(mean(o^2) + eps) * (1 - diff)                   over a head's vdim entries
-    lambda    = exp(sum lq1 * lk1) - exp(sum lq2 * lk2) + diff                                     one number for the layer
+    lambda    = exp(sum lq1 * lk1) - exp(sum lq2 * lk2) + diff                                     worked out once, at load
 
 and W_o projects the heads side by side.  Head h reads key/value head h // (heads / kv_heads).  Scores, temperature, softmax,
 lambda and the combination of the two maps are float32.  The cache keeps a token's two keys of a head as one row of 2 * dim

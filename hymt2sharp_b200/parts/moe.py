@@ -12,8 +12,8 @@ experts, expert(x) = W_down (act(W_gate x) * (W_up x)) (`gate_proj` given; act "
 over the stacked matrices, whose epilogue applies SiLU and multiplies (the general CUDA-core kernel, and another activation:
 a small kernel behind it).  The scores may be the sigmoid of each output
 (`scores="sigmoid"`), the weights the chosen scores' shares of their sum (`weights="chosen_share"`, `share_eps` added to the
-sum), and the choice limited to groups: the outputs form `groups` equal groups of neighbours, and only those of the `keep`
-groups whose two largest scores have the largest sums can be chosen.  The shared expert may have a gate per token
+sum), and the choice limited to groups: outputs side by side are cut into `groups` runs of equal length, the runs are ranked by
+what their two best scores add up to, and the choice is among the outputs of the first `keep` runs.  The shared expert may have a gate per token
 (`shared_gate`, a stored [1, hidden] matrix): its output is multiplied by sigmoid(W x); that product is one more row of the
 router's.
 

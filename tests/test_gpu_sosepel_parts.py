@@ -79,7 +79,7 @@ MIXERS = {
     "tc 64/128, 3 heads on each": (128, dict(heads=6, kv_heads=2, dim=64, vdim=128, scale=0.5, diff=0.35, softcap=15.0, q_temp=dict(coef=0.1, every=7))),
     "tc 64/128, no cap": (128, dict(heads=2, kv_heads=1, dim=64, vdim=128, scale=0.3, diff=0.3)),
     "tc 64/128, a cap too wide for a fixed offset": (128, dict(heads=2, kv_heads=1, dim=64, vdim=128, scale=0.6, diff=0.3, softcap=90.0, q_temp=dict(coef=0.2, every=20))),
-    "tc 32/64": (96, dict(heads=4, kv_heads=2, dim=32, vdim=64, scale=0.9, diff=0.25, softcap=6.0, q_temp=dict(coef=0.3, every=40))),
+    "tc 32/64": (96, dict(heads=6, kv_heads=2, dim=32, vdim=64, scale=0.9, diff=0.25, softcap=6.0, q_temp=dict(coef=0.3, every=40))),
     "tc 32/128": (64, dict(heads=2, kv_heads=1, dim=32, vdim=128, scale=0.9, diff=0.7, softcap=20.0)),
     "tc 128/64": (128, dict(heads=2, kv_heads=1, dim=128, vdim=64, scale=0.4, diff=0.3, softcap=7.0, q_temp=dict(coef=0.5, every=100))),
     "tc 128/128": (128, dict(heads=2, kv_heads=2, dim=128, vdim=128, scale=0.4, diff=0.3, softcap=25.0)),
@@ -243,7 +243,7 @@ def test_pair_embedding_over_steps_batches_and_reused_slots(dtype):
 
 
 # -- routing and the mixture -----------------------------------------------------------------------------------------------------
-@pytest.mark.parametrize("E, top, groups", [(6, 2, (3, 2)), (8, 3, (4, 3)), (5, 1, (5, 3)), (7, 7, None), (64, 6, (8, 3)), (130, 5, (65, 4)), (12, 3, (2, 1))])
+@pytest.mark.parametrize("E, top, groups", [(6, 2, (3, 2)), (10, 4, (5, 3)), (5, 1, (5, 3)), (7, 7, None), (64, 6, (8, 3)), (130, 5, (65, 4)), (12, 3, (2, 1))])
 @pytest.mark.parametrize("T", [1, 5, 300])
 def test_sigmoid_routing_in_groups(T, E, top, groups):
     from hymt2sharp_b200.kernels import ops
@@ -271,7 +271,7 @@ def test_sigmoid_routing_in_groups(T, E, top, groups):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("T, W, E, top, groups, ff, shared", [(3, 44, 6, 2, (3, 2), 9, 7), (200, 64, 8, 3, (4, 3), 24, 40), (9, 128, 12, 3, (4, 2), 48, 48),
+@pytest.mark.parametrize("T, W, E, top, groups, ff, shared", [(3, 44, 6, 2, (3, 2), 9, 7), (200, 64, 10, 4, (5, 3), 24, 40), (9, 128, 12, 3, (4, 2), 48, 48),
                                                               (260, 128, 8, 4, None, 64, 96), (5, 64, 4, 2, None, 24, None)])
 def test_mixture_with_a_gated_shared_expert(dtype, T, W, E, top, groups, ff, shared):
     """Stored and added; every expert has its own size of weights, so that a wrong one shows."""
