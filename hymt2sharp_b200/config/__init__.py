@@ -5,9 +5,10 @@ from .novunex import NovunexConfig
 from .rutetar import RutetarConfig
 from .pulenex import PulenexConfig
 from .sosepel import SosepelConfig
+from .gomerax import GomeraxConfig
 from .registry import (Architecture, register_architecture, get_architecture,
                        known_architectures, load_config)
 
 __all__ = ["ConfigError", "ConfigReader", "read_config_json", "architecture_name", "HunyuanDenseConfig", "PemezenConfig", "NovunexConfig", "RutetarConfig",
-           "PulenexConfig", "SosepelConfig",
+           "PulenexConfig", "SosepelConfig", "GomeraxConfig",
            "Architecture", "register_architecture", "get_architecture", "known_architectures", "load_config"]

@@ -45,7 +45,8 @@ struct AttnParams {
     int v_from_k;           // the values are the first dv entries of the key rows (one vector per token serves as both)
     float scale;
     int* status;            // may be null; [0] = 2 when a row is longer than max_splits * split_keys covers
-    int sink;               // the softmax has one more term in its denominator, of score 0 and without a value
+    int sink;               // the softmax has one more term in its denominator, of score 0 and without a value,
+    const float* sink_scores;   // or of a score of the head's own ([nh], not scaled) where this is given
     int maps;               // maps a head: rows of q and of the keys hold maps * d entries, outputs maps rows a head
     float softcap;          // > 0: scores become softcap * tanh(score / softcap)
     float temp_coef;        // != 0: the temperature of the queries
@@ -194,12 +195,12 @@ attention_simt_kernel(AttnParams p) {
             ml[1] = l;
         }
     } else {
-        // with a sink: p_j = exp(s_j - M) / (exp(-M) + sum_j exp(s_j - M)) with M = max(m, 0), so that neither term overflows
+        // with a sink of score z: p_j = exp(s_j - M) / (exp(z - M) + sum_j exp(s_j - M)) with M = max(m, z), so that neither term overflows
         float up = 1.f;
         if (p.sink) {
-            const float M = fmaxf(m, 0.f);
+            const float z = p.sink_scores ? p.sink_scores[head] : 0.f, M = fmaxf(m, z);
             up = expf(m - M);
-            l = l * up + expf(-M);
+            l = l * up + expf(z - M);
         }
         const float inv = l > 0.f ? up / l : 0.f;
 #pragma unroll
@@ -237,9 +238,10 @@ __global__ void attention_merge_kernel(AttnParams p, int total_tokens) {
         return;
     }
     const float* ml = p.part_ml + (size_t)row * p.max_splits * 2;
-    float M = p.sink ? 0.f : -INFINITY;   // the sink is one more partial with maximum 0 and sum 1
+    const float z = p.sink && p.sink_scores ? p.sink_scores[row / p.maps % p.nh] : 0.f;
+    float M = p.sink ? z : -INFINITY;     // the sink is one more partial whose maximum is its score and whose sum is 1
     for (int s = s_begin; s < s_end; s++) M = fmaxf(M, ml[2 * s]);
-    float L = p.sink ? expf(-M) : 0.f;
+    float L = p.sink ? expf(z - M) : 0.f;
     for (int s = s_begin; s < s_end; s++) L += ml[2 * s + 1] * expf(ml[2 * s] - M);
     const float inv = L > 0.f ? 1.0f / L : 0.f;
     const float* pa = p.part_acc + (size_t)row * p.max_splits * p.dv;
@@ -313,8 +315,9 @@ HYMT2_API int hymt2_diff_combine(void* out, int out_dtype, const float* a, int t
 // (part_acc [token, head, split, d], part_ml [token, head, split, (max, sum)]).
 int hymt2_attention_merge_launch(void* out, int dtype, const int* cu_seqlens, const int* slot_ids, const int* kv_lens,
                                  float* part_acc, float* part_ml, int tokens, int nh, int d, int window, int split_keys,
-                                 int max_splits, cudaStream_t stream, int* status) {
+                                 int max_splits, cudaStream_t stream, int* status, const float* sink_scores) {
     AttnParams p{};
+    p.sink = sink_scores ? 1 : 0; p.sink_scores = sink_scores;
     p.status = status;
     p.out = out; p.cu_seqlens = cu_seqlens; p.slot_ids = slot_ids; p.kv_lens = kv_lens;
     p.part_acc = part_acc; p.part_ml = part_ml; p.nh = nh; p.d = d; p.dv = d; p.window = window; p.maps = 1;
@@ -338,7 +341,8 @@ static int attention_simt_general(void* out, const void* q, const void* k_cache,
                                   int batch, int tokens, int max_new_tokens, int nh, int nkv, int d, int dv,
                                   float scale, int window, int split_keys, int max_splits,
                                   float* part_acc, float* part_ml, cudaStream_t stream, int* status, int sink = 0,
-                                  int maps = 1, float softcap = 0.f, float temp_coef = 0.f, int temp_every = 1) {
+                                  int maps = 1, float softcap = 0.f, float temp_coef = 0.f, int temp_every = 1,
+                                  const float* sink_scores = nullptr) {
     if (tokens == 0 || batch == 0) return HYMT2_OK;
     HYMT2_REQUIRE(batch > 0 && tokens > 0 && nh > 0 && nkv > 0, "attention: bad sizes");
     HYMT2_REQUIRE(nh % nkv == 0, "attention: %d heads are not a multiple of %d kv heads", nh, nkv);
@@ -362,7 +366,8 @@ static int attention_simt_general(void* out, const void* q, const void* k_cache,
     p.split_keys = split_keys; p.max_splits = split_keys > 0 ? max_splits : 1;
     p.scale = scale;
     p.status = status;
-    p.sink = sink;
+    p.sink = sink || sink_scores ? 1 : 0;
+    p.sink_scores = sink_scores;
     HYMT2_REQUIRE(maps >= 1 && (maps == 1 || v_cache) && softcap >= 0.f && temp_every > 0, "attention: %d maps, a cap of %g, a temperature every %d positions",
                   maps, (double)softcap, temp_every);
     p.maps = maps; p.softcap = softcap; p.temp_coef = temp_coef; p.temp_every = temp_every;
@@ -429,16 +434,16 @@ HYMT2_API int hymt2_attention_simt_maps(void* out, const void* q, const void* k_
 
 // Attention over a cache that holds ONE vector per token and layer, shared by all heads: the key of every head
 // is the whole vector (width d), its value the first dv entries.  (A low-rank key/value cache read in its
-// compressed form: the queries come already multiplied into the compressed space.)
+// compressed form: the queries come already multiplied into the compressed space.)  `sink_scores` [nh] or null: a sink a head.
 HYMT2_API int hymt2_attention_shared_vector(void* out, const void* q, const void* cache, int dtype,
                                             const int* block_table, int table_stride, int block_tokens,
                                             const int* cu_seqlens, const int* slot_ids, const int* kv_lens,
                                             int batch, int tokens, int max_new_tokens, int nh, int d, int dv,
-                                            float scale, int window, int split_keys, int max_splits,
+                                            float scale, int window, const float* sink_scores, int split_keys, int max_splits,
                                             float* part_acc, float* part_ml, cudaStream_t stream, int* status) {
     return attention_simt_general(out, q, cache, nullptr, dtype, block_table, table_stride, block_tokens, cu_seqlens, slot_ids,
                                   kv_lens, batch, tokens, max_new_tokens, nh, 1, d, dv, scale, window, split_keys, max_splits,
-                                  part_acc, part_ml, stream, status);
+                                  part_acc, part_ml, stream, status, 0, 1, 0.f, 0.f, 1, sink_scores);
 }
 
 // ---------------------------------------------------------------------------

@@ -1,7 +1,8 @@
 // The end of a block whose sublayers read the same rows: their outputs join the residual together, each multiplied entry by
-// entry by a stored vector, and the norm that reads the residual next is computed on the way.  One block of threads a token:
+// entry by a stored vector where it has one, and the norm that reads the residual next is computed on the way.  One block of
+// threads a token:
 //
-//     v = x + sum_b gain_b * y_b                                       (up to MAX_BRANCHES plain branches)
+//     v = x + sum_b gain_b * (y_b + bias_b)                            (up to MAX_BRANCHES plain branches; gain and bias may be absent)
 //           + gain_r * (sum_k weight[k] * routed[pair_row[k]] + sigmoid(z) * shared)      (a mixture's pieces, if there is one)
 //     x <- v;   h = v / sqrt(mean(v^2) + eps) * norm_gain              (if the next reader's norm is known)
 //
@@ -11,17 +12,18 @@
 
 namespace {
 
-constexpr int MAX_BRANCHES = 2, MAX_TOP = 32;
+constexpr int MAX_BRANCHES = 3, MAX_TOP = 32;
 
 struct JoinParams {
     float* x;                        // [T, width]
     const float* y[MAX_BRANCHES];    // [T, width]
-    const float* gain[MAX_BRANCHES]; // [width]
+    const float* gain[MAX_BRANCHES]; // [width] or null
+    const float* bias[MAX_BRANCHES]; // [width] or null
     int branches, width;
     const float* routed;             // sorted rows [rows, width], or null
     const int* pair_row;             // [T, top]
     const float* weight;             // [T, top]
-    const float* routed_gain;        // [width]
+    const float* routed_gain;        // [width] or null
     int top;
     const float* shared;             // [T, width] or null
     const float* z;                  // the shared branch's gate in front of its sigmoid, one a token (row stride ldz), or null: 1
@@ -54,9 +56,20 @@ join_branches_kernel(JoinParams p) {
     auto piece = [&](int c) {
         Pack<float, V> v = load_pack<float, V>(p.x + t * width + c);
         for (int b = 0; b < p.branches; b++) {
-            const Pack<float, V> y = load_pack<float, V>(p.y[b] + t * width + c), g = load_pack<float, V>(p.gain[b] + c);
+            Pack<float, V> y = load_pack<float, V>(p.y[b] + t * width + c);
+            if (p.bias[b]) {
+                const Pack<float, V> z = load_pack<float, V>(p.bias[b] + c);
 #pragma unroll
-            for (int k = 0; k < V; k++) v.v[k] = fmaf(y.v[k], g.v[k], v.v[k]);
+                for (int k = 0; k < V; k++) y.v[k] += z.v[k];
+            }
+            if (p.gain[b]) {
+                const Pack<float, V> g = load_pack<float, V>(p.gain[b] + c);
+#pragma unroll
+                for (int k = 0; k < V; k++) v.v[k] = fmaf(y.v[k], g.v[k], v.v[k]);
+            } else {
+#pragma unroll
+                for (int k = 0; k < V; k++) v.v[k] += y.v[k];
+            }
         }
         if (p.routed) {
             float m[V];
@@ -73,9 +86,14 @@ join_branches_kernel(JoinParams p) {
 #pragma unroll
                 for (int k = 0; k < V; k++) m[k] = fmaf(share, y.v[k], m[k]);
             }
-            const Pack<float, V> g = load_pack<float, V>(p.routed_gain + c);
+            if (p.routed_gain) {
+                const Pack<float, V> g = load_pack<float, V>(p.routed_gain + c);
 #pragma unroll
-            for (int k = 0; k < V; k++) v.v[k] = fmaf(m[k], g.v[k], v.v[k]);
+                for (int k = 0; k < V; k++) v.v[k] = fmaf(m[k], g.v[k], v.v[k]);
+            } else {
+#pragma unroll
+                for (int k = 0; k < V; k++) v.v[k] += m[k];
+            }
         }
         store_pack<float, V>(p.x + t * width + c, v);
 #pragma unroll
@@ -131,22 +149,28 @@ void launch_join(const JoinParams& p, int tokens, bool vec, cudaStream_t stream)
 
 }  // namespace
 
-// `routed` null: no mixture; `h` null: no norm.  Gains of branches are float32; the norm's gain has a type of its own.
-HYMT2_API int hymt2_join_branches(float* x, const float* y0, const float* gain0, const float* y1, const float* gain1, const float* routed,
-                                  const int* pair_row, const float* weight, int top, const float* routed_gain, const float* shared,
-                                  const float* z, long ldz, void* h, int h_dtype, const void* norm_gain, int norm_gain_dtype, float eps,
-                                  int tokens, int width, cudaStream_t stream) {
+// `branches` plain branches: y, gain and bias are host arrays of that many device pointers (a gain or a bias may be null).
+// `routed` null: no mixture; `h` null: no norm.  Gains and biases of branches are float32; the norm's gain has a type of its own.
+HYMT2_API int hymt2_join_branches(float* x, const float* const* y, const float* const* gain, const float* const* bias, int branches,
+                                  const float* routed, const int* pair_row, const float* weight, int top, const float* routed_gain,
+                                  const float* shared, const float* z, long ldz, void* h, int h_dtype, const void* norm_gain,
+                                  int norm_gain_dtype, float eps, int tokens, int width, cudaStream_t stream) {
     if (tokens == 0) return HYMT2_OK;
     HYMT2_REQUIRE(tokens > 0 && width > 0 && x, "join_branches: bad sizes");
-    HYMT2_REQUIRE(!y0 == !gain0 && !y1 == !gain1 && (y0 || !y1), "join_branches: a branch comes with its gain, the first before the second");
-    HYMT2_REQUIRE(!routed || (pair_row && weight && routed_gain && top > 0 && top <= MAX_TOP), "join_branches: at most %d chosen experts are taken", MAX_TOP);
+    HYMT2_REQUIRE(branches >= 0 && branches <= MAX_BRANCHES, "join_branches: %d plain branches (at most %d)", branches, MAX_BRANCHES);
+    HYMT2_REQUIRE(!routed || (pair_row && weight && top > 0 && top <= MAX_TOP), "join_branches: at most %d chosen experts are taken", MAX_TOP);
     HYMT2_REQUIRE(!shared || routed, "join_branches: a shared expert stands beside routed ones");
     HYMT2_REQUIRE(!h || norm_gain, "join_branches: a norm needs its gain");
-    JoinParams p{x, {y0, y1}, {gain0, gain1}, y1 ? 2 : (y0 ? 1 : 0), width, routed, pair_row, weight, routed_gain, top, shared, z, ldz, h, norm_gain, eps};
-    bool vec = width % 4 == 0;
-    for (const void* q : {(const void*)x, (const void*)y0, (const void*)gain0, (const void*)y1, (const void*)gain1, (const void*)routed,
-                          (const void*)routed_gain, (const void*)shared, (const void*)h, norm_gain})
-        vec = vec && (uintptr_t)q % 16 == 0;
+    JoinParams p = {};
+    p.x = x; p.branches = branches; p.width = width; p.routed = routed; p.pair_row = pair_row; p.weight = weight; p.routed_gain = routed_gain;
+    p.top = top; p.shared = shared; p.z = z; p.ldz = ldz; p.h = h; p.norm_gain = norm_gain; p.eps = eps;
+    uintptr_t bits = (uintptr_t)x | (uintptr_t)routed | (uintptr_t)routed_gain | (uintptr_t)shared | (uintptr_t)h | (uintptr_t)norm_gain;
+    for (int b = 0; b < branches; b++) {
+        HYMT2_REQUIRE(y[b], "join_branches: branch %d is missing", b);
+        p.y[b] = y[b]; p.gain[b] = gain[b]; p.bias[b] = bias[b];
+        bits |= (uintptr_t)y[b] | (uintptr_t)gain[b] | (uintptr_t)bias[b];
+    }
+    const bool vec = width % 4 == 0 && bits % 16 == 0;
     HYMT2_DISPATCH_DTYPE(norm_gain_dtype, TW, HYMT2_DISPATCH_DTYPE(h_dtype, TH, (launch_join<TW, TH>(p, tokens, vec, stream))));
     return hymt2_check_launch("join_branches");
 }

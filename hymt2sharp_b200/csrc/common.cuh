@@ -121,6 +121,35 @@ cudaError_t launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t s
         else { hymt2_set_error("unknown dtype code %d", (int)(code)); return HYMT2_ERR_ARGUMENT; } \
     } while (0)
 
+// What a gated product makes of a gate entry g and its up entry u, the product's two sums for output feature n of N:
+//     GLU_SILU     g * sigmoid(g) * u
+//     GLU_CLAMPED  g <- min(g, limit), u <- clamp(u, -limit, limit): g * sigmoid(alpha * g) * (u + 1)
+// in float32; `bias` (or null): [2N], the gate rows' entries, then the up rows', added to the sums first.
+enum { GLU_SILU = 0, GLU_CLAMPED = 1 };
+struct GluRule {
+    int kind = GLU_SILU;
+    float limit = 0.f, alpha = 1.f;
+    const float* bias = nullptr;
+};
+__device__ __forceinline__ float silu_mul(float g, float u) { return g / (1.0f + expf(-g)) * u; }
+__device__ __forceinline__ float glu_at(const GluRule& r, float g, float u, int n, int N) {
+    if (r.bias) { g += r.bias[n]; u += r.bias[N + n]; }
+    if (r.kind == GLU_SILU) return silu_mul(g, u);
+    g = fminf(g, r.limit);
+    u = fminf(fmaxf(u, -r.limit), r.limit);
+    return g / (1.0f + expf(-r.alpha * g)) * (u + 1.0f);
+}
+// V neighbouring features from n on (those from N on are computed without a bias and never used); the rule is looked at once
+template <int V> __device__ __forceinline__ void glu_pack(const GluRule& r, const float* g, const float* u, float* o, int n, int N) {
+    if (r.kind == GLU_SILU && !r.bias) {
+#pragma unroll
+        for (int i = 0; i < V; i++) o[i] = silu_mul(g[i], u[i]);
+        return;
+    }
+#pragma unroll
+    for (int i = 0; i < V; i++) o[i] = n + i < N ? glu_at(r, g[i], u[i], n + i, N) : 0.f;
+}
+
 // V neighbouring elements in one access of V * sizeof(T) bytes (the caller has checked the alignment).
 template <typename T, int V> struct Pack { T v[V]; };
 template <typename T, int V> __device__ __forceinline__ Pack<T, V> load_pack(const T* p) {

@@ -29,6 +29,40 @@ HYMT2_API int hymt2_embed(float* out, const void* table, int table_dtype, const 
     return hymt2_check_launch("embed");
 }
 
+// The same with a stored vector per position: out[t] = table[id] * scale + positions[pos[t]] (not scaled), written a second time to
+// `copy` where one is given (a model that needs the embedding's output again further up).  A position outside the table gives
+// status 3 and zeros.
+template <typename T>
+__global__ void embed_positions_kernel(float* __restrict__ out, float* __restrict__ copy, const T* __restrict__ table, const T* __restrict__ positions,
+                                       const int* __restrict__ ids, const int* __restrict__ token_pos, int hidden, int vocab, int max_positions,
+                                       float scale, int* status) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const size_t t = blockIdx.x;
+    const int id = ids[t], pos = token_pos[t];
+    const bool ok = id >= 0 && id < vocab && pos >= 0 && pos < max_positions;
+    if (!ok && threadIdx.x == 0) atomicExch(status, id < 0 || id >= vocab ? 1 : 3);
+    const T* row = table + (size_t)(ok ? id : 0) * hidden;
+    const T* at = positions + (size_t)(ok ? pos : 0) * hidden;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+        const float v = ok ? fmaf(to_float(row[i]), scale, to_float(at[i])) : 0.f;
+        out[t * hidden + i] = v;
+        if (copy) copy[t * hidden + i] = v;
+    }
+}
+
+HYMT2_API int hymt2_embed_positions(float* out, float* copy, const void* table, const void* positions, int table_dtype, const int* ids,
+                                    const int* token_pos, int tokens, int hidden, int vocab, int max_positions, float scale, int* status,
+                                    cudaStream_t stream) {
+    if (tokens == 0) return HYMT2_OK;
+    HYMT2_REQUIRE(tokens > 0 && hidden > 0 && vocab > 0 && max_positions > 0 && positions, "embed_positions: bad sizes tokens=%d hidden=%d vocab=%d positions=%d",
+                  tokens, hidden, vocab, max_positions);
+    HYMT2_DISPATCH_DTYPE(table_dtype, T,
+        launch_pdl(embed_positions_kernel<T>, dim3(tokens), dim3(256), 0, stream, out, copy, (const T*)table, (const T*)positions, ids, token_pos,
+                   hidden, vocab, max_positions, scale, status));
+    return hymt2_check_launch("embed_positions");
+}
+
 // The same with a second table: out[t] = table[id] * scale + pairs[row], row = (previous token * mul_prev + id * mul_cur) mod
 // buckets, and row `buckets` for a sequence's first token (position 0).  The token in front of a step's first one is the
 // int32 at `state_offset` of the sequence's state row, which then receives the step's last token: the block of a sequence's

@@ -8,7 +8,7 @@
 // Epilogues:
 //   0 store      C = acc
 //   1 accumulate C += acc                      (projection back into the residual stream)
-//   2 swiglu     C = silu(acc_gate) * acc_up   (W holds N gate rows, then N up rows;
+//   2 swiglu     C = silu(acc_gate) * acc_up, or what another GluRule says   (W holds N gate rows, then N up rows;
 //                                               src/HyMT2Sharp/Ops.cs:1053)
 #include "common.cuh"
 
@@ -39,7 +39,7 @@ __device__ __forceinline__ void load4(const T* row, int k, int K, bool row_ok, b
 template <typename TA, typename TW, typename TC, int EPI>
 __global__ void __launch_bounds__(THREADS)
 gemm_simt_kernel(TC* __restrict__ C, const TA* __restrict__ A, const TW* __restrict__ W, int M, int N, int K,
-                 long lda, long ldw, long ldc, bool vec_a, bool vec_w, long a_bs, long w_bs, long c_bs) {
+                 long lda, long ldw, long ldc, bool vec_a, bool vec_w, long a_bs, long w_bs, long c_bs, GluRule glu) {
     constexpr int NB = EPI == EPI_SWIGLU ? 2 : 1;
     // a batch of products with the same sizes: blockIdx.z picks the operands (strides in elements)
     A += (size_t)blockIdx.z * a_bs;
@@ -111,8 +111,7 @@ gemm_simt_kernel(TC* __restrict__ C, const TA* __restrict__ A, const TW* __restr
             } else if constexpr (EPI == EPI_ACCUMULATE) {
                 *c = from_float<TC>(to_float(*c) + acc[0][i][j]);
             } else {
-                const float g = acc[0][i][j], u = acc[NB - 1][i][j];
-                *c = from_float<TC>(g / (1.0f + expf(-g)) * u);
+                *c = from_float<TC>(glu_at(glu, acc[0][i][j], acc[NB - 1][i][j], n, N));
             }
         }
     }
@@ -120,13 +119,13 @@ gemm_simt_kernel(TC* __restrict__ C, const TA* __restrict__ A, const TW* __restr
 
 template <typename TA, typename TW, typename TC>
 int launch(void* C, const void* A, const void* W, int M, int N, int K, long lda, long ldw, long ldc, int epi,
-           cudaStream_t stream, int batch = 1, long a_bs = 0, long w_bs = 0, long c_bs = 0) {
+           cudaStream_t stream, int batch = 1, long a_bs = 0, long w_bs = 0, long c_bs = 0, GluRule glu = GluRule{}) {
     dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM, batch);
     const bool vec_a = (lda % 4 == 0) && ((uintptr_t)A % 16 == 0) && (a_bs * sizeof(TA)) % 16 == 0;
     const bool vec_w = (ldw % 4 == 0) && ((uintptr_t)W % 16 == 0) && (w_bs * sizeof(TW)) % 16 == 0;
 #define HYMT2_GEMM_CASE(E)                                                                                  \
     gemm_simt_kernel<TA, TW, TC, E><<<grid, THREADS, 0, stream>>>((TC*)C, (const TA*)A, (const TW*)W, M, N, K, \
-                                                                  lda, ldw, ldc, vec_a, vec_w, a_bs, w_bs, c_bs)
+                                                                  lda, ldw, ldc, vec_a, vec_w, a_bs, w_bs, c_bs, glu)
     if (epi == EPI_STORE) HYMT2_GEMM_CASE(EPI_STORE);
     else if (epi == EPI_ACCUMULATE) HYMT2_GEMM_CASE(EPI_ACCUMULATE);
     else HYMT2_GEMM_CASE(EPI_SWIGLU);
@@ -266,13 +265,13 @@ gemm_skinny_batched_kernel(TC* __restrict__ C, const T* __restrict__ A, const T*
 // The grouped product for few sorted rows (a decode step): row tiles of GROUP_SKINNY_ROWS rows, a warp per output column
 // reads its weight row once, 16 bytes a lane, and keeps a float32 sum for every row of the tile.  The time is that of
 // reading the matrices of the groups in use once.  For gated experts (EPI_SWIGLU: a group's matrix holds N gate rows, then N up
-// rows) the warp's two weight rows are a gate row and its up row, and one column silu(gate) * up comes out.
+// rows) the warp's two weight rows are a gate row and its up row, and one column comes out, what the GluRule makes of the two.
 constexpr int GROUP_SKINNY_ROWS = 8, GROUP_SKINNY_COLS = 2;   // rows of a tile; output columns (weight rows) of a warp
 
 template <typename T, typename TC, int EPI>
 __global__ void __launch_bounds__(SKINNY_WARPS * 32)
 gemm_skinny_grouped_kernel(TC* __restrict__ C, const T* __restrict__ A, const T* __restrict__ W, const int* __restrict__ tile_group,
-                           const int* __restrict__ row_source, int gather, int N, int K, long lda, long ldc, long w_gs, bool vec) {
+                           const int* __restrict__ row_source, int gather, int N, int K, long lda, long ldc, long w_gs, bool vec, GluRule glu) {
     pdl_wait();
     pdl_launch_dependents();
     const int group = tile_group[blockIdx.y];
@@ -358,7 +357,7 @@ gemm_skinny_grouped_kernel(TC* __restrict__ C, const T* __restrict__ A, const T*
         if (ok[m]) {
             if constexpr (GATED) {
                 const float gate = warp_sum(acc[0][m]), up = warp_sum(acc[1][m]);
-                if (lane == 0) C[(size_t)(m0 + m) * ldc + n0] = from_float<TC>(gate / (1.0f + expf(-gate)) * up);
+                if (lane == 0) C[(size_t)(m0 + m) * ldc + n0] = from_float<TC>(glu_at(glu, gate, up, n0, N));
                 continue;
             }
 #pragma unroll
@@ -376,14 +375,14 @@ gemm_skinny_grouped_kernel(TC* __restrict__ C, const T* __restrict__ A, const T*
 // C[M,N] (ldc) = epilogue(A[M,K] (lda) · W[N,K]^T (ldw)); for the swiglu epilogue W has 2N rows.
 HYMT2_API int hymt2_gemm_simt(void* C, int c_dtype, const void* A, int a_dtype, const void* W, int w_dtype,
                               int M, int N, int K, long lda, long ldw, long ldc, int epilogue,
-                              cudaStream_t stream) {
+                              int glu_kind, float glu_limit, float glu_alpha, const float* glu_bias, cudaStream_t stream) {
     if (M == 0 || N == 0) return HYMT2_OK;
     HYMT2_REQUIRE(M > 0 && N > 0 && K > 0, "gemm: bad sizes M=%d N=%d K=%d", M, N, K);
     HYMT2_REQUIRE(epilogue >= 0 && epilogue <= 2, "gemm: unknown epilogue %d", epilogue);
     HYMT2_REQUIRE(lda >= K && ldw >= K && ldc >= N, "gemm: a leading dimension is smaller than its row");
     HYMT2_REQUIRE((M + BM - 1) / BM <= 65535, "gemm: M=%d needs more than 65535 row tiles", M);
     HYMT2_DISPATCH_DTYPE(a_dtype, TA, HYMT2_DISPATCH_DTYPE(w_dtype, TW, HYMT2_DISPATCH_DTYPE(c_dtype, TC,
-        return (launch<TA, TW, TC>(C, A, W, M, N, K, lda, ldw, ldc, epilogue, stream)))));
+        return (launch<TA, TW, TC>(C, A, W, M, N, K, lda, ldw, ldc, epilogue, stream, 1, 0, 0, 0, GluRule{glu_kind, glu_limit, glu_alpha, glu_bias})))));
     return HYMT2_OK;
 }
 
@@ -447,8 +446,9 @@ HYMT2_API int hymt2_gemm_simt_group_tile() { return BM; }
 // The grouped product for few rows: row tiles of hymt2_gemm_skinny_group_tile() sorted rows, A and W of one type.
 HYMT2_API int hymt2_gemm_skinny_grouped(void* C, int c_dtype, const void* A, const void* W, int dtype, const int* tile_group,
                                         const int* row_source, int gather, int tiles, int N, int K, long lda, long ldc, long w_gs,
-                                        int epilogue, cudaStream_t stream) {
+                                        int epilogue, int glu_kind, float glu_limit, float glu_alpha, cudaStream_t stream) {
     if (tiles == 0 || N == 0) return HYMT2_OK;
+    const GluRule glu{glu_kind, glu_limit, glu_alpha, nullptr};
     HYMT2_REQUIRE(tiles > 0 && tiles <= 65535 && N > 0 && K > 0, "gemm_skinny_grouped: bad sizes tiles=%d N=%d K=%d", tiles, N, K);
     HYMT2_REQUIRE(epilogue == EPI_STORE || epilogue == EPI_RELU_SQUARED || epilogue == EPI_SWIGLU, "gemm_skinny_grouped: unknown epilogue %d", epilogue);
     HYMT2_REQUIRE(lda >= K && ldc >= N && tile_group && row_source, "gemm_skinny_grouped: bad arguments");
@@ -460,13 +460,13 @@ HYMT2_API int hymt2_gemm_skinny_grouped(void* C, int c_dtype, const void* A, con
         HYMT2_DISPATCH_DTYPE(c_dtype, TC, {
             if (epilogue == EPI_STORE)
                 launch_pdl(gemm_skinny_grouped_kernel<T, TC, EPI_STORE>, grid, dim3(SKINNY_WARPS * 32), 0, stream, (TC*)C, (const T*)A,
-                           (const T*)W, tile_group, row_source, gather, N, K, lda, ldc, w_gs, vec);
+                           (const T*)W, tile_group, row_source, gather, N, K, lda, ldc, w_gs, vec, glu);
             else if (epilogue == EPI_SWIGLU)
                 launch_pdl(gemm_skinny_grouped_kernel<T, TC, EPI_SWIGLU>, grid, dim3(SKINNY_WARPS * 32), 0, stream, (TC*)C, (const T*)A,
-                           (const T*)W, tile_group, row_source, gather, N, K, lda, ldc, w_gs, vec);
+                           (const T*)W, tile_group, row_source, gather, N, K, lda, ldc, w_gs, vec, glu);
             else
                 launch_pdl(gemm_skinny_grouped_kernel<T, TC, EPI_RELU_SQUARED>, grid, dim3(SKINNY_WARPS * 32), 0, stream, (TC*)C,
-                           (const T*)A, (const T*)W, tile_group, row_source, gather, N, K, lda, ldc, w_gs, vec);
+                           (const T*)A, (const T*)W, tile_group, row_source, gather, N, K, lda, ldc, w_gs, vec, glu);
         });
     });
     return hymt2_check_launch("gemm_skinny_grouped");

@@ -21,7 +21,7 @@
 //            (Where a ring for two CTAs on an SM would be too shallow, each split CTA has an SM to
 //            itself and a deep ring; partial tiles then go through a global workspace, folded by the
 //            CTA that arrives last at the tile's counter, also in split order.)
-// Epilogues: store, accumulate into float32 C, SwiGLU (silu(gate) * up; W holds N gate rows,
+// Epilogues: store, accumulate into float32 C, SwiGLU (silu(gate) * up, or another GluRule; W holds N gate rows,
 // then N up rows; src/HyMT2Sharp/Ops.cs:1053), and for the fused q/k/v projection with heads of 128 the rotation, the
 // per-head norm and the append to the paged cache (RopeEpilogue).  Rows and K beyond the matrices are zero-filled
 // by TMA and masked in the epilogue, so any T and N are taken; K, lda and ldw must be multiples
@@ -132,6 +132,7 @@ struct GemmTcParams {
     const int* tile_group = nullptr;
     long group_rows = 0;
     int act = 0;             // store epilogue: 1 = the square of relu on the way out
+    GluRule glu;             // EPI_SWIGLU: what a gate and an up entry become
 };
 
 // The copies of one stage (activations, weights, and for a split weight tile its second half) with, in front of them, a
@@ -202,8 +203,6 @@ __device__ __forceinline__ void tmem_load<32>(uint32_t taddr, float* v) {
     tmem_load16(taddr, v);
     tmem_load16(taddr + 16, v + 16);
 }
-
-__device__ __forceinline__ float silu_mul(float g, float u) { return g / (1.0f + expf(-g)) * u; }
 
 __device__ __forceinline__ float bf16_round(float x) { return __bfloat162float(__float2bfloat16_rn(x)); }
 __device__ __forceinline__ void store_bf16x16(__nv_bfloat16* dst, const float* v) {   // dst is 32-byte aligned
@@ -517,6 +516,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
             }
         };
 
+        const bool plain_glu = p.glu.kind == GLU_SILU && !p.glu.bias;
         // one chunk of CH accumulator columns: g (and u for SwiGLU) -> C
         auto emit = [&](int c, const float* g, const float* u) {
             const int n = a_row0 + row;                    // output feature
@@ -537,7 +537,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 const float r = scaled ? scale_s[c + j] : 1.0f;
                 if (EPI == EPI_STORE) *dst = from_float<TC>(g[j] * r);
                 else if (EPI == EPI_ACCUMULATE) *dst = from_float<TC>(old[j] + g[j]);
-                else *dst = from_float<TC>(silu_mul(g[j] * r, u[j] * r));
+                else *dst = from_float<TC>(plain_glu ? silu_mul(g[j] * r, u[j] * r) : glu_at(p.glu, g[j] * r, u[j] * r, n, p.N));
             }
         };
 
@@ -667,8 +667,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                                 for (int i = 0; i < 4; i++) o[i] = n4 + i < p.N ? to_float(dst[i]) + gv[i] : 0.f;
                             }
                         } else {
+if constexpr (EPI == EPI_SWIGLU) glu_pack<4>(p.glu, gv, uv, o, n4, p.N);
+                            else {
 #pragma unroll
-                            for (int i = 0; i < 4; i++) o[i] = EPI == EPI_STORE ? gv[i] : silu_mul(gv[i], uv[i]);
+                                for (int i = 0; i < 4; i++) o[i] = gv[i];
+                            }
                         }
                         if (c_vec) {
                             if constexpr (sizeof(TC) == 4) *reinterpret_cast<float4*>(dst) = make_float4(o[0], o[1], o[2], o[3]);
@@ -767,7 +770,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                         float o[4];
 #pragma unroll
                         for (int i = 0; i < 4; i++)
-                            o[i] = EPI == EPI_STORE ? gv[i] * r : EPI == EPI_ACCUMULATE ? gv[i] : silu_mul(gv[i] * r, uv[i] * r);
+                            o[i] = EPI == EPI_STORE ? gv[i] * r : EPI == EPI_ACCUMULATE ? gv[i] : plain_glu ? silu_mul(gv[i] * r, uv[i] * r)
+                                 : n0 + i < p.N ? glu_at(p.glu, gv[i] * r, uv[i] * r, n0 + i, p.N) : 0.f;
                         if (whole && (((uintptr_t)dst) & (4 * sizeof(TC) - 1)) == 0) {
                             if constexpr (sizeof(TC) == 4) {
                                 float4 v = make_float4(o[0], o[1], o[2], o[3]);
@@ -1046,10 +1050,14 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __gri
 #pragma unroll
                 for (int j8 = 0; j8 < 16; j8 += 8) {
                     float o[8];
+                    if constexpr (EPI == EPI_SWIGLU) {
 #pragma unroll
-                    for (int q = 0; q < 8; q++)
-                        o[q] = EPI == EPI_SWIGLU ? silu_mul(g[j8 + q] * row_scale, u[j8 + q] * row_scale)
-                             : EPI == EPI_STORE ? g[j8 + q] * row_scale : g[j8 + q];
+                        for (int q = 0; q < 8; q++) { g[j8 + q] *= row_scale; u[j8 + q] *= row_scale; }
+                        glu_pack<8>(p.glu, g + j8, u + j8, o, n0 + j8, p.N);
+                    } else {
+#pragma unroll
+                        for (int q = 0; q < 8; q++) o[q] = EPI == EPI_STORE ? g[j8 + q] * row_scale : g[j8 + q];
+                    }
                     if (EPI == EPI_STORE && p.act == 1) {
 #pragma unroll
                         for (int q = 0; q < 8; q++) { const float z = fmaxf(o[q], 0.f); o[q] = z * z; }
@@ -1337,7 +1345,7 @@ int norm_out_tiles(const Plan& pl, int epilogue, int N) {
 
 int run_gemm_tc(void* C, int c_dtype, const void* X, const void* W, int T, int N, int K, long lda, long ldw, long ldc,
                 int epilogue, float* workspace, long workspace_floats, int* counters, int num_counters, int* status,
-                cudaStream_t stream, uint32_t wait_limit, int withhold_block, NormSide norm = NormSide{}) {
+                cudaStream_t stream, uint32_t wait_limit, int withhold_block, NormSide norm = NormSide{}, GluRule glu = GluRule{}) {
     if (T == 0 || N == 0) return HYMT2_OK;
     HYMT2_REQUIRE(T > 0 && N > 0 && K > 0, "gemm_tc: bad sizes T=%d N=%d K=%d", T, N, K);
     HYMT2_REQUIRE(K % 8 == 0 && lda % 8 == 0 && ldw % 8 == 0, "gemm_tc: K, lda and ldw must be multiples of 8 (K=%d lda=%ld ldw=%ld)", K, lda, ldw);
@@ -1367,6 +1375,7 @@ int run_gemm_tc(void* C, int c_dtype, const void* X, const void* W, int T, int N
     if (norm.ss_in) HYMT2_REQUIRE(epilogue != EPI_ACCUMULATE && norm.ss_in_tiles > 0 && norm.ss_width > 0, "gemm_tc: bad row-scale arguments");
     GemmTcParams p{C, ldc, T, N, K, pl.stages, pl.bn, pl.splits, pl.k_blocks_per_split, pl.cluster ? 1 : 0, workspace, counters, status,
                    RopeEpilogue{}, wait_limit, withhold_block, norm};
+    p.glu = glu;
     // (from 64 token columns on: below that the fold is short, and two thirds of the CTAs leaving early, so that the next
     // kernel's CTAs find room, is worth more; batch 8: 1.63 against 1.82 ms a step, batch 64: 4.05 against 3.95)
     p.together = (pl.swapped && pl.splits > 1 && !pl.cluster && pl.bn >= 64 && (long)pl.grid.x * pl.grid.y * pl.splits <= pl.sm_count) ? 1 : 0;
@@ -1396,9 +1405,10 @@ HYMT2_API int hymt2_gemm_tc(void* C, int c_dtype, const void* X, const void* W, 
 // A grouped product on the persistent kernel: X holds tiles * 128 token rows sorted by group (segments of whole tiles),
 // W the groups' matrices [N, K] one after the other, tile_group[tile] the group of a row tile, tile_group[tiles] the number of
 // tiles in use (the first ones; the others do not run).
-// C[tiles * 128, N] = act(X W[group]^T); act 0: as it is, 1: the square of relu.
+// C[tiles * 128, N] = act(X W[group]^T); act 0: as it is, 1: the square of relu, 2: gate and up rows by the rule of `glu_*`.
 HYMT2_API int hymt2_gemm_tc_grouped(void* C, int c_dtype, const void* X, const void* W, const int* tile_group, int tiles, int groups,
-                                    int N, int K, long lda, long ldc, int act, int* status, cudaStream_t stream) {
+                                    int N, int K, long lda, long ldc, int act, int glu_kind, float glu_limit, float glu_alpha, int* status,
+                                    cudaStream_t stream) {
     if (tiles == 0 || N == 0) return HYMT2_OK;
     HYMT2_REQUIRE(tiles > 0 && groups > 0 && N > 0 && K > 0 && tile_group, "gemm_tc_grouped: bad sizes tiles=%d groups=%d N=%d K=%d", tiles, groups, N, K);
     HYMT2_REQUIRE(K % 8 == 0 && lda % 8 == 0 && N % 8 == 0, "gemm_tc_grouped: K, lda and N must be multiples of 8 (K=%d lda=%ld N=%d)", K, lda, N);
@@ -1418,6 +1428,7 @@ HYMT2_API int hymt2_gemm_tc_grouped(void* C, int c_dtype, const void* X, const v
     p.tile_group = tile_group;
     p.group_rows = rows_w;
     p.act = act == 1 ? 1 : 0;
+    p.glu = GluRule{glu_kind, glu_limit, glu_alpha, nullptr};
     return launch_persistent(ma, mb, p, pl, epi, c_dtype, stream);
 }
 
@@ -1436,11 +1447,11 @@ HYMT2_API int hymt2_gemm_tc_norm(void* C, int c_dtype, const void* X, const void
                                  long ldc, int epilogue, float* workspace, long workspace_floats, int* counters,
                                  int num_counters, int* status, cudaStream_t stream, const float* ss_in, int ss_in_tiles,
                                  int ss_width, float ss_eps, void* norm_out, const void* norm_gain, int norm_gain_dtype,
-                                 float* ss_out) {
+                                 float* ss_out, int glu_kind, float glu_limit, float glu_alpha, const float* glu_bias) {
     HYMT2_REQUIRE(!norm_out || norm_gain_dtype == HYMT2_BF16 || norm_gain_dtype == HYMT2_F32, "gemm_tc_norm: the gain must be bfloat16 or float32");
     NormSide ns{(__nv_bfloat16*)norm_out, norm_gain, norm_gain_dtype == HYMT2_BF16 ? 1 : 0, ss_out, 0, ss_in, ss_in_tiles, ss_width, ss_eps};
     return run_gemm_tc(C, c_dtype, X, W, T, N, K, lda, ldw, ldc, epilogue, workspace, workspace_floats, counters, num_counters,
-                       status, stream, WAIT_LIMIT, -1, ns);
+                       status, stream, WAIT_LIMIT, -1, ns, GluRule{glu_kind, glu_limit, glu_alpha, glu_bias});
 }
 
 // The same product with one fault put in on purpose, for the test of the bounded waits: the producer announces

@@ -9,6 +9,9 @@
 //   * rotates the shared key part by the token's position and writes it behind it, entries [rank, rank + rot);
 //   * rotates the `rot` part of every head's query and writes it to q_out[t, h, rank .. rank + rot): the place
 //     behind the head's `rank` entries, which the product with the key up-projection fills.
+// Where the queries come out of a latent vector of their own, the projection starts with that vector instead: it is normed
+// with its gain into cq_out, and the heads' queries, once a product has made them, come through this kernel in a second
+// call, as a projection without a compressed row.
 // Rotation: of the first `rot_dims` entries, (2i, 2i+1) are a pair that turns by angle = position * inv_freq[i]
 // (a float32 product); cosine and sine are multiplied by `amplitude`; entries from rot_dims on pass unchanged.
 // Cache plane: [block][token in block][rank + rot]; block_table[slot * table_stride + pos / block_tokens] names
@@ -29,7 +32,11 @@ struct LatentPrepParams {
     const float* gain;      // [rank]
     const float* inv_freq;  // [rot_dims / 2]
     long ldp;
-    int q_cols;             // where the compressed row starts inside a projection row (= heads * (dim + rot))
+    int q_cols;             // where the compressed row starts inside a projection row: behind the queries (heads * (dim + rot)), or
+                            // behind a compressed query of q_rank entries
+    const float* q_gain;    // [q_rank]: the projection starts with a compressed query, which is normed into cq_out; null: with the queries
+    void* cq_out;           // [T, q_rank]
+    int q_rank;
     int table_stride, block_tokens, heads, dim, rot, rank, rot_dims;
     float eps, amplitude;
 };
@@ -89,6 +96,17 @@ latent_prep_kernel(LatentPrepParams p) {
             if (dst2) dst2[p.rank + i] = kr[i];
         }
     }
+    if (p.cq_out) {   // the compressed query: normed as the latent vector is; there are no heads' queries yet
+        float qs = 0.f;
+        for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) {
+            const float v = to_float(row[i]);
+            qs = fmaf(v, v, qs);
+        }
+        const float scale = 1.0f / sqrtf(block_sum(qs, scratch) / (float)p.q_rank + p.eps);
+        T* o = (T*)p.cq_out + (size_t)t * p.q_rank;
+        for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) o[i] = from_float<T>(to_float(row[i]) * scale * p.q_gain[i]);
+        return;
+    }
     // the heads' rotated query parts
     const int per_head = half + (p.rot - p.rot_dims);
     for (int item = threadIdx.x; item < p.heads * per_head; item += blockDim.x) {
@@ -110,14 +128,17 @@ latent_prep_kernel(LatentPrepParams p) {
 
 HYMT2_API int hymt2_latent_prep(const void* proj, long ldp, int q_cols, void* q_out, void* rows_out, void* cache, int dtype,
                                 const int* block_table, int table_stride, int block_tokens, const int* token_seq,
-                                const int* token_pos, const int* slot_ids, const float* gain, const float* inv_freq,
+                                const int* token_pos, const int* slot_ids, const float* gain, const float* q_gain, void* cq_out, int q_rank,
+                                const float* inv_freq,
                                 int rot_dims, float amplitude, float eps, int tokens, int heads, int dim, int rot, int rank,
                                 cudaStream_t stream) {
     if (tokens == 0) return HYMT2_OK;
-    HYMT2_REQUIRE(tokens > 0 && heads > 0 && dim >= 0 && rot >= 0 && rank > 0, "latent_prep: bad sizes");
+    HYMT2_REQUIRE(tokens > 0 && heads >= 0 && dim >= 0 && rot >= 0 && rank > 0, "latent_prep: bad sizes");
     HYMT2_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= rot, "latent_prep: %d rotated entries of %d", rot_dims, rot);
     HYMT2_REQUIRE(rot_dims == 0 || inv_freq != nullptr, "latent_prep: no frequencies");
+    HYMT2_REQUIRE(!cq_out || (q_gain && q_rank > 0 && q_rank <= q_cols && heads == 0), "latent_prep: a compressed query of %d entries", q_rank);
     LatentPrepParams p;
+    p.q_gain = q_gain; p.cq_out = cq_out; p.q_rank = q_rank;
     p.proj = proj; p.q_out = q_out; p.rows_out = rows_out; p.cache = cache; p.block_table = block_table; p.token_seq = token_seq;
     p.token_pos = token_pos; p.slot_ids = slot_ids; p.gain = gain; p.inv_freq = inv_freq; p.ldp = ldp; p.q_cols = q_cols;
     p.table_stride = table_stride; p.block_tokens = block_tokens; p.heads = heads; p.dim = dim; p.rot = rot; p.rank = rank;

@@ -24,7 +24,7 @@
 
 int hymt2_attention_merge_launch(void* out, int dtype, const int* cu_seqlens, const int* slot_ids, const int* kv_lens,
                                  float* part_acc, float* part_ml, int tokens, int nh, int d, int window, int split_keys,
-                                 int max_splits, cudaStream_t stream, int* status);
+                                 int max_splits, cudaStream_t stream, int* status, const float* sink_scores);
 
 namespace {
 
@@ -54,6 +54,7 @@ struct LatentMmaParams {
     float* part_ml;       // [T * nh, splits, 2]
     int table_stride, nh, d, dv, window, split_keys, max_splits;
     float scale;
+    const float* sink;    // [nh] or null: one more term of this score in a head's softmax, not scaled and without a value
     // the expanded form: q is the projection [T, ldq_g] with head h's d entries at column h * d; out is [T, ld_out]
     const bf16* kexp;     // [T, ld_kexp]: head h's unrotated key entries at column h * dim
     const bf16* vexp;     // [T, ld_vexp]: head h's values at column h * dv
@@ -113,7 +114,13 @@ latent_attention_mma_kernel(LatentMmaParams p) {
         r += step_r; c += step_c;
         if (c >= d) { c -= d; r++; }
     }
-    if (tid < MT) { m_s[tid] = -INFINITY; l_s[tid] = 0.f; corr_s[tid] = 1.f; }
+    if (tid < MT) {
+        // (a row opens with its sink, maximum and sum; where the keys are cut, the merge brings the sink in)
+        const bool opens = p.sink && p.split_keys == 0;
+        m_s[tid] = opens ? p.sink[EXPANDED ? head : (r0 + tid) % p.nh] : -INFINITY;
+        l_s[tid] = opens ? 1.f : 0.f;
+        corr_s[tid] = 1.f;
+    }
 
     // which row of its 16 each entry of an accumulator fragment belongs to
     // A tile of at most 16 live rows (a decode step's heads) is `narrow`: all warps share the one live row fragment and
@@ -331,7 +338,7 @@ HYMT2_API int hymt2_latent_attention_mma_supported(int d, int dv, int block_toke
 
 HYMT2_API int hymt2_latent_attention_mma(void* out, const void* q, const void* cache, const int* block_table, int table_stride,
                                          int block_tokens, const int* cu_seqlens, const int* slot_ids, const int* kv_lens, int batch,
-                                         int tokens, int max_new_tokens, int nh, int d, int dv, float scale, int window,
+                                         int tokens, int max_new_tokens, int nh, int d, int dv, float scale, int window, const float* sink,
                                          int split_keys, int max_splits, float* part_acc, float* part_ml, int* status,
                                          cudaStream_t stream) {
     if (batch == 0 || tokens == 0) return HYMT2_OK;
@@ -342,7 +349,7 @@ HYMT2_API int hymt2_latent_attention_mma(void* out, const void* q, const void* c
     LatentMmaParams p;
     p.q = (const bf16*)q; p.out = (bf16*)out; p.cache = (const bf16*)cache; p.block_table = block_table; p.cu_seqlens = cu_seqlens;
     p.slot_ids = slot_ids; p.kv_lens = kv_lens; p.part_acc = part_acc; p.part_ml = part_ml; p.table_stride = table_stride; p.nh = nh;
-    p.d = d; p.dv = dv; p.window = window; p.split_keys = split_keys; p.max_splits = split_keys > 0 ? max_splits : 1; p.scale = scale;
+    p.d = d; p.dv = dv; p.window = window; p.split_keys = split_keys; p.max_splits = split_keys > 0 ? max_splits : 1; p.scale = scale; p.sink = sink;
     const long row_tiles = ((long)max_new_tokens * nh + MT - 1) / MT;
     HYMT2_REQUIRE(row_tiles <= 2147483647L && (long)batch * p.max_splits <= 65535, "latent_attention_mma: grid too large");
     const dim3 grid((unsigned)row_tiles, 1, (unsigned)(batch * p.max_splits));
@@ -359,7 +366,7 @@ HYMT2_API int hymt2_latent_attention_mma(void* out, const void* q, const void* c
     else rc = launch(latent_attention_mma_kernel<16, false>);
     if (rc == HYMT2_OK && split_keys > 0)
         rc = hymt2_attention_merge_launch(out, HYMT2_BF16, cu_seqlens, slot_ids, kv_lens, part_acc, part_ml, tokens, nh, dv, window,
-                                          split_keys, max_splits, stream, status);
+                                          split_keys, max_splits, stream, status, sink);
     return rc;
 }
 
@@ -372,7 +379,7 @@ HYMT2_API int hymt2_latent_attention_expanded_supported(int dim, int rot, int dv
 HYMT2_API int hymt2_latent_attention_expanded(void* out, long ld_out, const void* q, long ldq, const void* kexp, long ld_kexp,
                                               const void* vexp, long ld_vexp, const void* krot, long ld_krot,
                                               const int* cu_seqlens, const int* slot_ids, const int* kv_lens, int batch,
-                                              int max_new_tokens, int nh, int dim, int rot, int dv, float scale, int window,
+                                              int max_new_tokens, int nh, int dim, int rot, int dv, float scale, int window, const float* sink,
                                               cudaStream_t stream) {
     if (batch == 0 || max_new_tokens == 0) return HYMT2_OK;
     HYMT2_REQUIRE(hymt2_latent_attention_expanded_supported(dim, rot, dv), "latent_attention_expanded: heads of %d + %d key entries and %d value entries are not taken", dim, rot, dv);
@@ -382,7 +389,7 @@ HYMT2_API int hymt2_latent_attention_expanded(void* out, long ld_out, const void
                   "latent_attention_expanded: operands and rows must be 16-byte aligned");
     LatentMmaParams p = {};
     p.q = (const bf16*)q; p.out = (bf16*)out; p.cu_seqlens = cu_seqlens; p.slot_ids = slot_ids; p.kv_lens = kv_lens;
-    p.nh = nh; p.d = dim + rot; p.dv = dv; p.window = window; p.split_keys = 0; p.max_splits = 1; p.scale = scale;
+    p.nh = nh; p.d = dim + rot; p.dv = dv; p.window = window; p.split_keys = 0; p.max_splits = 1; p.scale = scale; p.sink = sink;
     p.kexp = (const bf16*)kexp; p.vexp = (const bf16*)vexp; p.krot = (const bf16*)krot;
     p.ldq_g = ldq; p.ld_out = ld_out; p.ld_kexp = ld_kexp; p.ld_vexp = ld_vexp; p.ld_krot = ld_krot; p.dim = dim;
     const dim3 grid((max_new_tokens + MT - 1) / MT, nh, batch);

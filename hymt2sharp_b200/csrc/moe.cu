@@ -5,9 +5,10 @@
 //
 //   route    scores s = softmax(z + bias) over ALL router outputs, or sigmoid(z + bias) of each (bias: optional); the `top`
 //            largest of s + correction are chosen (ties: the lower index), with several groups of neighbouring outputs only
-//            from the `keep` groups whose two largest have the largest sums; a chosen output's weight is its s, without the
-//            correction, either as it is or (`renorm`) divided by the sum over the chosen ones (for softmax scores that is
-//            the softmax over the chosen outputs alone)
+//            from the `keep` groups whose two largest choice scores have the largest sums (`group_best` 1: whose largest one is
+//            the largest); a chosen output's weight is its s, without the correction, either as it is or (`renorm`) divided by
+//            the sum over the chosen ones (for softmax scores that is the softmax over the chosen outputs alone), times
+//            `weight_scale`
 //   count    how many (token, choice) pairs name each expert that has tensors (outputs from `experts` on name identity
 //            experts, which need no product)
 //   place    every expert's pairs, in token order, get consecutive rows of a sorted list; an expert's segment is padded to
@@ -31,6 +32,8 @@ struct RouteRule {
     int renorm;                // weights: divided by (the sum over the chosen ones + share_eps)
     float share_eps;
     int groups, keep;          // equal groups of neighbouring outputs, of which the best `keep` take part (groups 1: all)
+    int group_best;            // a group is worth its largest choice score (1), or what its two largest add up to (2)
+    float weight_scale;        // the weights are multiplied by this behind everything else
     int outputs, top;
     long ldz;                  // row stride of the router's outputs
 };
@@ -58,7 +61,7 @@ __device__ __forceinline__ void route_token(const RouteRule& r, const float* __r
     for (int i = lane; i < outputs; i += 32) c[i] = s[i] + (r.correction ? r.correction[i] : 0.f);   // (a lane's own entries)
     __syncwarp();
     if (r.groups > 1) {
-        // a group is worth what its two best scores add up to; it stays if fewer than `keep` are worth more (of equals the
+        // a group is worth its best score, or what its two best add up to; it stays if fewer than `keep` are worth more (of equals the
         // lower number counts as more)
         const int per = outputs / r.groups;
         for (int g = lane; g < r.groups; g += 32) {
@@ -67,7 +70,7 @@ __device__ __forceinline__ void route_token(const RouteRule& r, const float* __r
                 if (c[i] > first) { second = first; first = c[i]; }
                 else if (c[i] > second) second = c[i];
             }
-            worth[g] = per > 1 ? first + second : first;
+            worth[g] = per > 1 && r.group_best == 2 ? first + second : first;
         }
         __syncwarp();
         for (int g = lane; g < r.groups; g += 32) {
@@ -101,7 +104,9 @@ __device__ __forceinline__ void route_token(const RouteRule& r, const float* __r
     if (r.renorm && lane == 0) {
         float chosen_sum = 0.f;
         for (int k = 0; k < r.top; k++) chosen_sum += weight[k];
-        for (int k = 0; k < r.top; k++) weight[k] /= chosen_sum + r.share_eps;
+        for (int k = 0; k < r.top; k++) weight[k] = weight[k] / (chosen_sum + r.share_eps) * r.weight_scale;
+    } else if (r.weight_scale != 1.f && lane == 0) {
+        for (int k = 0; k < r.top; k++) weight[k] *= r.weight_scale;
     }
 }
 
@@ -356,15 +361,17 @@ static int check_rule(const char* what, const RouteRule& r, int tokens) {
     HYMT2_REQUIRE(tokens > 0 && r.outputs > 0 && r.top > 0 && r.top <= r.outputs && r.ldz >= r.outputs, "%s: bad sizes tokens=%d outputs=%d top=%d", what,
                   tokens, r.outputs, r.top);
     HYMT2_REQUIRE(r.scores == SCORES_SOFTMAX || r.scores == SCORES_SIGMOID, "%s: unknown kind of scores %d", what, r.scores);
+    HYMT2_REQUIRE(r.group_best == 1 || r.group_best == 2, "%s: a group's worth is its best score or the sum of its two best, not of %d", what, r.group_best);
     HYMT2_REQUIRE(r.groups > 0 && r.outputs % r.groups == 0 && r.keep > 0 && r.keep <= r.groups && (r.groups == 1 || r.top <= r.keep * (r.outputs / r.groups)),
                   "%s: %d of %d groups hold fewer than %d of %d outputs", what, r.keep, r.groups, r.top, r.outputs);
     return HYMT2_OK;
 }
 
 HYMT2_API int hymt2_moe_route(int* chosen, float* weight, const float* logits, long ldz, const float* correction, const float* bias, int scores,
-                              int renorm, float share_eps, int groups, int keep, int tokens, int outputs, int top, cudaStream_t stream) {
+                              int renorm, float share_eps, int groups, int keep, int group_best, float weight_scale, int tokens, int outputs, int top,
+                              cudaStream_t stream) {
     if (tokens == 0) return HYMT2_OK;
-    const RouteRule r{correction, bias, scores, renorm, share_eps, groups, keep, outputs, top, ldz};
+    const RouteRule r{correction, bias, scores, renorm, share_eps, groups, keep, group_best, weight_scale, outputs, top, ldz};
     const int rc = check_rule("moe_route", r, tokens);
     if (rc != HYMT2_OK) return rc;
     const size_t smem = (size_t)ROUTE_WARPS * route_floats(outputs, groups) * sizeof(float);
@@ -402,10 +409,10 @@ HYMT2_API int hymt2_moe_combine(float* out, const float* y, const void* x, int x
 // moe_route and moe_place in one launch for a step of few tokens (tokens * top <= 1024, experts <= 4096).
 HYMT2_API int hymt2_moe_route_place_small(int* chosen, float* weight, int* pair_row, int* row_token, int* tile_group, const float* logits,
                                           long ldz, const float* correction, const float* bias, int scores, int renorm, float share_eps,
-                                          int groups, int keep, int tokens, int outputs, int top, int experts, int tile, int max_tiles,
+                                          int groups, int keep, int group_best, float weight_scale, int tokens, int outputs, int top, int experts, int tile, int max_tiles,
                                           cudaStream_t stream) {
     if (tokens == 0) return HYMT2_OK;
-    const RouteRule r{correction, bias, scores, renorm, share_eps, groups, keep, outputs, top, ldz};
+    const RouteRule r{correction, bias, scores, renorm, share_eps, groups, keep, group_best, weight_scale, outputs, top, ldz};
     const int rc = check_rule("moe_route_place_small", r, tokens);
     if (rc != HYMT2_OK) return rc;
     HYMT2_REQUIRE(experts >= 0 && experts <= outputs && tile > 0, "moe_route_place_small: bad sizes");

@@ -25,6 +25,7 @@ class DecoderModel:
         self.state_bytes = 0
         self._ones = None
         self.pairs = self.join = None            # the bigram table; the product that joins the residual with the embedding's output
+        self.positions = None                    # the table of positions
         self.pair_state_offset = 0
         # a step can be captured into a CUDA graph only if every part launches kernels and nothing else
         self.graph_safe = all(getattr(b, "graph_safe", False) for b in self.blocks)
@@ -36,6 +37,8 @@ class DecoderModel:
         t = {s.embedding: TensorSpec((s.vocab, s.hidden))}
         if s.bigram is not None:
             t[s.bigram.table] = TensorSpec((s.bigram.buckets + 1, s.hidden))
+        if s.positions is not None:
+            t[s.positions] = TensorSpec((s.max_positions, s.hidden))
         if s.join is not None:
             t[s.join] = TensorSpec((s.hidden, 2 * s.hidden))
         for b in self.blocks:
@@ -98,6 +101,10 @@ class DecoderModel:
             self.pairs = compute_form(weights[s.bigram.table], device, dtype)
             if self.pairs.dtype != self.embedding.dtype:
                 self.pairs = self.pairs.to(self.embedding.dtype)
+        if s.positions is not None:
+            self.positions = compute_form(weights[s.positions], device, dtype)
+            if self.positions.dtype != self.embedding.dtype:
+                self.positions = self.positions.to(self.embedding.dtype)
         if s.join is not None:
             self.join = Linear(compute_form(weights[s.join], device, dtype), role="join")
         for b in self.blocks:
@@ -144,14 +151,21 @@ class DecoderModel:
         visit(self.join)
         return total
 
-    def _embed(self, out: torch.Tensor, ctx) -> None:
+    def _embed(self, out: torch.Tensor, ctx, copy: torch.Tensor | None = None) -> None:
+        """The embedding's output; `copy`: float32 rows that receive it as well."""
         s = self.spec
+        if s.positions is not None:
+            ops.embed_positions(out, self.embedding, self.positions, ctx.tokens, ctx.token_pos, ctx.status,
+                                1.0 if s.embed_scale is None else s.embed_scale, copy)
+            return
         if s.bigram is None:
             ops.embed(out, self.embedding, ctx.tokens, ctx.status, s.embed_scale or 1.0)
         else:
             ops.embed_pairs(out, self.embedding, self.pairs, ctx.tokens, ctx.token_seq, ctx.token_pos, ctx.cu_seqlens, ctx.slot_ids,
                             ctx.cache.state, self.pair_state_offset, 1.0 if s.embed_scale is None else s.embed_scale, s.bigram.mul_prev,
                             s.bigram.mul_cur, ctx.status)
+        if copy is not None:
+            ops.place_rows(copy, out)
 
     # -- one step -----------------------------------------------------------------
     def forward(self, ctx, want_rows: torch.Tensor | None, num_want: int) -> torch.Tensor:
@@ -159,9 +173,12 @@ class DecoderModel:
         of the token rows that `want_rows` names (int32, device)."""
         T = ctx.num_tokens
         streams = self.spec.residual_streams
+        again = None        # the embedding's output, for runs that add it once more
         if streams is None:
             residual = torch.empty((T, self.spec.hidden), dtype=torch.float32, device=ctx.device)
-            self._embed(residual, ctx)
+            if any(run.adds for run in self.spec.order):
+                again = torch.empty_like(residual)
+            self._embed(residual, ctx, again)
         else:
             residual = torch.empty((streams, T, self.spec.hidden), dtype=torch.float32, device=ctx.device)
             self._embed(residual[0], ctx)
@@ -177,10 +194,17 @@ class DecoderModel:
             if run.joins:
                 ops.place_rows(joined[:, :self.spec.hidden], residual)
                 self.join(joined, out=residual)
+            if ctx.add_ahead is not None:       # (the block in front did not add it)
+                ops.join_branches(residual, [(ctx.add_ahead, None)])
+                ctx.add_ahead = None
+            if i + 1 < len(order) and order[i + 1].adds:
+                ctx.add_ahead = again
+                if not getattr(self.blocks[run.layer], "takes_add_ahead", False):
+                    nxt = None                  # (it cannot prepare what the next block reads)
             ctx.next_first_norm = getattr(nxt, "first_norm", lambda: None)() if nxt is not None else None
             ctx.block_ahead = nxt
             self.blocks[run.layer].forward(residual, ctx, slots)
-        ctx.next_first_norm = ctx.prenormed = ctx.block_ahead = None
+        ctx.next_first_norm = ctx.prenormed = ctx.block_ahead = ctx.add_ahead = None
         if streams is not None:
             # the streams are added up (a read with weights of one and no norm); the final norm reads the sum
             total = torch.empty((T, self.spec.hidden), dtype=torch.float32, device=ctx.device)

@@ -27,10 +27,12 @@ class Run:
     plane of its own), and an entry may read the cache plane that an earlier entry
     wrote (`cache_from` = that entry's index in the order) instead of writing one.
     With `joins` the residual x becomes W [x; x0] before the layer runs, x0 being the
-    embedding's output and W the matrix that the spec's `join` names."""
+    embedding's output and W the matrix that the spec's `join` names; with `adds` it
+    becomes x + x0."""
     layer: int
     cache_from: int | None = None
     joins: bool = False
+    adds: bool = False
 
 
 @dataclass
@@ -54,12 +56,19 @@ class ModelSpec:
     residual_streams: int | None = None
     bigram: Bigram | None = None      # (None: the embedding's rows alone)
     join: str | None = None           # checkpoint name of the [hidden, 2 hidden] matrix of the runs that say `joins`
+    positions: str | None = None      # checkpoint name of a [max_positions, hidden] table: row p is added at position p (not scaled)
 
     def __post_init__(self):
         if not self.order:
             self.order = [Run(i) for i in range(len(self.layers))]
         if any(run.joins for run in self.order) and (self.join is None or self.residual_streams is not None):
             raise ValueError("a run that joins the residual with the embedding's output needs the matrix's name and one residual stream")
+        if any(run.adds for run in self.order) and (self.residual_streams is not None or self.order[0].adds):
+            raise ValueError("the embedding's output is added to a residual in one stream, behind the first run")
+        if any(run.adds and run.joins for run in self.order):
+            raise ValueError("a run either joins the residual with the embedding's output or adds it")
+        if self.positions is not None and (self.max_positions is None or self.bigram is not None or self.residual_streams is not None):
+            raise ValueError("a table of positions comes with its length, without a table of pairs and with one residual stream")
         for i, run in enumerate(self.order):
             if not (0 <= run.layer < len(self.layers)):
                 raise ValueError(f"order[{i}] names layer {run.layer}, the model has {len(self.layers)}")

@@ -8,12 +8,14 @@ import torch
 from . import ops
 
 
-def try_matmul(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, epilogue: int, row_scale: tuple | None = None) -> bool:
+def try_matmul(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, epilogue: int, row_scale: tuple | None = None, glu=None,
+               glu_bias: torch.Tensor | None = None) -> bool:
     """bfloat16 operands with 16-byte aligned rows go to the tcgen05 kernel; anything else is refused.  `row_scale`: see
-    ops.gemm_tc (the activations are a norm's input times its gain; the row scale is applied to the sums)."""
+    ops.gemm_tc (the activations are a norm's input times its gain; the row scale is applied to the sums), and so `glu` and
+    `glu_bias` (the rule of the gated epilogue)."""
     if not ops.gemm_tc_supported(out, x, w, epilogue):
         return False
-    ops.gemm_tc(out, x, w, epilogue, ops.device_status(out.device), row_scale=row_scale, checked=True)
+    ops.gemm_tc(out, x, w, epilogue, ops.device_status(out.device), row_scale=row_scale, checked=True, glu=glu, glu_bias=glu_bias)
     return True
 
 

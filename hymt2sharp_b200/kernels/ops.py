@@ -194,6 +194,22 @@ def embed(out: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, status: tor
                               c_int(H), c_int(table.shape[0]), c_float(scale), _ptr(status), _stream()), "embed")
 
 
+def embed_positions(out: torch.Tensor, table: torch.Tensor, positions: torch.Tensor, ids: torch.Tensor, token_pos: torch.Tensor,
+                    status: torch.Tensor, scale: float = 1.0, copy: torch.Tensor | None = None) -> None:
+    """out[t] = float32(table[ids[t]]) * scale + positions[token_pos[t]]; out is [T, hidden] float32, and so is `copy`, which
+    receives the same rows."""
+    _need(out, "out", torch.float32, 2); _need(table, "table", None, 2); _need(positions, "positions", table.dtype, 2)
+    _need(ids, "ids", torch.int32, 1); _need(token_pos, "token_pos", torch.int32, 1)
+    T, H = out.shape
+    if copy is not None:
+        _need(copy, "copy", torch.float32, 2)
+    if table.shape[1] != H or positions.shape[1] != H or ids.shape[0] < T or token_pos.shape[0] < T or (copy is not None and copy.shape != out.shape):
+        raise KernelError(f"embed_positions: shapes out {tuple(out.shape)} table {tuple(table.shape)} positions {tuple(positions.shape)}")
+    _check(_lib().hymt2_embed_positions(_ptr(out), _ptr(copy), _ptr(table), _ptr(positions), c_int(dtype_code(table.dtype)), _ptr(ids), _ptr(token_pos),
+                                        c_int(T), c_int(H), c_int(table.shape[0]), c_int(positions.shape[0]), c_float(scale), _ptr(status),
+                                        _stream()), "embed_positions")
+
+
 def embed_pairs(out: torch.Tensor, table: torch.Tensor, pairs: torch.Tensor, ids: torch.Tensor, token_seq: torch.Tensor, token_pos: torch.Tensor,
                 cu_seqlens: torch.Tensor, slot_ids: torch.Tensor, state: torch.Tensor, state_offset: int, scale: float, mul_prev: int,
                 mul_cur: int, status: torch.Tensor) -> None:
@@ -285,7 +301,33 @@ def silu_mul(out: torch.Tensor, gate_up: torch.Tensor) -> None:
                                  _stream()), "silu_mul")
 
 
-def gemm_simt(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, epilogue: int = EPILOGUE_STORE) -> None:
+@dataclass(frozen=True)
+class GluRule:
+    """What the gated epilogue (EPILOGUE_SWIGLU) makes of a gate entry g and an up entry u: kind "silu": g sigmoid(g) u; "clamped":
+    with g = min(g, limit) and u = clamp(u, -limit, limit), g sigmoid(alpha g) (u + 1)."""
+    kind: str = "silu"
+    limit: float = 0.0
+    alpha: float = 1.0
+
+
+GLU_KINDS = {"silu": 0, "clamped": 1}
+GLU_SILU = GluRule()
+
+
+def _glu_arguments(glu: GluRule | None, bias: torch.Tensor | None, n: int, epilogue: int, with_bias: bool = True) -> tuple:
+    glu = glu or GLU_SILU
+    if bias is not None:
+        _f32(bias, "glu bias", 2 * n)
+    if epilogue != EPILOGUE_SWIGLU and (glu is not GLU_SILU or bias is not None):
+        raise KernelError("a gate's rule or bias belongs to the gated epilogue")
+    if glu.kind not in GLU_KINDS or (glu.kind == "clamped" and not glu.limit > 0):
+        raise KernelError(f"gated epilogue '{glu.kind}' with a limit of {glu.limit} (known: {', '.join(GLU_KINDS)}; a limit is positive)")
+    args = (c_int(GLU_KINDS[glu.kind]), c_float(glu.limit), c_float(glu.alpha))
+    return (*args, _ptr(bias)) if with_bias else args
+
+
+def gemm_simt(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, epilogue: int = EPILOGUE_STORE, glu: GluRule | None = None,
+              glu_bias: torch.Tensor | None = None) -> None:
     """out[M, N] = epilogue(a[M, K] @ w[N, K]^T) on CUDA cores, float32 accumulation in K order.
     With EPILOGUE_SWIGLU w has 2N rows (gate rows, then up rows)."""
     for t, n in ((out, "out"), (a, "a"), (w, "w")):
@@ -299,7 +341,7 @@ def gemm_simt(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, epilogue: int
     _check(_lib().hymt2_gemm_simt(_ptr(out), c_int(dtype_code(out.dtype)), _ptr(a), c_int(dtype_code(a.dtype)),
                                   _ptr(w), c_int(dtype_code(w.dtype)), c_int(M), c_int(N), c_int(K),
                                   c_long(a.stride(0)), c_long(w.stride(0)), c_long(out.stride(0)),
-                                  c_int(epilogue), _stream()), "gemm_simt")
+                                  c_int(epilogue), *_glu_arguments(glu, glu_bias, N, epilogue), _stream()), "gemm_simt")
 
 
 _status: dict = {}
@@ -309,7 +351,7 @@ _status_of: dict = {}   # the same by what callers pass (a torch.device with an 
 def device_status(device) -> torch.Tensor:
     """The int32[4] status word of a device: kernels set [0] when a device-side check fails or a
     bounded wait gives up (1: token id outside the table; 2: a sequence longer than the split attention was given
-    room for; 101-106: a wait of the tensor-core GEMM (106: for the partial sums of a tile's other CTAs); 108-119: of the prompt attention; 120-129: of the decode
+    room for; 3: a position outside the table of positions; 101-106: a wait of the tensor-core GEMM (106: for the partial sums of a tile's other CTAs); 108-119: of the prompt attention; 120-129: of the decode
     attention)."""
     hit = _status_of.get(device)
     if hit is not None:
@@ -387,9 +429,11 @@ def _plan_scratch(T: int, N: int, K: int, epilogue: int) -> tuple:
 
 
 def gemm_tc(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, epilogue: int, status: torch.Tensor,
-            row_scale: tuple | None = None, norm_after: tuple | None = None, checked: bool = False) -> None:
+            row_scale: tuple | None = None, norm_after: tuple | None = None, checked: bool = False, glu: GluRule | None = None,
+            glu_bias: torch.Tensor | None = None) -> None:
     """out[T, N] = epilogue(a[T, K] @ w[N, K]^T) on the tcgen05 tensor cores (bfloat16 operands,
-    float32 accumulation in tensor memory).  With EPILOGUE_SWIGLU w has 2N rows.
+    float32 accumulation in tensor memory).  With EPILOGUE_SWIGLU w has 2N rows; `glu` names another rule than silu(gate) * up,
+    `glu_bias` [2N] float32 is added to the gate's and up's sums first.
 
     An RMSNorm can be folded into the products around it.  `row_scale` = (ss [T, tiles] float32, width, eps): `a` holds
     bf16(x * gain) and the sums are multiplied by 1 / sqrt(sum(ss[t]) / width + eps) (store and SwiGLU epilogues).
@@ -425,7 +469,8 @@ def gemm_tc(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, epilogue: int, 
                                      _ptr(ws), c_long(ws.numel() if ws is not None else 0), _ptr(cnt),
                                      c_int(cnt.numel() if cnt is not None else 0), _ptr(status), _stream(),
                                      _ptr(ss_in), c_int(tiles_in), c_int(width), c_float(eps), _ptr(normed), _ptr(gain),
-                                     c_int(dtype_code(gain.dtype) if gain is not None else F32), _ptr(ss_out)), "gemm_tc")
+                                     c_int(dtype_code(gain.dtype) if gain is not None else F32), _ptr(ss_out),
+                                     *_glu_arguments(glu, glu_bias, N, epilogue)), "gemm_tc")
 
 
 def gemm_tc_debug(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, epilogue: int, status: torch.Tensor,
@@ -963,13 +1008,15 @@ def gemm_simt_batched(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, batch
 def latent_prep(proj: torch.Tensor, q_cols: int, q_out: torch.Tensor | None, cache_plane: torch.Tensor | None, block_table: torch.Tensor,
                 block_tokens: int, token_seq: torch.Tensor, token_pos: torch.Tensor, slot_ids: torch.Tensor, gain: torch.Tensor,
                 inv_freq: torch.Tensor | None, rot_dims: int, amplitude: float, eps: float, heads: int, dim: int, rot: int,
-                rank: int, rows_out: torch.Tensor | None = None) -> None:
+                rank: int, rows_out: torch.Tensor | None = None, q_latent: tuple | None = None) -> None:
     """From a token's fused projection [heads * (dim + rot) query entries | rank latent entries | rot shared key entries]:
     the normed latent vector and the rotated shared key part go to the token's cache row [rank + rot]; every head's
     rotated query part goes to q_out[t, h, rank : rank + rot].  Pairs (2i, 2i+1) turn by position * inv_freq[i], cosine
     and sine times `amplitude`.  cache_plane None: nothing is cached.  q_out None: the rotated query parts are written
     back into proj, in place.  rows_out [T, rank + rot]: the cache rows once more, side by side for all tokens.  With neither a
-    cache plane nor rows_out the projection need not hold a compressed row at all (only the queries are read)."""
+    cache plane nor rows_out the projection need not hold a compressed row at all (only the queries are read).
+    q_latent = (gain [q_rank] float32, out [T, q_rank]): the projection starts with a compressed query of q_rank = q_cols entries in
+    place of the heads' queries (heads is then 0): out = its RMS norm with the gain."""
     ldp = _rows_view(proj, "proj")
     T = proj.shape[0]
     dl = rank + rot
@@ -979,7 +1026,7 @@ def latent_prep(proj: torch.Tensor, q_cols: int, q_out: torch.Tensor | None, cac
         _need(rows_out, "rows_out", proj.dtype, 2)
     # a run without a compressed row of its own (it reads another run's cache) brings the queries alone
     rowless = cache_plane is None and rows_out is None
-    if proj.shape[1] < q_cols + (0 if rowless else dl) or q_cols != heads * (dim + rot) or (q_out is not None and q_out.shape != (T, heads * dl)) \
+    if proj.shape[1] < q_cols + (0 if rowless else dl) or (q_latent is None and q_cols != heads * (dim + rot)) or (q_out is not None and q_out.shape != (T, heads * dl)) \
             or (rows_out is not None and rows_out.shape != (T, dl)):
         raise KernelError(f"latent_prep: shapes proj {tuple(proj.shape)} do not fit {heads} heads of {dim} + {rot} and a row of {dl}")
     if cache_plane is not None:
@@ -990,9 +1037,16 @@ def latent_prep(proj: torch.Tensor, q_cols: int, q_out: torch.Tensor | None, cac
     for t, n in ((token_seq, "token_seq"), (token_pos, "token_pos"), (slot_ids, "slot_ids")):
         _need(t, n, torch.int32, 1)
     _f32(gain, "gain", rank); _f32(inv_freq, "inv_freq", rot_dims // 2)
+    q_gain = cq = None
+    if q_latent is not None:
+        q_gain, cq = q_latent
+        _f32(q_gain, "q_gain", q_cols); _need(cq, "cq", proj.dtype, 2)
+        if heads or cq.shape != (T, q_cols) or proj.shape[1] < q_cols:
+            raise KernelError(f"latent_prep: a compressed query {tuple(cq.shape)} out of {q_cols} columns")
     _check(_lib().hymt2_latent_prep(_ptr(proj), c_long(ldp), c_int(q_cols), _ptr(q_out), _ptr(rows_out), _ptr(cache_plane), c_int(dtype_code(proj.dtype)),
                                     _ptr(block_table), c_int(block_table.stride(0)), c_int(block_tokens), _ptr(token_seq),
-                                    _ptr(token_pos), _ptr(slot_ids), _ptr(gain), _ptr(inv_freq), c_int(rot_dims), c_float(amplitude),
+                                    _ptr(token_pos), _ptr(slot_ids), _ptr(gain), _ptr(q_gain), _ptr(cq),
+                                    c_int(q_cols if cq is not None else 0), _ptr(inv_freq), c_int(rot_dims), c_float(amplitude),
                                     c_float(eps), c_int(T), c_int(heads), c_int(dim), c_int(rot), c_int(rank), _stream()), "latent_prep")
 
 
@@ -1000,12 +1054,14 @@ def attention_shared_vector(out: torch.Tensor, q: torch.Tensor, cache_plane: tor
                             cu_seqlens: torch.Tensor, slot_ids: torch.Tensor, kv_lens: torch.Tensor, batch: int,
                             max_new_tokens: int, nh: int, d: int, dv: int, scale: float, window: int = 0, split_keys: int = 0,
                             max_splits: int = 0, part_acc: torch.Tensor | None = None, part_ml: torch.Tensor | None = None,
-                            status: torch.Tensor | None = None) -> None:
+                            status: torch.Tensor | None = None, sink: torch.Tensor | None = None) -> None:
     """Causal attention of the new tokens over a cache of ONE vector [d] per token that all heads share: it is every
     head's key, and its first dv entries are every head's value.  q [T, nh * d], out [T, nh * dv]; CUDA cores, float32
-    scores and softmax.  Splits as attention_simt (the partials are [T, nh, splits, dv])."""
+    scores and softmax.  Splits as attention_simt (the partials are [T, nh, splits, dv]).  `sink` [nh] float32: a head's softmax
+    has one more term of that score (not scaled, without a value) in its denominator."""
     if status is None:
         status = device_status(out.device)
+    _f32(sink, "sink", nh)
     _need(out, "out", None, 2); _need(q, "q", out.dtype, 2); _need(cache_plane, "cache_plane", out.dtype, 4)
     T = out.shape[0]
     if out.shape[1] != nh * dv or q.shape[1] != nh * d or q.shape[0] < T or cache_plane.shape[1] != 1 or cache_plane.shape[3] != d:
@@ -1020,7 +1076,7 @@ def attention_shared_vector(out: torch.Tensor, q: torch.Tensor, cache_plane: tor
     _check(_lib().hymt2_attention_shared_vector(_ptr(out), _ptr(q), _ptr(cache_plane), c_int(dtype_code(out.dtype)), _ptr(block_table),
                                                 c_int(block_table.stride(0)), c_int(cache_plane.shape[2]), _ptr(cu_seqlens),
                                                 _ptr(slot_ids), _ptr(kv_lens), c_int(batch), c_int(T), c_int(max_new_tokens),
-                                                c_int(nh), c_int(d), c_int(dv), c_float(scale), c_int(window), c_int(split_keys),
+                                                c_int(nh), c_int(d), c_int(dv), c_float(scale), c_int(window), _ptr(sink), c_int(split_keys),
                                                 c_int(max_splits), _ptr(part_acc), _ptr(part_ml), _stream(), _ptr(status)),
            "attention_shared_vector", 2 if split_keys > 0 else 1)
 
@@ -1043,11 +1099,12 @@ def latent_attention_mma(out: torch.Tensor, q: torch.Tensor, cache_plane: torch.
                          cu_seqlens: torch.Tensor, slot_ids: torch.Tensor, kv_lens: torch.Tensor, batch: int, max_new_tokens: int,
                          nh: int, d: int, dv: int, scale: float, window: int = 0, split_keys: int = 0, max_splits: int = 0,
                          part_acc: torch.Tensor | None = None, part_ml: torch.Tensor | None = None,
-                         status: torch.Tensor | None = None) -> None:
+                         status: torch.Tensor | None = None, sink: torch.Tensor | None = None) -> None:
     """attention_shared_vector in bfloat16 on the tensor cores (16x16x16 fragments, float32 sums and softmax): the same
     arguments and the same partials when split."""
     if status is None:
         status = device_status(out.device)
+    _f32(sink, "sink", nh)
     _need(out, "out", torch.bfloat16, 2); _need(q, "q", torch.bfloat16, 2); _need(cache_plane, "cache_plane", torch.bfloat16, 4)
     T = out.shape[0]
     if out.shape[1] != nh * dv or q.shape != (T, nh * d) or cache_plane.shape[1] != 1 or cache_plane.shape[3] != d:
@@ -1062,7 +1119,7 @@ def latent_attention_mma(out: torch.Tensor, q: torch.Tensor, cache_plane: torch.
     _check(_lib().hymt2_latent_attention_mma(_ptr(out), _ptr(q), _ptr(cache_plane), _ptr(block_table), c_int(block_table.stride(0)),
                                              c_int(cache_plane.shape[2]), _ptr(cu_seqlens), _ptr(slot_ids), _ptr(kv_lens), c_int(batch),
                                              c_int(T), c_int(max_new_tokens), c_int(nh), c_int(d), c_int(dv), c_float(scale),
-                                             c_int(window), c_int(split_keys), c_int(max_splits), _ptr(part_acc), _ptr(part_ml),
+                                             c_int(window), _ptr(sink), c_int(split_keys), c_int(max_splits), _ptr(part_acc), _ptr(part_ml),
                                              _ptr(status), _stream()), "latent_attention_mma", 2 if split_keys > 0 else 1)
 
 
@@ -1095,11 +1152,13 @@ def latent_attention_expanded_supported(dtype: torch.dtype, dim: int, rot: int, 
 
 def latent_attention_expanded(out: torch.Tensor, q: torch.Tensor, kexp: torch.Tensor, vexp: torch.Tensor, krot: torch.Tensor,
                               cu_seqlens: torch.Tensor, slot_ids: torch.Tensor, kv_lens: torch.Tensor, batch: int,
-                              max_new_tokens: int, nh: int, dim: int, rot: int, dv: int, scale: float, window: int = 0) -> None:
+                              max_new_tokens: int, nh: int, dim: int, rot: int, dv: int, scale: float, window: int = 0,
+                              sink: torch.Tensor | None = None) -> None:
     """Causal attention of whole prompts that start at position 0, bfloat16 on the tensor cores, with keys and values per
     head: q [T, >= nh * (dim + rot)] (head h at column h * (dim + rot), its last rot entries rotated), kexp [T, nh * dim],
     vexp [T, nh * dv], krot [T, rot] the rotated key part of all heads; out [T, nh * dv].  All may be columns of wider
-    matrices."""
+    matrices.  `sink` as attention_shared_vector."""
+    _f32(sink, "sink", nh)
     T = out.shape[0]
     for t, n in ((out, "out"), (q, "q"), (kexp, "kexp"), (vexp, "vexp"), (krot, "krot")):
         _rows_view(t, n, torch.bfloat16)
@@ -1113,7 +1172,7 @@ def latent_attention_expanded(out: torch.Tensor, q: torch.Tensor, kexp: torch.Te
                                                   c_long(kexp.stride(0)), _ptr(vexp), c_long(vexp.stride(0)), _ptr(krot),
                                                   c_long(krot.stride(0)), _ptr(cu_seqlens), _ptr(slot_ids), _ptr(kv_lens), c_int(batch),
                                                   c_int(max_new_tokens), c_int(nh), c_int(dim), c_int(rot), c_int(dv), c_float(scale),
-                                                  c_int(window), _stream()), "latent_attention_expanded")
+                                                  c_int(window), _ptr(sink), _stream()), "latent_attention_expanded")
 
 
 
@@ -1357,12 +1416,15 @@ SCORES = {"softmax": 0, "sigmoid": 1}
 class RouteRule:
     """How a router's outputs become scores, and scores a choice: `scores` "softmax" (over all outputs) or "sigmoid" (of each);
     `renormalise`: the chosen scores are divided by their sum + share_eps; with groups > 1 only the outputs of the `keep`
-    groups (equal ones, of neighbours) whose two largest scores have the largest sums can be chosen."""
+    groups (equal ones, of neighbours) whose two largest choice scores have the largest sums (`group_best` 1: whose largest is the
+    largest) can be chosen; the weights are multiplied by `weight_scale` at the end."""
     scores: str = "softmax"
     renormalise: bool = False
     share_eps: float = 0.0
     groups: int = 1
     keep: int = 1
+    group_best: int = 2
+    weight_scale: float = 1.0
 
 
 def _rule_arguments(what: str, logits, correction, bias, rule: RouteRule, outputs: int | None, chosen, weight):
@@ -1376,7 +1438,7 @@ def _rule_arguments(what: str, logits, correction, bias, rule: RouteRule, output
     if rule.scores not in SCORES:
         raise KernelError(f"{what}: scores '{rule.scores}' are not known (known: {', '.join(SCORES)})")
     return T, R, top, (c_long(ldz), _ptr(correction), _ptr(bias), c_int(SCORES[rule.scores]), c_int(1 if rule.renormalise else 0),
-                       c_float(rule.share_eps), c_int(rule.groups), c_int(rule.keep))
+                       c_float(rule.share_eps), c_int(rule.groups), c_int(rule.keep), c_int(rule.group_best), c_float(rule.weight_scale))
 
 
 def moe_route(chosen: torch.Tensor, weight: torch.Tensor, logits: torch.Tensor, correction: torch.Tensor | None,
@@ -1424,17 +1486,18 @@ def gemm_group_tile(kernel: str = "simt") -> int:
 
 
 def gemm_grouped(kernel: str, out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, row_token: torch.Tensor,
-                 gather: bool, epilogue: int = EPILOGUE_STORE) -> None:
+                 gather: bool, epilogue: int = EPILOGUE_STORE, glu: GluRule | None = None) -> None:
     """out[r] = epilogue(a[source(r)] @ w[tile_group[r // tile]]^T) for the sorted rows r of moe_place: w [experts, N, K];
     source(r) = row_token[r] with `gather` (a holds one row per token), r itself otherwise (a holds sorted rows); padding
     rows and unused tiles are skipped ("tc": computed and never read).  Epilogues: EPILOGUE_STORE, EPILOGUE_RELU_SQUARED, and for "skinny"
-    and "tc" EPILOGUE_SWIGLU (w [experts, 2N, K] holds an expert's N gate rows, then its N up rows; out = silu(gate) * up).
+    and "tc" EPILOGUE_SWIGLU (w [experts, 2N, K] holds an expert's N gate rows, then its N up rows; out = silu(gate) * up, or what `glu` says).
     kernel "simt": CUDA cores, any sizes and types; "skinny": CUDA cores, tiles of 8 rows, a and w of one type, the time of
     reading the weights once; "tc": tcgen05, bfloat16, no gather (see moe_gather), K and N multiples of 8."""
     _need(out, "out", None, 2); _need(a, "a", None, 2); _need(w, "w", None, 3)
     _need(tile_group, "tile_group", torch.int32, 1); _need(row_token, "row_token", torch.int32, 1)
     tiles, tile = tile_group.numel() - 1, gemm_group_tile(kernel)
     gated = epilogue == EPILOGUE_SWIGLU
+    rule = _glu_arguments(glu, None, 0, epilogue, with_bias=False)
     N, K = w.shape[1] // (2 if gated else 1), w.shape[2]
     if gated and (w.shape[1] % 2 or kernel == "simt" or (kernel == "tc" and out.dtype != torch.bfloat16)):
         raise KernelError(f"gemm_grouped: gated experts are not taken by '{kernel}' with w {tuple(w.shape)} and out {out.dtype}")
@@ -1450,14 +1513,14 @@ def gemm_grouped(kernel: str, out: torch.Tensor, a: torch.Tensor, w: torch.Tenso
             raise KernelError("gemm_grouped: the kernel for few rows wants a and w of one type")
         _check(_lib().hymt2_gemm_skinny_grouped(_ptr(out), c_int(dtype_code(out.dtype)), _ptr(a), _ptr(w), c_int(dtype_code(w.dtype)),
                                                 _ptr(tile_group), _ptr(row_token), c_int(1 if gather else 0), c_int(tiles), c_int(N), c_int(K),
-                                                c_long(a.stride(0)), c_long(out.stride(0)), c_long(w.shape[1] * K), c_int(epilogue), _stream()),
+                                                c_long(a.stride(0)), c_long(out.stride(0)), c_long(w.shape[1] * K), c_int(epilogue), *rule, _stream()),
                "gemm_skinny_grouped")
     else:
         if gather or a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
             raise KernelError("gemm_grouped: the tensor-core kernel wants sorted bfloat16 rows")
         _check(_lib().hymt2_gemm_tc_grouped(_ptr(out), c_int(dtype_code(out.dtype)), _ptr(a), _ptr(w), _ptr(tile_group), c_int(tiles),
                                             c_int(w.shape[0]), c_int(N), c_int(K), c_long(a.stride(0)), c_long(out.stride(0)),
-                                            c_int(2 if gated else 1 if epilogue == EPILOGUE_RELU_SQUARED else 0), _ptr(device_status(out.device)), _stream()),
+                                            c_int(2 if gated else 1 if epilogue == EPILOGUE_RELU_SQUARED else 0), *rule, _ptr(device_status(out.device)), _stream()),
                "gemm_tc_grouped")
 
 
@@ -1576,23 +1639,26 @@ def moe_combine_norm(residual: torch.Tensor, rows: torch.Tensor | None, branch: 
            "moe_combine_norm")
 
 
-JOIN_MAX_TOP = 32
+JOIN_MAX_TOP, JOIN_MAX_BRANCHES = 32, 3
 
 
 def join_branches(x: torch.Tensor, branches: list, mixture: tuple | None = None, norm: tuple | None = None) -> torch.Tensor | None:
-    """x (float32 [T, W]) += sum over `branches` (at most two (y, gain) pairs, float32 [T, W] and [W]) of gain * y, plus, with `mixture`
-    = (y, pair_row, weight, gain, shared, z): gain * (sum_k weight[t, k] * y[pair_row[t, k]] + sigmoid(z[t]) * shared[t]), shared
-    float32 [T, W] or None, z a float32 column [T, 1] or None (factor 1).  `norm` = (gain, eps, out): out = the RMS norm of the new
-    rows, which is also returned.  One kernel, one block a token."""
+    """x (float32 [T, W]) += sum over `branches` (at most JOIN_MAX_BRANCHES of (y, gain) or (y, gain, bias), float32 [T, W] and [W], gain and
+    bias None where there is none) of gain * (y + bias), plus, with `mixture` = (y, pair_row, weight, gain, shared, z): gain * (sum_k
+    weight[t, k] * y[pair_row[t, k]] + sigmoid(z[t]) * shared[t]), gain [W] or None, shared float32 [T, W] or None, z a float32 column
+    [T, 1] or None (factor 1).  `norm` = (gain, eps, out): out = the RMS norm of the new rows, which is also returned.  One kernel,
+    one block a token."""
     _need(x, "x", torch.float32, 2)
     T, W = x.shape
-    if len(branches) > 2:
-        raise KernelError("join_branches: at most two plain branches")
-    for y, g in branches:
-        _need(y, "branch", torch.float32, 2); _f32(g, "gain", W)
-        if y.shape != x.shape or g is None:
+    n = len(branches)
+    if n > JOIN_MAX_BRANCHES:
+        raise KernelError(f"join_branches: {n} plain branches (at most {JOIN_MAX_BRANCHES})")
+    branches = [(b[0], b[1], b[2] if len(b) > 2 else None) for b in branches]
+    for y, g, b in branches:
+        _need(y, "branch", torch.float32, 2); _f32(g, "gain", W); _f32(b, "bias", W)
+        if y.shape != x.shape:
             raise KernelError(f"join_branches: a branch of {tuple(y.shape)} for rows {tuple(x.shape)}")
-    pad = list(branches) + [(None, None)] * (2 - len(branches))
+    columns = [(c_void_p * max(n, 1))(*[b[k].data_ptr() if b[k] is not None else None for b in branches]) for k in range(3)]
     y = pair_row = weight = gain = shared = z = h = ngain = None
     top, ldz, eps = 0, 0, 0.0
     if mixture is not None:
@@ -1600,7 +1666,7 @@ def join_branches(x: torch.Tensor, branches: list, mixture: tuple | None = None,
         _need(y, "routed", torch.float32, 2); _need(pair_row, "pair_row", torch.int32, 2); _need(weight, "weight", torch.float32, 2)
         _f32(gain, "gain", W)
         top = pair_row.shape[1]
-        if y.shape[1] != W or pair_row.shape[0] != T or weight.shape != pair_row.shape or gain is None or top > JOIN_MAX_TOP:
+        if y.shape[1] != W or pair_row.shape[0] != T or weight.shape != pair_row.shape or top > JOIN_MAX_TOP:
             raise KernelError(f"join_branches: routed rows {tuple(y.shape)}, pairs {tuple(pair_row.shape)} for rows {tuple(x.shape)}")
         if shared is not None:
             _need(shared, "shared", torch.float32, 2)
@@ -1615,9 +1681,8 @@ def join_branches(x: torch.Tensor, branches: list, mixture: tuple | None = None,
         _need(ngain, "norm gain", None, 1); _need(h, "normed rows", None, 2)
         if ngain.shape[0] != W or h.shape != x.shape:
             raise KernelError("join_branches: the norm does not fit the rows")
-    _check(_lib().hymt2_join_branches(_ptr(x), _ptr(pad[0][0]), _ptr(pad[0][1]), _ptr(pad[1][0]), _ptr(pad[1][1]), _ptr(y), _ptr(pair_row),
-                                      _ptr(weight), c_int(top), _ptr(gain), _ptr(shared), _ptr(z), c_long(ldz), _ptr(h),
-                                      c_int(dtype_code(h.dtype) if h is not None else F32), _ptr(ngain),
+    _check(_lib().hymt2_join_branches(_ptr(x), *columns, c_int(n), _ptr(y), _ptr(pair_row), _ptr(weight), c_int(top), _ptr(gain), _ptr(shared),
+                                      _ptr(z), c_long(ldz), _ptr(h), c_int(dtype_code(h.dtype) if h is not None else F32), _ptr(ngain),
                                       c_int(dtype_code(ngain.dtype) if ngain is not None else F32), c_float(eps), c_int(T), c_int(W), _stream()),
            "join_branches")
     return h

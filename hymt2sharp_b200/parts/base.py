@@ -165,6 +165,9 @@ class StepContext:
     prenormed: object = None
     # the block that runs next (None behind the last one), for a block whose last kernel can prepare that block's input
     block_ahead: object = None
+    # float32 rows [T, hidden] that are to be added to the residual behind the running block; a block with `takes_add_ahead`
+    # may do it in its own last kernel (before it prepares the next block's input) and then sets this to None
+    add_ahead: torch.Tensor | None = None
 
     @property
     def decode(self) -> bool:

@@ -226,14 +226,19 @@ class ParallelBlock:
 
         h = norm(x);   x <- x + gain_m * mixer(h) + gain_f * ff(h)          (no feed-forward: the last term is absent)
 
-    gain_m and gain_f are stored vectors of the model's width (`mixer_gain`, `ff_gain`: their names), applied entry by entry in
-    float32.  The sublayers store into float32 buffers of their own; one kernel adds them to the residual, a mixture of
+    gain_m and gain_f are stored vectors of the model's width (`mixer_gain`, `ff_gain`: their names; None: the sublayer's output as it
+    is), applied entry by entry in float32.  The sublayers store into float32 buffers of their own; one kernel adds them to the residual, a mixture of
     experts from its experts' rows (a feed-forward that offers `pieces`), and norms the new rows for the block that runs next
-    when that is a parallel block too (`ctx.block_ahead`); those rows wait in `ctx.shared["parallel_rows"]`."""
+    when that is a parallel block too (`ctx.block_ahead`); those rows wait in `ctx.shared["parallel_rows"]`.
+    The same kernel adds a feed-forward's output bias (a part with `output_bias` that takes `bias_later`) and rows that the model
+    wants added behind this block (`ctx.add_ahead`, see engine.model)."""
 
-    def __init__(self, norm: PartSpec, mixer: PartSpec, mixer_gain: str, feed_forward: PartSpec | None = None, ff_gain: str | None = None):
-        if (feed_forward is None) != (ff_gain is None):
-            raise ValueError("a feed-forward comes with the name of its gain")
+    takes_add_ahead = True
+
+    def __init__(self, norm: PartSpec, mixer: PartSpec, mixer_gain: str | None = None, feed_forward: PartSpec | None = None,
+                 ff_gain: str | None = None):
+        if feed_forward is None and ff_gain is not None:
+            raise ValueError("a gain of the feed-forward needs a feed-forward")
         self.norm = build_part("norm", norm)
         self.mixer = build_part("mixer", mixer)
         self.feed_forward = build_part("feed_forward", feed_forward) if feed_forward is not None else None
@@ -272,14 +277,14 @@ class ParallelBlock:
         return None   # (its rows come from the sum at the end of the block in front, not from a product)
 
     @staticmethod
-    def _stored(part, h, like, ctx, *slot):
+    def _stored(part, h, like, ctx, *slot, **how):
         import torch
         y = torch.empty(like.shape, dtype=torch.float32, device=like.device)
         if getattr(part, "can_store", False):
-            part.forward(h, y, ctx, *slot, store=True)
+            part.forward(h, y, ctx, *slot, store=True, **how)
         else:
             y.zero_()
-            part.forward(h, y, ctx, *slot)
+            part.forward(h, y, ctx, *slot, **how)
         return y
 
     def forward(self, residual, ctx, slots) -> None:
@@ -299,7 +304,11 @@ class ParallelBlock:
                 y, pair_row, weight, shared, z = pieces
                 mixture = (y, pair_row, weight, self.gains[1], shared, z)
             else:
-                branches.append((self._stored(ff, h, residual, ctx), self.gains[1]))
+                bias = getattr(ff, "output_bias", None)
+                branches.append((self._stored(ff, h, residual, ctx, **({} if bias is None else {"bias_later": True})), self.gains[1], bias))
+        if ctx.add_ahead is not None:
+            branches.append((ctx.add_ahead, None))
+            ctx.add_ahead = None
         ctx.prenormed = None
         nxt = ctx.block_ahead
         if not isinstance(nxt, ParallelBlock) or getattr(nxt.norm, "groups", 0) != 1:

@@ -16,6 +16,9 @@ A prompt that starts at position 0 brings all of its keys along, and a head's ow
 times narrower than the compressed row: there the bfloat16 engine rebuilds every head's keys and values with one product
 over all tokens and runs the attention per head, which is the same sums in another order (EXPAND_FROM_TOKENS).
 
+`q_rank`: the queries come out of a latent vector of their own, q = W_q (gain * unit_rms(W_dq x)) (`dq_proj`, `dq_norm`; `q_proj` is then
+W_q [., q_rank]): its down-projection is the first rows of the fused projection, its norm runs with the compressed row's.
+`sink`: a stored score a head, one more term exp(sink_h) in the softmax's denominator, neither scaled nor with a value.
 `own_kv` False: the layer has no down-projection and no latent norm; it attends over the compressed rows that another run
 cached (the model's order names it), with its own up-projections, queries, window and gate.  `cache_window`: the positions that
 the cache keeps for this plane when that is more than the layer's own window (readers of one plane may look back differently
@@ -44,7 +47,8 @@ class LatentAttention:
     def __init__(self, hidden: int, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, scale: float, eps: float,
                  position: PartSpec | None, gate: str | None, q_proj: str, dkv_proj: str, dkv_norm: str, uk_proj: str,
                  uv_proj: str, o_proj: str, g_proj: str | None = None, window: int | None = None, own_kv: bool = True,
-                 cache_window: int | None = None):
+                 cache_window: int | None = None, q_rank: int | None = None, dq_proj: str | None = None, dq_norm: str | None = None,
+                 sink: str | None = None):
         if gate not in (None, "element", "head"):
             raise ValueError(f"output gate '{gate}': known are 'element' (one value per output entry), 'head' and None")
         if gate is not None and g_proj is None:
@@ -55,20 +59,29 @@ class LatentAttention:
         self.cache_window = self.window if cache_window is None else int(cache_window)
         if self.cache_window and (not self.window or self.cache_window < self.window):
             raise ValueError(f"a cache that keeps {self.cache_window} positions is too short for a window of {self.window or 'everything'}")
-        self.names = dict(q=q_proj, dkv=dkv_proj, cn=dkv_norm, uk=uk_proj, uv=uv_proj, o=o_proj, g=g_proj)
+        if (q_rank is None) != (dq_proj is None) or (q_rank is None) != (dq_norm is None):
+            raise ValueError("a latent vector of the queries comes with its width, its projection and its norm")
+        self.q_rank = None if q_rank is None else int(q_rank)
+        self.names = dict(q=q_proj, dkv=dkv_proj, cn=dkv_norm, uk=uk_proj, uv=uv_proj, o=o_proj, g=g_proj, dq=dq_proj, qn=dq_norm, s=sink)
         self.position = build_part("position", position) if position is not None else None
         self.q_cols = heads * (dim + rot_dim)
+        self.row_at = self.q_cols if q_rank is None else self.q_rank     # where the compressed row starts in the fused projection
         self.gate_cols = 0 if gate is None else (heads * vdim if gate == "element" else heads)
-        self.proj = self.out = self.uk_t = self.uv = self.c_gain = self.ukv = None
+        self.proj = self.out = self.uk_t = self.uv = self.c_gain = self.ukv = self.uq = self.q_gain = self.sink = None
 
     # -- what it needs ----------------------------------------------------------
     def tensors(self):
         n, H = self.names, self.heads
-        t = {n["q"]: TensorSpec((self.q_cols, self.hidden)), n["uk"]: TensorSpec((H * self.dim, self.rank)),
+        t = {n["q"]: TensorSpec((self.q_cols, self.hidden if self.q_rank is None else self.q_rank)), n["uk"]: TensorSpec((H * self.dim, self.rank)),
              n["uv"]: TensorSpec((H * self.vdim, self.rank)), n["o"]: TensorSpec((self.hidden, H * self.vdim))}
         if self.own_kv:
             t[n["dkv"]] = TensorSpec((self.rank + self.rot, self.hidden))
             t[n["cn"]] = TensorSpec((self.rank,), init="gain")
+        if self.q_rank is not None:
+            t[n["dq"]] = TensorSpec((self.q_rank, self.hidden))
+            t[n["qn"]] = TensorSpec((self.q_rank,), init="gain")
+        if n["s"] is not None:
+            t[n["s"]] = TensorSpec((H,))
         if self.gate is not None:
             t[n["g"]] = TensorSpec((self.gate_cols, self.hidden))
         if self.position is not None:
@@ -84,12 +97,17 @@ class LatentAttention:
 
     def load(self, weights, device, dtype):
         n, H = self.names, self.heads
-        rows = [weights[n["q"]]] + ([weights[n["dkv"]]] if self.own_kv else []) + ([weights[n["g"]]] if self.gate is not None else [])
+        rows = [weights[n["q" if self.q_rank is None else "dq"]]] + ([weights[n["dkv"]]] if self.own_kv else []) + ([weights[n["g"]]] if self.gate is not None else [])
         total = sum(r.shape[0] for r in rows)
         if total % 8:
             # rows of zeros, so that a token's projection is a whole number of 16-byte pieces and kernels may read it by them
             rows.append(torch.zeros((8 - total % 8, self.hidden), dtype=rows[0].dtype))
         self.proj = Linear(compute_form(torch.cat(rows, dim=0), device, dtype), role="q_dkv_gate")
+        if self.q_rank is not None:
+            self.uq = Linear(compute_form(weights[n["q"]], device, dtype), role="uq")
+            self.q_gain = weights[n["qn"]].to(device).float().contiguous()
+        if n["s"] is not None:
+            self.sink = weights[n["s"]].to(device).float().contiguous()
         self.out = Linear(compute_form(weights[n["o"]], device, dtype), ops.EPILOGUE_ACCUMULATE, role="o_proj")
         self.out_store = Linear(self.out.weight, ops.EPILOGUE_STORE, role="o_proj")
         # per head: W_uk[h]^T [kv_rank, dim] (the query goes into the compressed space) and W_uv[h] [vdim, kv_rank]
@@ -113,7 +131,7 @@ class LatentAttention:
         table = ctx.cache.tables[slot.group]
         if slot.writes != self.own_kv:
             raise ValueError("a latent attention without a down-projection reads another run's cache plane, and only such a one does")
-        proj = self.proj(x, ctx=ctx)                                   # [T, queries | latent row (if its own) | gate]
+        proj = self.proj(x, ctx=ctx)                                   # [T, queries or their latent vector | latent row (if its own) | gate]
         kept = ("latent_rows", slot.group, slot.plane)                 # a step's compressed rows side by side, for the plane's readers
         if (self.ukv is not None and not ctx.decode and ctx.max_new_tokens >= EXPAND_FROM_TOKENS and ctx.host_starts
                 and not any(ctx.host_starts) and (self.own_kv or kept in ctx.shared)):
@@ -121,13 +139,10 @@ class LatentAttention:
             self._gate_and_project(out, proj, residual, ctx, store)
             return
         q = torch.empty((T, H * dl), dtype=proj.dtype, device=proj.device)
-        ops.latent_prep(proj, self.q_cols, q, plane if slot.writes else None, table, ctx.cache.block_tokens, ctx.token_seq,
-                        ctx.token_pos, ctx.slot_ids, self.c_gain, rotary.inv_freq if rotary else None,
-                        rotary.rope_dim if rotary else 0, rotary.amplitude if rotary else 1.0, self.eps, H, self.dim,
-                        self.rot, self.rank)
+        source = self._prepare(proj, q, rotary, plane if slot.writes else None, table, ctx)
         # q[t, h, :kv_rank] = W_uk[h]^T q_h[:dim]
         ops.tag = "q_absorb"
-        matmul_batched(q, proj, self.uk_t, self.dim + self.rot, dl)
+        matmul_batched(q, source, self.uk_t, self.dim + self.rot, dl)
         ops.tag = None
         mixed = torch.empty((T, H * self.rank), dtype=q.dtype, device=q.device)
         self.attend(mixed, q, plane, table, ctx)
@@ -137,9 +152,24 @@ class LatentAttention:
         ops.tag = None
         self._gate_and_project(out, proj, residual, ctx, store)
 
+    def _prepare(self, proj, q_out, rotary, plane, table, ctx, rows_out=None) -> torch.Tensor:
+        """Norms, rotations and the cache rows of the step's tokens; returns the matrix whose first columns are the heads' queries.
+        Their rotated parts go to `q_out` (behind the places of the compressed entries) or, with None, stay in place."""
+        table_args = (table, ctx.cache.block_tokens, ctx.token_seq, ctx.token_pos, ctx.slot_ids, self.c_gain)
+        turn_args = (rotary.inv_freq if rotary else None, rotary.rope_dim if rotary else 0, rotary.amplitude if rotary else 1.0, self.eps)
+        if self.q_rank is None:
+            ops.latent_prep(proj, self.q_cols, q_out, plane, *table_args, *turn_args, self.heads, self.dim, self.rot, self.rank, rows_out=rows_out)
+            return proj
+        cq = torch.empty((proj.shape[0], self.q_rank), dtype=proj.dtype, device=proj.device)
+        ops.latent_prep(proj, self.q_rank, None, plane, *table_args, *turn_args, 0, self.dim, self.rot, self.rank, rows_out=rows_out,
+                        q_latent=(self.q_gain, cq))
+        q = self.uq(cq, ctx=ctx)
+        ops.latent_prep(q, self.q_cols, q_out, None, *table_args, *turn_args, self.heads, self.dim, self.rot, self.rank)
+        return q
+
     def _gate_and_project(self, out, proj, residual, ctx, store: bool) -> None:
         if self.gate is not None:
-            g0 = self.q_cols + (self.rank + self.rot if self.own_kv else 0)
+            g0 = self.row_at + (self.rank + self.rot if self.own_kv else 0)
             ops.sigmoid_gate(out, proj[:, g0:g0 + self.gate_cols], self.heads, self.vdim, self.gate == "head")
         if store:
             self.out_store(out, out=residual)
@@ -156,15 +186,12 @@ class LatentAttention:
             ctx.shared[kept] = rows
         else:
             rows = ctx.shared[kept]
-        ops.latent_prep(proj, self.q_cols, None, plane, table, ctx.cache.block_tokens, ctx.token_seq, ctx.token_pos, ctx.slot_ids,
-                        self.c_gain, rotary.inv_freq if rotary else None, rotary.rope_dim if rotary else 0,
-                        rotary.amplitude if rotary else 1.0, self.eps, H, self.dim, self.rot, self.rank,
-                        rows_out=rows if self.own_kv else None)
+        q = self._prepare(proj, None, rotary, plane, table, ctx, rows_out=rows if self.own_kv else None)
         kv = self.ukv(rows[:, :self.rank], ctx=ctx)                    # [T, H * dim | H * vdim]
         out = torch.empty((T, H * self.vdim), dtype=proj.dtype, device=proj.device)
-        ops.latent_attention_expanded(out, proj[:, :self.q_cols], kv[:, :H * self.dim], kv[:, H * self.dim:], rows[:, self.rank:],
+        ops.latent_attention_expanded(out, q[:, :self.q_cols], kv[:, :H * self.dim], kv[:, H * self.dim:], rows[:, self.rank:],
                                       ctx.cu_seqlens, ctx.slot_ids, ctx.kv_lens, ctx.num_seqs, ctx.max_new_tokens, H, self.dim,
-                                      self.rot, self.vdim, self.scale, self.window)
+                                      self.rot, self.vdim, self.scale, self.window, self.sink)
         return out
 
     def attend(self, out, q, plane, table, ctx) -> None:
@@ -179,7 +206,7 @@ class LatentAttention:
             acc = torch.empty(ctx.num_tokens * self.heads * max_splits * self.rank, dtype=torch.float32, device=out.device)
             ml = torch.empty(ctx.num_tokens * self.heads * max_splits * 2, dtype=torch.float32, device=out.device)
         run(out, q, plane, table, ctx.cu_seqlens, ctx.slot_ids, ctx.kv_lens, ctx.num_seqs, ctx.max_new_tokens, self.heads,
-            self.rank + self.rot, self.rank, self.scale, self.window, split, max_splits, acc, ml)
+            self.rank + self.rot, self.rank, self.scale, self.window, split, max_splits, acc, ml, sink=self.sink)
 
 
 register_part("mixer", "latent_attention", LatentAttention)

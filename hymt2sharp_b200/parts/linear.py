@@ -23,10 +23,13 @@ fold_norms = True
 
 
 class Linear:
-    """y = epilogue(x @ W^T) with W [out, in]; for the SwiGLU epilogue W is [2*out, in]."""
+    """y = epilogue(x @ W^T) with W [out, in]; for the SwiGLU epilogue W is [2*out, in], and `glu` (ops.GluRule, None: silu(gate) * up)
+    and `glu_bias` (float32 [2*out] or None) say what becomes of a gate and an up entry."""
 
-    def __init__(self, weight: torch.Tensor, epilogue: int = ops.EPILOGUE_STORE, role: str | None = None):
+    def __init__(self, weight: torch.Tensor, epilogue: int = ops.EPILOGUE_STORE, role: str | None = None, glu: "ops.GluRule | None" = None,
+                 glu_bias: torch.Tensor | None = None):
         self.weight = weight
+        self.glu, self.glu_bias = glu, glu_bias
         self.epilogue = epilogue
         self.role = role   # what a profile books this product under
         rows = weight.shape[0]
@@ -41,10 +44,10 @@ class Linear:
         ops.tag = self.role
         try:
             if isinstance(x, Prenormed):
-                if self.epilogue != ops.EPILOGUE_ACCUMULATE and fast.try_matmul(out, x.normed, self.weight, self.epilogue, x.row_scale()):
+                if self.epilogue != ops.EPILOGUE_ACCUMULATE and fast.try_matmul(out, x.normed, self.weight, self.epilogue, x.row_scale(), self.glu, self.glu_bias):
                     return out
                 x = x.materialize(ctx)
-            matmul(out, x, self.weight, self.epilogue)
+            matmul(out, x, self.weight, self.epilogue, self.glu, self.glu_bias)
         finally:
             ops.tag = None
         return out
@@ -97,8 +100,8 @@ def matmul_batched(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, x_step: 
     ops.gemm_simt_batched(out, x, w, batch, x_step, out_step)
 
 
-def matmul(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, epilogue: int) -> None:
+def matmul(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, epilogue: int, glu=None, glu_bias: torch.Tensor | None = None) -> None:
     """Picks the kernel: tensor-core kernels where they take the shape and types, else CUDA cores."""
-    if fast.try_matmul(out, x, w, epilogue):
+    if fast.try_matmul(out, x, w, epilogue, None, glu, glu_bias):
         return
-    ops.gemm_simt(out, x, w, epilogue)
+    ops.gemm_simt(out, x, w, epilogue, glu, glu_bias)

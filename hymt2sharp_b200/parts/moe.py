@@ -8,12 +8,14 @@ the correction and not renormalised.  A shared expert (any feed-forward part) ru
 
 Chosen by parameters beyond that: a bias of the router (`router_bias`, a stored vector added to z); weights that are the
 softmax over the CHOSEN outputs only (`weights="chosen_softmax"`; the choice by score is then the choice by z); and gated
-experts, expert(x) = W_down (act(W_gate x) * (W_up x)) (`gate_proj` given; act "silu"): gate and up are one grouped product
-over the stacked matrices, whose epilogue applies SiLU and multiplies (the general CUDA-core kernel, and another activation:
+experts, expert(x) = W_down (act(W_gate x) * (W_up x)) (`gate_proj` given; act "silu", "gelu_tanh", or "clamped": with g = min(W_gate x, limit)
+and u = clamp(W_up x, -limit, limit), W_down (g * sigmoid(alpha * g) * (u + 1))): gate and up are one grouped product over the
+stacked matrices, whose epilogue applies the activation and multiplies (the general CUDA-core kernel, and "gelu_tanh":
 a small kernel behind it).  The scores may be the sigmoid of each output
 (`scores="sigmoid"`), the weights the chosen scores' shares of their sum (`weights="chosen_share"`, `share_eps` added to the
 sum), and the choice limited to groups: outputs side by side are cut into `groups` runs of equal length, the runs are ranked by
-what their two best scores add up to, and the choice is among the outputs of the first `keep` runs.  The shared expert may have a gate per token
+what their two best scores (with the correction) add up to, or by their best one (`group_best=1`), and the choice is among the outputs of
+the first `keep` runs.  `weight_scale` multiplies the weights at the end.  The shared expert may have a gate per token
 (`shared_gate`, a stored [1, hidden] matrix): its output is multiplied by sigmoid(W x); that product is one more row of the
 router's.
 
@@ -32,7 +34,7 @@ from .base import PartSpec, build_part, register_part
 from .linear import Linear, compute_form
 
 ACTIVATIONS = {"relu2": ops.EPILOGUE_RELU_SQUARED}      # experts without a gate: an epilogue of the grouped product
-GATED_ACTIVATIONS = {"silu": ops.GATED_SILU, "gelu_tanh": ops.GATED_GELU_TANH}
+GATED_ACTIVATIONS = {"silu": ops.GATED_SILU, "gelu_tanh": ops.GATED_GELU_TANH, "clamped": None}   # (None: a kernel of its own)
 WEIGHTS = ("scores", "chosen_softmax", "chosen_share")
 SKINNY_MAX_PAIRS = 512        # up to this many (token, choice) pairs in a step the kernel for few rows runs the experts,
 SKINNY_PAIRS_BESIDE_TC = 64   # where the tensor cores take the operands only up to this many: beyond, most experts meet several
@@ -46,7 +48,8 @@ class RoutedExperts:
     def __init__(self, hidden: int, experts: int, identity: int, top: int, intermediate: int, activation: str, router: str,
                  up_proj: str, down_proj: str, correction: str | None = None, shared: PartSpec | None = None,
                  gate_proj: str | None = None, router_bias: str | None = None, weights: str = "scores", scores: str = "softmax",
-                 share_eps: float = 0.0, groups: int = 1, keep: int = 1, shared_gate: str | None = None):
+                 share_eps: float = 0.0, groups: int = 1, keep: int = 1, shared_gate: str | None = None, group_best: int = 2,
+                 weight_scale: float = 1.0, limit: float = 0.0, alpha: float = 1.0):
         """`up_proj` / `down_proj` / `gate_proj`: the tensor names of expert e with `{}` in place of e."""
         known = GATED_ACTIVATIONS if gate_proj is not None else ACTIVATIONS
         if activation not in known:
@@ -60,16 +63,22 @@ class RoutedExperts:
         outputs = experts + identity
         if groups < 1 or outputs % groups or not (0 < keep <= groups) or (groups > 1 and top > keep * (outputs // groups)):
             raise ValueError(f"{outputs} outputs in {groups} groups of which {keep} are kept cannot give {top} choices")
+        if group_best not in (1, 2):
+            raise ValueError(f"groups are ranked by their best score or by the sum of their two best, not of {group_best}")
+        if activation == "clamped" and not limit > 0:
+            raise ValueError(f"a clamp at {limit}: the limit must be positive")
         if shared_gate is not None and shared is None:
             raise ValueError("a gate of the shared expert needs a shared expert")
         self.gated = gate_proj is not None
-        self.rule = ops.RouteRule(scores=scores, renormalise=weights != "scores", share_eps=float(share_eps), groups=int(groups), keep=int(keep))
+        self.rule = ops.RouteRule(scores=scores, renormalise=weights != "scores", share_eps=float(share_eps), groups=int(groups), keep=int(keep),
+                                  group_best=int(group_best), weight_scale=float(weight_scale))
+        self.glu = ops.GluRule("clamped", float(limit), float(alpha)) if activation == "clamped" else ops.GLU_SILU
         if experts < 0 or identity < 0 or not (0 < top <= experts + identity):
             raise ValueError(f"{top} of {experts} + {identity} experts cannot be chosen")
         self.hidden, self.experts, self.identity, self.top = int(hidden), int(experts), int(identity), int(top)
         self.intermediate, self.activation = int(intermediate), activation
         self.names = dict(r=router, c=correction, u=up_proj, d=down_proj, g=gate_proj, b=router_bias, sg=shared_gate)
-        self.bias = self.unit_gain = None
+        self.bias = None
         self.shared = build_part("feed_forward", shared) if shared is not None else None
         self.router = self.correction = self.up = self.down = None
 
@@ -156,14 +165,18 @@ class RoutedExperts:
             rows, gather = torch.empty((tiles * tile, self.hidden), dtype=x.dtype, device=dev), False
             ops.moe_gather(rows, x, row_token)
         ops.tag = "experts_up"
-        if self.gated and self.activation == "silu" and kernel != "simt":
+        if self.gated and self.activation in ("silu", "clamped") and kernel != "simt":
             act = torch.empty((tiles * tile, self.intermediate), dtype=x.dtype, device=dev)
-            ops.gemm_grouped(kernel, act, rows, self.up, tile_group, row_token, gather, ops.EPILOGUE_SWIGLU)
+            ops.gemm_grouped(kernel, act, rows, self.up, tile_group, row_token, gather, ops.EPILOGUE_SWIGLU, self.glu)
         elif self.gated:
             both = torch.empty((tiles * tile, 2 * self.intermediate), dtype=x.dtype, device=dev)
             ops.gemm_grouped(kernel, both, rows, self.up, tile_group, row_token, gather, ops.EPILOGUE_STORE)
             act = torch.empty((tiles * tile, self.intermediate), dtype=x.dtype, device=dev)
-            ops.gated_act(act, both, GATED_ACTIVATIONS[self.activation])   # (rows of tiles not in use hold whatever was there: nobody reads them)
+            # (rows of tiles not in use hold whatever was there: nobody reads them)
+            if self.activation == "clamped":
+                ops.clamped_glu(act, both, None, self.glu.limit, self.glu.alpha)
+            else:
+                ops.gated_act(act, both, GATED_ACTIVATIONS[self.activation])
         else:
             act = torch.empty((tiles * tile, self.intermediate), dtype=x.dtype, device=dev)
             ops.gemm_grouped(kernel, act, rows, self.up, tile_group, row_token, gather, ACTIVATIONS[self.activation])
@@ -202,18 +215,13 @@ class RoutedExperts:
             if store:
                 residual.zero_()
             y, pair_row, weight, shared, z = pieces
-            ops.join_branches(residual, [], (y, pair_row, weight, self._ones(x.device), shared, z))
+            ops.join_branches(residual, [], (y, pair_row, weight, None, shared, z))
             return
         y, pair_row, weight, _ = self._experts(x, ctx)
         ops.moe_combine(residual, y, x, pair_row, weight, add=not store)
         if self.shared is not None:
             self.shared.forward(x, residual, ctx)
         ctx.prenormed = None
-
-    def _ones(self, device) -> torch.Tensor:
-        if self.unit_gain is None:
-            self.unit_gain = torch.ones(self.hidden, dtype=torch.float32, device=device)
-        return self.unit_gain
 
     def forward_then_norm(self, x: torch.Tensor, residual: torch.Tensor, norm, ctx, rows_dtype=None):
         """residual += norm(mixture(x)) for a block whose norm stands behind the sublayer: the experts' rows are added up,

@@ -3,6 +3,9 @@
 Gate and up are one product over the stacked weight [2F, H] whose epilogue applies
 the activation, so the [T, 2F] intermediate never reaches memory.
 
+The projections may have biases: the gate's and the up projection's are added in that epilogue, the output's behind the down product
+(or, asked with `bias_later`, by the block, which adds the sublayer's output up anyway: `output_bias`).
+
 `activation` "gelu_tanh" puts the tanh form of GELU in SiLU's place: residual += (gelu_tanh(x·Wg^T) * (x·Wu^T)) · Wd^T.
 The product's epilogue knows SiLU only, so that form stores gate and up side by side and a small kernel follows."""
 from __future__ import annotations
@@ -18,27 +21,50 @@ from .linear import Linear, compute_form
 ACTIVATIONS = {"silu": ops.GATED_SILU, "gelu_tanh": ops.GATED_GELU_TANH}
 
 
+def _gated_tensors(h: int, f: int, n: dict) -> dict:
+    t = {n["g"]: TensorSpec((f, h)), n["u"]: TensorSpec((f, h)), n["d"]: TensorSpec((h, f))}
+    if n["gb"] is not None:
+        t[n["gb"]] = TensorSpec((f,))
+        t[n["ub"]] = TensorSpec((f,))
+    if n["db"] is not None:
+        t[n["db"]] = TensorSpec((h,))
+    return t
+
+
+def _gated_biases(weights, n: dict, device) -> tuple:
+    """(gate's and up projection's biases side by side, the output's), float32 on the device or None."""
+    bias_in = torch.cat([weights[n["gb"]], weights[n["ub"]]]).to(device).float().contiguous() if n["gb"] is not None else None
+    bias_out = weights[n["db"]].to(device).float().contiguous() if n["db"] is not None else None
+    return bias_in, bias_out
+
+
 class SwiGLU:
     graph_safe = True  # its forward only launches kernels on the current stream
     takes_prenormed = True  # x may be a parts.base.Prenormed: the gate/up product applies the norm's row scale itself
     can_store = True   # forward(..., store=True) overwrites `residual` with its output instead of adding to it
 
-    def __init__(self, hidden: int, intermediate: int, gate_proj: str, up_proj: str, down_proj: str, activation: str = "silu"):
+    def __init__(self, hidden: int, intermediate: int, gate_proj: str, up_proj: str, down_proj: str, activation: str = "silu",
+                 gate_bias: str | None = None, up_bias: str | None = None, down_bias: str | None = None):
         if activation not in ACTIVATIONS:
             raise ValueError(f"activation '{activation}' is not known (known: {', '.join(ACTIVATIONS)})")
+        if (gate_bias is None) != (up_bias is None):
+            raise ValueError("the gate's and the up projection's biases come together or not at all")
+        if gate_bias is not None and activation != "silu":
+            raise ValueError(f"biases in front of '{activation}' are not built (only in front of 'silu')")
         self.hidden, self.intermediate, self.activation = int(hidden), int(intermediate), activation
-        self.names = dict(g=gate_proj, u=up_proj, d=down_proj)
-        self.gate_up = self.down = None
+        self.names = dict(g=gate_proj, u=up_proj, d=down_proj, gb=gate_bias, ub=up_bias, db=down_bias)
+        self.gate_up = self.down = self.output_bias = None
 
     def tensors(self):
-        h, f, n = self.hidden, self.intermediate, self.names
-        return {n["g"]: TensorSpec((f, h)), n["u"]: TensorSpec((f, h)), n["d"]: TensorSpec((h, f))}
+        return _gated_tensors(self.hidden, self.intermediate, self.names)
 
     def load(self, weights, device, dtype):
         n = self.names
         stacked = torch.cat([weights[n["g"]], weights[n["u"]]], dim=0)
         fused = self.activation == "silu"
-        self.gate_up = Linear(compute_form(stacked, device, dtype), ops.EPILOGUE_SWIGLU if fused else ops.EPILOGUE_STORE, role="gate_up")
+        bias_in, self.output_bias = _gated_biases(weights, n, device)
+        self.gate_up = Linear(compute_form(stacked, device, dtype), ops.EPILOGUE_SWIGLU if fused else ops.EPILOGUE_STORE, role="gate_up",
+                              glu_bias=bias_in)
         self.down = Linear(compute_form(weights[n["d"]], device, dtype), ops.EPILOGUE_ACCUMULATE, role="down")
         self.down_store = Linear(self.down.weight, ops.EPILOGUE_STORE, role="down")
 
@@ -46,7 +72,7 @@ class SwiGLU:
         """The weights that this part's first kernel streams."""
         return self.gate_up.weight if self.gate_up is not None else None
 
-    def forward(self, x, residual: torch.Tensor, ctx, store: bool = False) -> None:
+    def forward(self, x, residual: torch.Tensor, ctx, store: bool = False, bias_later: bool = False) -> None:
         act = self.gate_up(x, ctx=ctx)
         if self.activation != "silu":
             both, act = act, torch.empty((act.shape[0], self.intermediate), dtype=act.dtype, device=act.device)
@@ -54,8 +80,10 @@ class SwiGLU:
         if store:
             self.down_store(act, out=residual)
             ctx.prenormed = None
-        else:
-            self.down.add_then_norm(act, residual, getattr(ctx, "norm_ahead", None), ctx)
+        else:   # (with a bias to come the rows are not final: nothing is prepared from them)
+            self.down.add_then_norm(act, residual, getattr(ctx, "norm_ahead", None) if self.output_bias is None else None, ctx)
+        if self.output_bias is not None and not bias_later:
+            ops.bias_act(residual, self.output_bias, 0)
 
 
 register_part("feed_forward", "swiglu", SwiGLU)
@@ -66,8 +94,8 @@ class ClampedGLU:
 
         g = min(W_gate x + b_gate, limit);  u = clamp(W_up x + b_up, -limit, limit);  y = g * sigmoid(alpha * g) * (u + 1);  out = W_down y + b_down
 
-    Gate and up are one product over the stacked weight; a small kernel adds the biases, clamps and applies the activation
-    (float32 arithmetic); the output bias is added behind the down product."""
+    Gate and up are one product over the stacked weight whose epilogue adds the biases, clamps and applies the activation to its
+    float32 sums; the output bias is added behind the down product, or by the block (`bias_later`, see SwiGLU)."""
     graph_safe = True
     can_store = True
 
@@ -79,42 +107,31 @@ class ClampedGLU:
             raise ValueError(f"a clamp at {limit}: the limit must be positive")
         self.hidden, self.intermediate, self.limit, self.alpha = int(hidden), int(intermediate), float(limit), float(alpha)
         self.names = dict(g=gate_proj, u=up_proj, d=down_proj, gb=gate_bias, ub=up_bias, db=down_bias)
-        self.gate_up = self.down = self.down_store = self.bias_in = self.bias_out = None
+        self.gate_up = self.down = self.down_store = self.output_bias = None
 
     def tensors(self):
-        h, f, n = self.hidden, self.intermediate, self.names
-        t = {n["g"]: TensorSpec((f, h)), n["u"]: TensorSpec((f, h)), n["d"]: TensorSpec((h, f))}
-        if n["gb"] is not None:
-            t[n["gb"]] = TensorSpec((f,))
-            t[n["ub"]] = TensorSpec((f,))
-        if n["db"] is not None:
-            t[n["db"]] = TensorSpec((h,))
-        return t
+        return _gated_tensors(self.hidden, self.intermediate, self.names)
 
     def load(self, weights, device, dtype):
         n = self.names
-        self.gate_up = Linear(compute_form(torch.cat([weights[n["g"]], weights[n["u"]]], dim=0), device, dtype), role="gate_up")
+        bias_in, self.output_bias = _gated_biases(weights, n, device)
+        self.gate_up = Linear(compute_form(torch.cat([weights[n["g"]], weights[n["u"]]], dim=0), device, dtype), ops.EPILOGUE_SWIGLU,
+                              role="gate_up", glu=ops.GluRule("clamped", self.limit, self.alpha), glu_bias=bias_in)
         self.down = Linear(compute_form(weights[n["d"]], device, dtype), ops.EPILOGUE_ACCUMULATE, role="down")
         self.down_store = Linear(self.down.weight, ops.EPILOGUE_STORE, role="down")
-        if n["gb"] is not None:
-            self.bias_in = torch.cat([weights[n["gb"]], weights[n["ub"]]]).to(device).float().contiguous()
-        if n["db"] is not None:
-            self.bias_out = weights[n["db"]].to(device).float().contiguous()
 
     def first_weights(self):
         return self.gate_up.weight if self.gate_up is not None else None
 
-    def forward(self, x, residual: torch.Tensor, ctx, store: bool = False) -> None:
-        both = self.gate_up(x, ctx=ctx)
-        act = torch.empty((both.shape[0], self.intermediate), dtype=both.dtype, device=both.device)
-        ops.clamped_glu(act, both, self.bias_in, self.limit, self.alpha)
+    def forward(self, x, residual: torch.Tensor, ctx, store: bool = False, bias_later: bool = False) -> None:
+        act = self.gate_up(x, ctx=ctx)
         ctx.prenormed = None
         if store:
             self.down_store(act, out=residual)
         else:
             self.down(act, out=residual)
-        if self.bias_out is not None:
-            ops.bias_act(residual, self.bias_out, 0)
+        if self.output_bias is not None and not bias_later:
+            ops.bias_act(residual, self.output_bias, 0)
 
 
 register_part("feed_forward", "clamped_glu", ClampedGLU)
