@@ -140,7 +140,7 @@ def reference_arm() -> int:
     return 0
 
 
-# ---- another design beside the flagship: `--design pemezen`, `--design novunex`, `--design rutetar`, `--design pulenex` ----------------------------
+# ---- another design beside the flagship: `--design pemezen`, `--design novunex`, `--design rutetar`, `--design pulenex`, ... ----------------------------
 # Sizes that resemble a real model's layers (random weights), and a Hunyuan-dense model of the same width, depth and
 # nearly the same number of weights per layer beside it: the closest model that the library has.
 DESIGN_SIZES = {
@@ -285,8 +285,35 @@ def sosepel_config(size: str, layers: int):
                                         embedding=dict(scale=6.0, bigram=dict(buckets=z["buckets"], mul_prev=4099, mul_cur=61))))
 
 
-DESIGN_NEIGHBOURS = {"sosepel": "novunex"}   # a design whose closest model is another one than the dense: that one stands beside both
-DESIGN_TABLES = {"sosepel": SOSEPEL_SIZES, "pemezen": DESIGN_SIZES, "novunex": NOVUNEX_SIZES, "rutetar": RUTETAR_SIZES, "pulenex": PULENEX_SIZES}
+# Gomerax: latent attention with a latent vector of the queries, in a window, with sinks (head sizes, latent width and window as Pulenex
+# has them); feed-forwards as Sosepel's (its dense ones have a gate: half the width)
+GOMERAX_SIZES = {
+    "s": dict(width=1024, vocab=32768, heads=8, dim=64, rot_dim=32, vdim=64, q_rank=512, kv_rank=256, window=1024, dense_ff=3776, experts=16, top=4,
+              groups=4, keep=2, ff=512, shared=1024, dense=DESIGN_SIZES["s"]["dense"]),
+    "m": dict(width=2048, vocab=65536, heads=16, dim=128, rot_dim=64, vdim=128, q_rank=1024, kv_rank=512, window=2048, dense_ff=7552, experts=32, top=4,
+              groups=8, keep=4, ff=1024, shared=2048, dense=DESIGN_SIZES["m"]["dense"]),
+}
+
+
+def gomerax_config(size: str, layers: int):
+    from hymt2sharp_b200.config import GomeraxConfig
+    z = GOMERAX_SIZES[size]
+    entries = []
+    for i in range(max(3, layers - 2)):
+        mixer = dict(heads=z["heads"], dim=z["dim"], rot_dim=z["rot_dim"], vdim=z["vdim"], q_rank=z["q_rank"], kv_rank=z["kv_rank"],
+                     scale=(z["dim"] + z["rot_dim"]) ** -0.5, mask=dict(size=z["window"]), rot=dict(dims=z["rot_dim"], base=250000.0))
+        mlp = dict(kind="dense", ff=z["dense_ff"]) if i % 4 == 0 else \
+            dict(kind="moe", expert=dict(ff=z["ff"], limit=7.0), router=dict(experts=z["experts"], top=z["top"], scale=1.8,
+                                                                             groups=dict(count=z["groups"], keep=z["keep"])),
+                 shared=dict(ff=z["shared"], limit=7.0))
+        entries.append(dict(type="latent_attention", mixer=mixer, mlp=mlp))
+    return GomeraxConfig.from_dict(dict(architecture="Gomerax", vocab=z["vocab"], width=z["width"], layers=entries, norm=dict(eps=1e-6),
+                                        max_positions=16384, loop=dict(start=1, stop=3, times=2), embedding=dict(scale=6.0)))
+
+
+# designs whose closest models are others than the dense: those stand beside both
+DESIGN_NEIGHBOURS = {"sosepel": ("novunex",), "gomerax": ("sosepel", "pulenex")}
+DESIGN_TABLES = {"gomerax": GOMERAX_SIZES, "sosepel": SOSEPEL_SIZES, "pemezen": DESIGN_SIZES, "novunex": NOVUNEX_SIZES, "rutetar": RUTETAR_SIZES, "pulenex": PULENEX_SIZES}
 
 
 def make_design_models(size: str, layers: int, design: str = "pemezen") -> dict:
@@ -304,13 +331,9 @@ def make_design_models(size: str, layers: int, design: str = "pemezen") -> dict:
             mixer = dict(heads=z["heads"], dim=z["dim"], rot_dim=z["rot_dim"], vdim=z["vdim"], kv_rank=z["kv_rank"],
                          scale=(z["dim"] + z["rot_dim"]) ** -0.5, rot=rot)
         entries.append(dict(type=kind, mixer=mixer, mlp=dict(kind="dense", ff=z["ff"])))
-    makers = {"novunex": novunex_config, "sosepel": sosepel_config}
+    makers = {"novunex": novunex_config, "rutetar": rutetar_config, "pulenex": pulenex_config, "sosepel": sosepel_config, "gomerax": gomerax_config}
     if design in makers:
         new = makers[design](size, layers)
-    elif design == "rutetar":
-        new = rutetar_config(size, layers)
-    elif design == "pulenex":
-        new = pulenex_config(size, layers)
     else:
         new = PemezenConfig.from_dict(dict(architecture="Pemezen", vocab=z["vocab"], width=z["width"], layers=entries,
                                            norm=dict(eps=1e-6, groups=2), canon=dict(taps=4), embedding=dict(scale=1.0), logit_softcap=30.0))
@@ -319,8 +342,7 @@ def make_design_models(size: str, layers: int, design: str = "pemezen") -> dict:
                                             rope_scaling={"type": "dynamic", "alpha": 1000.0}, **z["dense"]))
     old_data = {k: v for k, v in old.to_dict().items()}
     folders = {}
-    beside = DESIGN_NEIGHBOURS.get(design)
-    for name, cfg in ((design, new), *(((beside, makers[beside](size, layers)),) if beside else ()),
+    for name, cfg in ((design, new), *((other, makers[other](size, layers)) for other in DESIGN_NEIGHBOURS.get(design, ())),
                       ("hunyuan_dense", HunyuanDenseConfig.from_dict(old_data))):
         folders[name] = write_random_model(tempfile.mkdtemp(prefix=f"hymt2_bench_{name}_"), cfg, 7, 0.02)
     return folders

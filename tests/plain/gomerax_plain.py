@@ -66,13 +66,13 @@ def layer_runs(config: dict) -> list:
 
 # -- latent attention ---------------------------------------------------------------------------------
 def turn(v: torch.Tensor, position: int, dims: int, base: float) -> torch.Tensor:
-    """The first `dims` entries of v [n] in neighbouring pairs, pair i by position * base^(-2i/dims)."""
+    """The first `dims` entries of v [.., n] in neighbouring pairs, pair i by position * base^(-2i/dims)."""
     out = v.clone()
     for i in range(dims // 2):
         a = position * base ** (-2.0 * i / dims)
         c, s = math.cos(a), math.sin(a)
-        out[2 * i] = v[2 * i] * c - v[2 * i + 1] * s
-        out[2 * i + 1] = v[2 * i + 1] * c + v[2 * i] * s
+        out[..., 2 * i] = v[..., 2 * i] * c - v[..., 2 * i + 1] * s
+        out[..., 2 * i + 1] = v[..., 2 * i + 1] * c + v[..., 2 * i] * s
     return out
 
 
@@ -92,8 +92,7 @@ def queries(h: torch.Tensor, w: dict, p: str, m: dict, eps: float) -> torch.Tens
     c = norm_plain(h @ w[p + "dq"].T, w[p + "dq.norm"], eps)
     q = (c @ w[p + "uq"].T).view(T, m["heads"], m["dim"] + m["rot_dim"]).clone()
     for t in range(T):
-        for a in range(m["heads"]):
-            q[t, a, m["dim"]:] = turn(q[t, a, m["dim"]:], t, m["rot"]["dims"], m["rot"]["base"])
+        q[t, :, m["dim"]:] = turn(q[t, :, m["dim"]:], t, m["rot"]["dims"], m["rot"]["base"])
     return q
 
 
@@ -105,17 +104,17 @@ def compressed(h: torch.Tensor, w: dict, p: str, m: dict, eps: float):
     return norm_plain(z[:, :m["kv_rank"]], w[p + "dkv.norm"], eps), k
 
 
-def attend(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scale: float, window, sink) -> torch.Tensor:
-    """One head: q, k [T, d], v [T, dv] -> [T, dv]."""
+def attend(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scale: float, window, sink, only=None) -> torch.Tensor:
+    """One head: q, k [T, d], v [T, dv] -> [T, dv] (`only`: zeros but for these tokens' rows)."""
     out = torch.zeros((q.shape[0], v.shape[1]), dtype=q.dtype)
-    for i in range(q.shape[0]):
-        seen = [j for j in range(q.shape[0]) if sees(i, j, window)]
-        a, b = seen[0], seen[-1] + 1
+    for i in range(q.shape[0]) if only is None else only:
+        seen = [j for j in range(i + 1) if sees(i, j, window)]
+        a, b = seen[0], i + 1
         out[i] = weights_with_sink((k[a:b] @ q[i]) * scale, sink) @ v[a:b]
     return out
 
 
-def attention(h: torch.Tensor, w: dict, p: str, m: dict, eps: float) -> torch.Tensor:
+def attention(h: torch.Tensor, w: dict, p: str, m: dict, eps: float, only=None) -> torch.Tensor:
     T, H = h.shape[0], m["heads"]
     q = queries(h, w, p, m, eps)
     c, kr = compressed(h, w, p, m, eps)
@@ -123,7 +122,8 @@ def attention(h: torch.Tensor, w: dict, p: str, m: dict, eps: float) -> torch.Te
     v = (c @ w[p + "uv"].T).view(T, H, m["vdim"])
     window = (m.get("mask") or {}).get("size")
     sink = w.get(p + "sink")
-    heads = [attend(q[:, a], torch.cat([k[:, a], kr], dim=1), v[:, a], m["scale"], window, None if sink is None else sink[a]) for a in range(H)]
+    heads = [attend(q[:, a], torch.cat([k[:, a], kr], dim=1), v[:, a], m["scale"], window, None if sink is None else sink[a], only)
+             for a in range(H)]
     return torch.cat(heads, dim=-1) @ w[p + "o"].T
 
 
