@@ -23,7 +23,7 @@
 // over the visible keys), :535-595 (combine).  A query at position p sees keys
 // [max(0, p - window + 1), p].
 // Values may be of another width than keys (DV entries a head, O has DV columns), and the softmax may have a sink: one
-// more term in its denominator, of score 0 and without a value, added to a row's sum at the end.
+// more term in its denominator, of score 0 or of a score of the head's own and without a value, added to a row's sum at the end.
 // Takes key and value sizes of 64 and 128 (in any pairing) and cache blocks of 64 tokens; other shapes stay with the
 // general kernel.
 //
@@ -68,6 +68,7 @@ struct PrefillParams {
     float scale, softcap, temp_coef;
     int temp_every;
     float lambda, eps, factor;
+    const float* sink_scores;  // [nh] or null: the sinks' scores (null: 0)
 };
 
 enum { FORM_CLASSIC = 0, FORM_MAPS = 1, FORM_MAPS_CAPPED = 2 };
@@ -469,7 +470,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         if (!MAPS && ok) {
             // the sink: a term exp2(0 - m) in the sum (m is the offset that every numerator of the row was taken against; a row
             // that sees a key has a finite one)
-            if (p.sink && m > -INFINITY) l += exp2f(-m);
+            if (p.sink && m > -INFINITY) l += exp2f((p.sink_scores ? p.sink_scores[head] * 1.4426950408889634f : 0.f) - m);
             const float inv = l > 0.f ? 1.0f / l : 0.f;
             __nv_bfloat16* dst = p.out + ((size_t)(tok0 + qtile * Q_ROWS + r) * p.nh + head) * DV;
 #pragma unroll
@@ -626,7 +627,7 @@ HYMT2_API int hymt2_attention_prefill_tc_kv(void* out, const void* q, const void
                                             long cache_blocks, const int* block_table, int table_stride, int block_tokens,
                                             const int* cu_seqlens, const int* slot_ids, const int* kv_lens, int batch,
                                             int tokens, int max_new_tokens, int nh, int nkv, int d, int dv, float scale, int window,
-                                            int sink, int* status, cudaStream_t stream) {
+                                            int sink, const float* sink_scores, int* status, cudaStream_t stream) {
     if (tokens == 0 || batch == 0) return HYMT2_OK;
     HYMT2_REQUIRE((d == 64 || d == 128) && (dv == 64 || dv == 128), "attention_prefill_tc: heads of %d and %d are not taken (64 and 128 are)", d, dv);
     HYMT2_REQUIRE(block_tokens == KEY_TILE, "attention_prefill_tc: cache blocks must hold %d tokens", KEY_TILE);
@@ -645,7 +646,8 @@ HYMT2_API int hymt2_attention_prefill_tc_kv(void* out, const void* q, const void
     cudaGetDevice(&dev);
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
     PrefillParams p{(__nv_bfloat16*)out, block_table, cu_seqlens, slot_ids, kv_lens, table_stride, nh, nkv, window,
-                    batch, qtiles, sms, scale * 1.4426950408889634f, status, sink, scale};
+                    batch, qtiles, sms, scale * 1.4426950408889634f, status, sink || sink_scores ? 1 : 0, scale};
+    p.sink_scores = sink_scores;
     dim3 grid((unsigned)(qtiles * nh * batch), 1, 1);
     if (d == 128) return dv == 128 ? launch<128, 128>(mq, mk, mv, p, grid, stream) : launch<128, 64>(mq, mk, mv, p, grid, stream);
     return dv == 128 ? launch<64, 128>(mq, mk, mv, p, grid, stream) : launch<64, 64>(mq, mk, mv, p, grid, stream);
@@ -658,7 +660,7 @@ HYMT2_API int hymt2_attention_prefill_tc(void* out, const void* q, const void* k
                                          int tokens, int max_new_tokens, int nh, int nkv, int d, float scale, int window,
                                          int* status, cudaStream_t stream) {
     return hymt2_attention_prefill_tc_kv(out, q, k_cache, v_cache, cache_blocks, block_table, table_stride, block_tokens, cu_seqlens,
-                                         slot_ids, kv_lens, batch, tokens, max_new_tokens, nh, nkv, d, d, scale, window, 0, status, stream);
+                                         slot_ids, kv_lens, batch, tokens, max_new_tokens, nh, nkv, d, d, scale, window, 0, nullptr, status, stream);
 }
 
 // Differential attention: q rows of nh * 2 * d entries (row stride ldq), keys' rows of 2 * d, out [tokens, nh * dv].  softcap 0: scores

@@ -124,6 +124,84 @@ latent_prep_kernel(LatentPrepParams p) {
     }
 }
 
+// Whole prompts from position 0 for the paged prompt attention: every head's queries, keys and values in the layout that kernel
+// reads, with heads of D and DV entries (D: dim + rot and zeros behind them).  One block per token, 16 bytes a thread and access:
+//   q_out[t, h] = [query entries | rotated query entries | zeros]
+//   k_out[block][h][place] = [own key entries | shared rotated key entries | zeros],  v_out[block][h][place] = values
+// A sequence's tokens fill blocks of BLOCK_TOKENS of its own, numbered through the step; table[slot][i] names its i-th block.
+constexpr int BLOCK_TOKENS = 64;
+
+struct LatentPlaceParams {
+    const __nv_bfloat16* q;       // [T, ldq], not rotated
+    const __nv_bfloat16* kv;      // [T, ld_kv]: heads' own key entries (dim each), then heads' values (dv each)
+    const __nv_bfloat16* shared;  // [T, ld_shared]: the shared key entries, rotated
+    long ldq, ld_kv, ld_shared;
+    __nv_bfloat16 *q_out, *k_out, *v_out;
+    int* table;
+    const int *token_seq, *token_pos, *cu_seqlens, *slot_ids;
+    const float* inv_freq;
+    int table_stride, heads, dim, rot, dv, D, rot_dims, max_blocks;
+    float amplitude;
+};
+
+__global__ void __launch_bounds__(256)
+latent_place_kernel(LatentPlaceParams p) {
+    extern __shared__ float smem[];   // [rot_dims / 2][2] cosine, sine
+    __shared__ int block_s;
+    pdl_wait();
+    pdl_launch_dependents();
+    const int t = blockIdx.x, seq = p.token_seq[t], pos = p.token_pos[t];
+    const int place = t - p.cu_seqlens[seq];
+    if (threadIdx.x == 0) {
+        int block = place / BLOCK_TOKENS;
+        for (int b = 0; b < seq; b++) block += (p.cu_seqlens[b + 1] - p.cu_seqlens[b] + BLOCK_TOKENS - 1) / BLOCK_TOKENS;
+        block_s = block;
+        const int slot = p.slot_ids[seq];
+        if (place % BLOCK_TOKENS == 0 && slot >= 0) p.table[(size_t)slot * p.table_stride + place / BLOCK_TOKENS] = block;
+    }
+    for (int i = threadIdx.x; i < p.rot_dims / 2; i += blockDim.x) {
+        float sn, c;
+        sincosf((float)pos * p.inv_freq[i], &sn, &c);
+        smem[2 * i] = c * p.amplitude;
+        smem[2 * i + 1] = sn * p.amplitude;
+    }
+    __syncthreads();
+    const int block = block_s;
+    if (block >= p.max_blocks) return;    // (never: the host makes room for every sequence's last block)
+    const int d8 = p.D / 8, dim8 = p.dim / 8, rot8 = p.rot / 8, dv8 = p.dv / 8;
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    const uint4* q = reinterpret_cast<const uint4*>(p.q + (size_t)t * p.ldq);
+    const uint4* kv = reinterpret_cast<const uint4*>(p.kv + (size_t)t * p.ld_kv);
+    const uint4* sh = reinterpret_cast<const uint4*>(p.shared + (size_t)t * p.ld_shared);
+    uint4* qo = reinterpret_cast<uint4*>(p.q_out) + (size_t)t * p.heads * d8;
+    const size_t row0 = (size_t)block * p.heads * BLOCK_TOKENS + place % BLOCK_TOKENS;
+    for (int i = threadIdx.x; i < p.heads * d8; i += blockDim.x) {
+        const int h = i / d8, c = i - h * d8;
+        uint4 k = zero, v = zero;
+        if (c < dim8) {
+            v = q[h * (dim8 + rot8) + c];
+            k = kv[h * dim8 + c];
+        } else if (c < dim8 + rot8) {
+            v = q[h * (dim8 + rot8) + c];
+            k = sh[c - dim8];
+            __nv_bfloat162* pair = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+                const int at = (c - dim8) * 4 + j;
+                if (2 * at >= p.rot_dims) continue;
+                const float a = __low2float(pair[j]), b = __high2float(pair[j]), cs = smem[2 * at], sn = smem[2 * at + 1];
+                pair[j] = __floats2bfloat162_rn(a * cs - b * sn, b * cs + a * sn);
+            }
+        }
+        qo[i] = v;
+        reinterpret_cast<uint4*>(p.k_out)[(row0 + (size_t)h * BLOCK_TOKENS) * d8 + c] = k;
+    }
+    for (int i = threadIdx.x; i < p.heads * dv8; i += blockDim.x) {
+        const int h = i / dv8, c = i - h * dv8;
+        reinterpret_cast<uint4*>(p.v_out)[(row0 + (size_t)h * BLOCK_TOKENS) * dv8 + c] = kv[p.heads * dim8 + i];
+    }
+}
+
 }  // namespace
 
 HYMT2_API int hymt2_latent_prep(const void* proj, long ldp, int q_cols, void* q_out, void* rows_out, void* cache, int dtype,
@@ -146,4 +224,25 @@ HYMT2_API int hymt2_latent_prep(const void* proj, long ldp, int q_cols, void* q_
     const size_t smem = sizeof(float) * ((size_t)rot_dims + 33);
     HYMT2_DISPATCH_DTYPE(dtype, T, launch_pdl(latent_prep_kernel<T>, dim3(tokens), dim3(128), smem, stream, p));
     return hymt2_check_launch("latent_prep");
+}
+
+// See latent_place_kernel; k_out holds max_blocks * heads * 64 rows of D entries, v_out as many of dv, table a row per cache slot.
+HYMT2_API int hymt2_latent_place(const void* q, long ldq, const void* kv, long ld_kv, const void* shared, long ld_shared, void* q_out, void* k_out,
+                                 void* v_out, int* table, int table_stride, int max_blocks, const int* token_seq, const int* token_pos,
+                                 const int* cu_seqlens, const int* slot_ids, const float* inv_freq, int rot_dims, float amplitude, int tokens,
+                                 int heads, int dim, int rot, int dv, int D, cudaStream_t stream) {
+    if (tokens == 0) return HYMT2_OK;
+    HYMT2_REQUIRE(tokens > 0 && heads > 0 && dim > 0 && rot >= 0 && dv > 0 && dim + rot <= D && max_blocks > 0, "latent_place: bad sizes");
+    HYMT2_REQUIRE(dim % 8 == 0 && rot % 8 == 0 && dv % 8 == 0 && D % 8 == 0 && ldq % 8 == 0 && ld_kv % 8 == 0 && ld_shared % 8 == 0, "latent_place: rows come in pieces of 8 entries");
+    HYMT2_REQUIRE(((uintptr_t)q | (uintptr_t)kv | (uintptr_t)shared | (uintptr_t)q_out | (uintptr_t)k_out | (uintptr_t)v_out) % 16 == 0, "latent_place: matrices must be 16-byte aligned");
+    HYMT2_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= rot && (rot_dims == 0 || inv_freq), "latent_place: %d rotated entries of %d", rot_dims, rot);
+    LatentPlaceParams p;
+    p.q = (const __nv_bfloat16*)q; p.kv = (const __nv_bfloat16*)kv; p.shared = (const __nv_bfloat16*)shared;
+    p.ldq = ldq; p.ld_kv = ld_kv; p.ld_shared = ld_shared;
+    p.q_out = (__nv_bfloat16*)q_out; p.k_out = (__nv_bfloat16*)k_out; p.v_out = (__nv_bfloat16*)v_out; p.table = table;
+    p.token_seq = token_seq; p.token_pos = token_pos; p.cu_seqlens = cu_seqlens; p.slot_ids = slot_ids; p.inv_freq = inv_freq;
+    p.table_stride = table_stride; p.heads = heads; p.dim = dim; p.rot = rot; p.dv = dv; p.D = D; p.rot_dims = rot_dims; p.max_blocks = max_blocks;
+    p.amplitude = amplitude;
+    launch_pdl(latent_place_kernel, dim3(tokens), dim3(256), sizeof(float) * (size_t)rot_dims, stream, p);
+    return hymt2_check_launch("latent_place");
 }

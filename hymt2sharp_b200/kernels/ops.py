@@ -1016,7 +1016,7 @@ def latent_prep(proj: torch.Tensor, q_cols: int, q_out: torch.Tensor | None, cac
     back into proj, in place.  rows_out [T, rank + rot]: the cache rows once more, side by side for all tokens.  With neither a
     cache plane nor rows_out the projection need not hold a compressed row at all (only the queries are read).
     q_latent = (gain [q_rank] float32, out [T, q_rank]): the projection starts with a compressed query of q_rank = q_cols entries in
-    place of the heads' queries (heads is then 0): out = its RMS norm with the gain."""
+    place of the heads' queries (heads is then 0): out = its RMS norm with the gain.  heads 0 without it: the queries are left alone."""
     ldp = _rows_view(proj, "proj")
     T = proj.shape[0]
     dl = rank + rot
@@ -1026,7 +1026,7 @@ def latent_prep(proj: torch.Tensor, q_cols: int, q_out: torch.Tensor | None, cac
         _need(rows_out, "rows_out", proj.dtype, 2)
     # a run without a compressed row of its own (it reads another run's cache) brings the queries alone
     rowless = cache_plane is None and rows_out is None
-    if proj.shape[1] < q_cols + (0 if rowless else dl) or (q_latent is None and q_cols != heads * (dim + rot)) or (q_out is not None and q_out.shape != (T, heads * dl)) \
+    if proj.shape[1] < q_cols + (0 if rowless else dl) or (heads and q_cols != heads * (dim + rot)) or (q_out is not None and q_out.shape != (T, heads * dl)) \
             or (rows_out is not None and rows_out.shape != (T, dl)):
         raise KernelError(f"latent_prep: shapes proj {tuple(proj.shape)} do not fit {heads} heads of {dim} + {rot} and a row of {dl}")
     if cache_plane is not None:
@@ -1148,6 +1148,32 @@ def latent_attention_expanded_supported(dtype: torch.dtype, dim: int, rot: int, 
     if hit is None:
         hit = _mma_ok[key] = bool(_lib().hymt2_latent_attention_expanded_supported(c_int(dim), c_int(rot), c_int(dv)))
     return hit
+
+
+LATENT_PLACE_BLOCK = 64    # tokens of a block that latent_place fills
+
+
+def latent_place(q: torch.Tensor, kv: torch.Tensor, shared: torch.Tensor, q_out: torch.Tensor, k_out: torch.Tensor, v_out: torch.Tensor,
+                 table: torch.Tensor, token_seq: torch.Tensor, token_pos: torch.Tensor, cu_seqlens: torch.Tensor, slot_ids: torch.Tensor,
+                 inv_freq: torch.Tensor | None, rot_dims: int, amplitude: float, heads: int, dim: int, rot: int, dv: int) -> None:
+    """For whole prompts from position 0, bfloat16: q [T, >= heads * (dim + rot)] not rotated, kv [T, heads * (dim + dv)] (all heads' own
+    key entries, then their values) and shared [T, rot] (the rotated key entries of all heads) become q_out [T, heads * D], k_out
+    [blocks, heads, 64, D] and v_out [blocks, heads, 64, dv], a head's D entries being its dim, its rot rotated ones and zeros: what
+    attention_prefill_tc_kv reads with `table` [slots, ..], whose rows of the step's slots are filled with the blocks' numbers."""
+    for t, n in ((q, "q"), (kv, "kv"), (shared, "shared")):
+        _rows_view(t, n, torch.bfloat16)
+    _need(q_out, "q_out", torch.bfloat16, 2); _need(k_out, "k_out", torch.bfloat16, 4); _need(v_out, "v_out", torch.bfloat16, 4)
+    _need(table, "table", torch.int32, 2); _f32(inv_freq, "inv_freq", rot_dims // 2)
+    T, D = q.shape[0], k_out.shape[3]
+    if kv.shape != (T, heads * (dim + dv)) or shared.shape != (T, rot) or q.shape[1] < heads * (dim + rot) or q_out.shape != (T, heads * D) \
+            or k_out.shape[1:3] != (heads, LATENT_PLACE_BLOCK) or v_out.shape != (*k_out.shape[:3], dv):
+        raise KernelError(f"latent_place: shapes q {tuple(q.shape)} kv {tuple(kv.shape)} k_out {tuple(k_out.shape)} v_out {tuple(v_out.shape)}")
+    for t, n in ((token_seq, "token_seq"), (token_pos, "token_pos"), (cu_seqlens, "cu_seqlens"), (slot_ids, "slot_ids")):
+        _need(t, n, torch.int32, 1)
+    _check(_lib().hymt2_latent_place(_ptr(q), c_long(q.stride(0)), _ptr(kv), c_long(kv.stride(0)), _ptr(shared), c_long(shared.stride(0)), _ptr(q_out),
+                                     _ptr(k_out), _ptr(v_out), _ptr(table), c_int(table.stride(0)), c_int(k_out.shape[0]), _ptr(token_seq),
+                                     _ptr(token_pos), _ptr(cu_seqlens), _ptr(slot_ids), _ptr(inv_freq), c_int(rot_dims), c_float(amplitude), c_int(T),
+                                     c_int(heads), c_int(dim), c_int(rot), c_int(dv), c_int(D), _stream()), "latent_place")
 
 
 def latent_attention_expanded(out: torch.Tensor, q: torch.Tensor, kexp: torch.Tensor, vexp: torch.Tensor, krot: torch.Tensor,
@@ -1558,9 +1584,11 @@ def _attention_kv_shapes(what: str, out, q, k_plane, v_plane, nh, nkv, d, dv) ->
 
 def attention_prefill_tc_kv(out: torch.Tensor, q: torch.Tensor, k_plane: torch.Tensor, v_plane: torch.Tensor, block_table: torch.Tensor,
                             cu_seqlens: torch.Tensor, slot_ids: torch.Tensor, kv_lens: torch.Tensor, batch: int, max_new_tokens: int,
-                            nh: int, nkv: int, d: int, dv: int, scale: float, window: int, sink: bool, status: torch.Tensor) -> None:
+                            nh: int, nkv: int, d: int, dv: int, scale: float, window: int, sink: bool, status: torch.Tensor,
+                            sink_scores: torch.Tensor | None = None) -> None:
     """attention_prefill_tc with keys of d and values of dv entries a head (64 or 128 each; out [T, nh * dv]) and optionally a
-    sink in the softmax."""
+    sink in the softmax, of score 0 or of the heads' own `sink_scores` [nh] float32."""
+    _f32(sink_scores, "sink_scores", nh)
     _attention_kv_shapes("attention_prefill_tc", out, q, k_plane, v_plane, nh, nkv, d, dv)
     _need(block_table, "block_table", torch.int32, 2)
     for t, n in ((cu_seqlens, "cu_seqlens"), (slot_ids, "slot_ids"), (kv_lens, "kv_lens")):
@@ -1569,7 +1597,7 @@ def attention_prefill_tc_kv(out: torch.Tensor, q: torch.Tensor, k_plane: torch.T
                                                 _ptr(block_table), c_int(block_table.stride(0)), c_int(k_plane.shape[2]),
                                                 _ptr(cu_seqlens), _ptr(slot_ids), _ptr(kv_lens), c_int(batch), c_int(out.shape[0]),
                                                 c_int(max_new_tokens), c_int(nh), c_int(nkv), c_int(d), c_int(dv), c_float(scale),
-                                                c_int(window), c_int(1 if sink else 0), _ptr(status), _stream()), "attention_prefill_tc")
+                                                c_int(window), c_int(1 if sink else 0), _ptr(sink_scores), _ptr(status), _stream()), "attention_prefill_tc")
 
 
 def attention_decode_kv(out: torch.Tensor, q: torch.Tensor, k_plane: torch.Tensor, v_plane: torch.Tensor, block_table: torch.Tensor,

@@ -14,7 +14,9 @@ the rotation are float32; the projections run in the engine's compute type.
 
 A prompt that starts at position 0 brings all of its keys along, and a head's own rows (dim + rot_dim, vdim) are several
 times narrower than the compressed row: there the bfloat16 engine rebuilds every head's keys and values with one product
-over all tokens and runs the attention per head, which is the same sums in another order (EXPAND_FROM_TOKENS).
+over all tokens and runs the attention per head, which is the same sums in another order (EXPAND_FROM_TOKENS).  Where a head's
+entries fit the tcgen05 prompt kernel (keys of up to 128 entries, values of 64 or 128), one kernel rotates the queries and lays
+all heads' queries, keys and values out as that kernel reads them; else the attention runs on the fragment kernel.
 
 `q_rank`: the queries come out of a latent vector of their own, q = W_q (gain * unit_rms(W_dq x)) (`dq_proj`, `dq_norm`; `q_proj` is then
 W_q [., q_rank]): its down-projection is the first rows of the fused projection, its norm runs with the compressed row's.
@@ -115,7 +117,11 @@ class LatentAttention:
         self.uk_t = compute_form(uk, device, dtype)
         self.uv = compute_form(weights[n["uv"]].reshape(H, self.vdim, self.rank), device, dtype)
         self.c_gain = weights[n["cn"]].to(device).float().contiguous() if self.own_kv else torch.ones(self.rank, dtype=torch.float32, device=device)
-        if self.rank % 8 == 0 and ops.latent_attention_expanded_supported(dtype, self.dim, self.rot, self.vdim):
+        # the tcgen05 prompt kernel's width of a head: its entries, and zeros up to 64 or 128 (None: not for these sizes)
+        key = self.dim + self.rot
+        fits = dtype == torch.bfloat16 and self.scale > 0 and key <= 128 and self.vdim in (64, 128) and self.dim % 8 == 0 and self.rot % 8 == 0
+        self.prompt_width = (64 if key <= 64 else 128) if fits else None
+        if self.rank % 8 == 0 and (fits or ops.latent_attention_expanded_supported(dtype, self.dim, self.rot, self.vdim)):
             # every head's key and value rows in one product over the latent vectors: [W_uk; W_uv]
             self.ukv = Linear(compute_form(torch.cat([weights[n["uk"]], weights[n["uv"]]], dim=0), device, dtype), role="kv_expand")
         if self.position is not None:
@@ -152,19 +158,21 @@ class LatentAttention:
         ops.tag = None
         self._gate_and_project(out, proj, residual, ctx, store)
 
-    def _prepare(self, proj, q_out, rotary, plane, table, ctx, rows_out=None) -> torch.Tensor:
+    def _prepare(self, proj, q_out, rotary, plane, table, ctx, rows_out=None, turn_queries: bool = True) -> torch.Tensor:
         """Norms, rotations and the cache rows of the step's tokens; returns the matrix whose first columns are the heads' queries.
-        Their rotated parts go to `q_out` (behind the places of the compressed entries) or, with None, stay in place."""
+        Their rotated parts go to `q_out` (behind the places of the compressed entries) or, with None, stay in place; without
+        `turn_queries` they are left to whoever reads them."""
         table_args = (table, ctx.cache.block_tokens, ctx.token_seq, ctx.token_pos, ctx.slot_ids, self.c_gain)
         turn_args = (rotary.inv_freq if rotary else None, rotary.rope_dim if rotary else 0, rotary.amplitude if rotary else 1.0, self.eps)
         if self.q_rank is None:
-            ops.latent_prep(proj, self.q_cols, q_out, plane, *table_args, *turn_args, self.heads, self.dim, self.rot, self.rank, rows_out=rows_out)
+            ops.latent_prep(proj, self.q_cols, q_out, plane, *table_args, *turn_args, self.heads if turn_queries else 0, self.dim, self.rot, self.rank, rows_out=rows_out)
             return proj
         cq = torch.empty((proj.shape[0], self.q_rank), dtype=proj.dtype, device=proj.device)
         ops.latent_prep(proj, self.q_rank, None, plane, *table_args, *turn_args, 0, self.dim, self.rot, self.rank, rows_out=rows_out,
                         q_latent=(self.q_gain, cq))
         q = self.uq(cq, ctx=ctx)
-        ops.latent_prep(q, self.q_cols, q_out, None, *table_args, *turn_args, self.heads, self.dim, self.rot, self.rank)
+        if turn_queries:
+            ops.latent_prep(q, self.q_cols, q_out, None, *table_args, *turn_args, self.heads, self.dim, self.rot, self.rank)
         return q
 
     def _gate_and_project(self, out, proj, residual, ctx, store: bool) -> None:
@@ -186,13 +194,29 @@ class LatentAttention:
             ctx.shared[kept] = rows
         else:
             rows = ctx.shared[kept]
-        q = self._prepare(proj, None, rotary, plane, table, ctx, rows_out=rows if self.own_kv else None)
+        q = self._prepare(proj, None, rotary, plane, table, ctx, rows_out=rows if self.own_kv else None, turn_queries=self.prompt_width is None)
         kv = self.ukv(rows[:, :self.rank], ctx=ctx)                    # [T, H * dim | H * vdim]
         out = torch.empty((T, H * self.vdim), dtype=proj.dtype, device=proj.device)
+        if self.prompt_width is not None:
+            self._attend_placed(out, q, kv, rows[:, self.rank:], rotary, ctx)
+            return out
         ops.latent_attention_expanded(out, q[:, :self.q_cols], kv[:, :H * self.dim], kv[:, H * self.dim:], rows[:, self.rank:],
                                       ctx.cu_seqlens, ctx.slot_ids, ctx.kv_lens, ctx.num_seqs, ctx.max_new_tokens, H, self.dim,
                                       self.rot, self.vdim, self.scale, self.window, self.sink)
         return out
+
+    def _attend_placed(self, out, q, kv, shared, rotary, ctx) -> None:
+        """Every head's queries, keys and values laid out for the tcgen05 prompt kernel, and that kernel."""
+        H, D, block = self.heads, self.prompt_width, ops.LATENT_PLACE_BLOCK
+        blocks = sum(-(-n // block) for n in ctx.host_new_tokens)
+        make = lambda *shape, dtype=q.dtype: torch.empty(shape, dtype=dtype, device=q.device)
+        qp, kp, vp = make(q.shape[0], H * D), make(blocks, H, block, D), make(blocks, H, block, self.vdim)
+        table = make(ctx.cache.max_slots, -(-ctx.max_new_tokens // block), dtype=torch.int32)
+        ops.latent_place(q, kv, shared, qp, kp, vp, table, ctx.token_seq, ctx.token_pos, ctx.cu_seqlens, ctx.slot_ids,
+                         rotary.inv_freq if rotary else None, rotary.rope_dim if rotary else 0, rotary.amplitude if rotary else 1.0, H, self.dim,
+                         self.rot, self.vdim)
+        ops.attention_prefill_tc_kv(out, qp, kp, vp, table, ctx.cu_seqlens, ctx.slot_ids, ctx.kv_lens, ctx.num_seqs, ctx.max_new_tokens, H, H, D,
+                                    self.vdim, self.scale, self.window, self.sink is not None, ops.device_status(q.device), self.sink)
 
     def attend(self, out, q, plane, table, ctx) -> None:
         # bfloat16 with rows in pieces of 16: the tensor-core kernel; 32-bit and odd sizes: the general CUDA-core kernel

@@ -91,6 +91,8 @@ MIXERS = {
     "pieces of 16": (96, _m(6, 16, 16, 16, 48, 32, 0.9, 65)),
     "pieces of 16, 20 heads": (96, _m(20, 48, 16, 48, 32, 80, 0.4)),
     "64 + 64": (128, _m(4, 64, 64, 64, 96, 64, 0.3, 64)),
+    "64 + 32, values of 128": (96, _m(5, 64, 32, 128, 48, 96, 0.3, 100)),
+    "40 + 24, values of 64": (64, _m(3, 40, 24, 64, 40, 48, 0.4)),
     "128 + 64": (128, _m(2, 128, 64, 128, 64, 256, 0.2, 190)),
     "80 + 48, values of 112": (80, _m(3, 80, 48, 112, 40, 64, 0.3, 130, 50.0)),
     "32 + 32, no window": (64, _m(8, 32, 32, 32, 24, 48, 0.6)),
@@ -158,7 +160,7 @@ CUTS = (("prompt", lambda q: [[(0, q + 1)]]), ("decoded", lambda q: [[(0, q)], [
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("name", ["odd", "pieces of 16", "128 + 64", "32 + 32, no window"])
+@pytest.mark.parametrize("name", ["odd", "pieces of 16", "64 + 64", "128 + 64", "40 + 24, values of 64"])
 @pytest.mark.parametrize("query, key", [(299, 0), (299, 1), (299, 63), (299, 64), (300, 127), (300, 128), (319, 255), (319, 256), (319, 319), (320, 319),
                                         (256, 255), (128, 0), (127, 64)])
 def test_far_keys_and_block_borders(name, dtype, query, key):
@@ -179,7 +181,7 @@ def test_far_keys_and_block_borders(name, dtype, query, key):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("name", ["odd", "pieces of 16", "128 + 64"])
+@pytest.mark.parametrize("name", ["odd", "pieces of 16", "64 + 32, values of 128"])
 @pytest.mark.parametrize("window", [2, 63, 64, 65, 128, 129, 200])
 def test_window_edges(name, dtype, window):
     """The key `window` - 1 places back is seen, the one `window` back is not, wherever the edge falls."""
@@ -201,7 +203,7 @@ def test_window_edges(name, dtype, window):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("name", ["odd", "pieces of 16, 20 heads", "128 + 64", "32 + 32, no window"])
+@pytest.mark.parametrize("name", ["odd", "pieces of 16, 20 heads", "128 + 64", "64 + 64", "40 + 24, values of 64", "32 + 32, no window"])
 def test_sinks_of_every_size(name, dtype):
     """Sinks far above, among and far below the scores, another one a head; whole prompts, whose first rows have few keys beside
     the sink, and decode steps with and without splits.  Without a sink the result is another."""
@@ -228,7 +230,7 @@ def test_sinks_of_every_size(name, dtype):
         helpers.assert_close(got.numpy(), none.numpy(), _name(dtype), f"{name} without a sink", factor=2.0)
 
 
-@pytest.mark.parametrize("name", ["odd", "pieces of 16", "128 + 64"])
+@pytest.mark.parametrize("name", ["odd", "pieces of 16", "64 + 64", "128 + 64"])
 def test_many_sequences_decode_together_and_alone(name):
     """Decode steps of more sequences than one, with lengths from 1 to several splits, against each of them alone: which other
     rows are in the batch does not show beyond rounding.  Prompts likewise."""
