@@ -285,12 +285,12 @@ def sosepel_config(size: str, layers: int):
                                         embedding=dict(scale=6.0, bigram=dict(buckets=z["buckets"], mul_prev=4099, mul_cur=61))))
 
 
-# Gomerax: latent attention with a latent vector of the queries, in a window, with sinks (head sizes, latent width and window as Pulenex
-# has them); feed-forwards as Sosepel's (its dense ones have a gate: half the width)
+# Gomerax: latent attention with a latent vector of the queries, in a window, with sinks (m: as many multiplications a (query, key) pair
+# as Pulenex' heads take, in twice the heads of half the size); feed-forwards as Sosepel's (its dense ones have a gate: half the width)
 GOMERAX_SIZES = {
     "s": dict(width=1024, vocab=32768, heads=8, dim=64, rot_dim=32, vdim=64, q_rank=512, kv_rank=256, window=1024, dense_ff=3776, experts=16, top=4,
               groups=4, keep=2, ff=512, shared=1024, dense=DESIGN_SIZES["s"]["dense"]),
-    "m": dict(width=2048, vocab=65536, heads=16, dim=128, rot_dim=64, vdim=128, q_rank=1024, kv_rank=512, window=2048, dense_ff=7552, experts=32, top=4,
+    "m": dict(width=2048, vocab=65536, heads=32, dim=64, rot_dim=32, vdim=64, q_rank=768, kv_rank=256, window=2048, dense_ff=7552, experts=32, top=4,
               groups=8, keep=4, ff=1024, shared=2048, dense=DESIGN_SIZES["m"]["dense"]),
 }
 

@@ -220,6 +220,8 @@ inline int merge_threads(int dv) { return dv > 256 ? 256 : (dv > 128 ? 128 : 64)
 // out[row] = sum_s acc_s * exp(m_s - M) / sum_s l_s * exp(m_s - M), chunks in index order.
 template <typename T>
 __global__ void attention_merge_kernel(AttnParams p, int total_tokens) {
+    pdl_wait();
+    pdl_launch_dependents();
     const int row = blockIdx.x;  // (token * nh + head) * maps + map
     const int t = row / (p.nh * p.maps);
     // the batch row of token t: cu_seqlens is short, a linear scan is enough
@@ -322,7 +324,7 @@ int hymt2_attention_merge_launch(void* out, int dtype, const int* cu_seqlens, co
     p.out = out; p.cu_seqlens = cu_seqlens; p.slot_ids = slot_ids; p.kv_lens = kv_lens;
     p.part_acc = part_acc; p.part_ml = part_ml; p.nh = nh; p.d = d; p.dv = d; p.window = window; p.maps = 1;
     p.split_keys = split_keys; p.max_splits = max_splits;
-    HYMT2_DISPATCH_DTYPE(dtype, T, (attention_merge_kernel<T><<<tokens * nh, merge_threads(d), 0, stream>>>(p, tokens)));
+    HYMT2_DISPATCH_DTYPE(dtype, T, (launch_pdl(attention_merge_kernel<T>, dim3(tokens * nh), dim3(merge_threads(d)), 0, stream, p, tokens)));
     return hymt2_check_launch("attention_merge");
 }
 

@@ -42,7 +42,7 @@ struct LatentPrepParams {
 };
 
 template <typename T>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(512)
 latent_prep_kernel(LatentPrepParams p) {
     extern __shared__ float smem[];   // [rot_dims / 2][2] cosine, sine; then 33 floats for the sum
     float* cs = smem;
@@ -61,15 +61,25 @@ latent_prep_kernel(LatentPrepParams p) {
         cs[2 * i] = c * p.amplitude;
         cs[2 * i + 1] = sn * p.amplitude;
     }
-    // the latent vector's sum of squares (block_sum synchronises, which also publishes cs)
+    // the latent vectors' sums of squares (block_sum synchronises, which also publishes cs)
     const T* lat = row + p.q_cols;
-    float ss = 0.f;
+    float ss = 0.f, qs = 0.f;
+    if (p.cq_out)
+        for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) {
+            const float v = to_float(row[i]);
+            qs = fmaf(v, v, qs);
+        }
     if (p.cache || p.rows_out)      // (a projection without a compressed row of its own is never read behind its queries)
         for (int i = threadIdx.x; i < p.rank; i += blockDim.x) {
             const float v = to_float(lat[i]);
             ss = fmaf(v, v, ss);
         }
     ss = block_sum(ss, scratch);
+    if (p.cq_out) {   // the compressed query: normed as the latent vector is; there are no heads' queries yet
+        const float scale = 1.0f / sqrtf(block_sum(qs, scratch) / (float)p.q_rank + p.eps);
+        T* o = (T*)p.cq_out + (size_t)t * p.q_rank;
+        for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) o[i] = from_float<T>(to_float(row[i]) * scale * p.q_gain[i]);
+    }
     const int dl = p.rank + p.rot;
     T* dst = nullptr;    // the token's cache row
     if (p.cache && slot >= 0) {
@@ -95,17 +105,6 @@ latent_prep_kernel(LatentPrepParams p) {
             if (dst) dst[p.rank + i] = kr[i];
             if (dst2) dst2[p.rank + i] = kr[i];
         }
-    }
-    if (p.cq_out) {   // the compressed query: normed as the latent vector is; there are no heads' queries yet
-        float qs = 0.f;
-        for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) {
-            const float v = to_float(row[i]);
-            qs = fmaf(v, v, qs);
-        }
-        const float scale = 1.0f / sqrtf(block_sum(qs, scratch) / (float)p.q_rank + p.eps);
-        T* o = (T*)p.cq_out + (size_t)t * p.q_rank;
-        for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) o[i] = from_float<T>(to_float(row[i]) * scale * p.q_gain[i]);
-        return;
     }
     // the heads' rotated query parts
     const int per_head = half + (p.rot - p.rot_dims);
@@ -202,6 +201,88 @@ latent_place_kernel(LatentPlaceParams p) {
     }
 }
 
+// A few tokens' queries (a decode step) into the compressed space, and their rotation:
+//   q_out[t, h, n] = sum_k uk_t[h, n, k] * q[t, h, k] for n < rank, k < dim;   q_out[t, h, rank ..] = the head's rotated part, turned
+// One launch, 16 tokens a block.  L lanes hold a weight row of `dim` entries, 16 bytes each, and take every token's entries past it; the weights are
+// asked for before the kernel in front is waited for.  A head's last block does its rotation.
+constexpr int ABSORB_THREADS = 256, ABSORB_COLS = 2, ABSORB_TOKENS = 16, ABSORB_MAX_TOKENS = 128;   // of a block; of a launch
+
+struct LatentAbsorbParams {
+    const void* q;       // [T, ldq]: head h's dim + rot entries at column h * (dim + rot)
+    const void* uk_t;    // [heads, rank, dim]
+    void* q_out;         // [T, heads * (rank + rot)]
+    const int* token_pos;
+    const float* inv_freq;
+    long ldq;
+    int tokens, heads, dim, rot, rank, rot_dims;
+    float amplitude;
+};
+
+template <typename T, int L>
+__global__ void __launch_bounds__(ABSORB_THREADS)
+latent_absorb_kernel(LatentAbsorbParams p) {
+    constexpr int V = 16 / sizeof(T), GROUPS = ABSORB_THREADS / L;
+    const int h = blockIdx.y, dl = p.rank + p.rot;
+    const T* q = (const T*)p.q + (size_t)h * (p.dim + p.rot);
+    T* out = (T*)p.q_out + (size_t)h * dl;
+    const size_t out_ld = (size_t)p.heads * dl;
+    const int t0 = blockIdx.z * ABSORB_TOKENS, t1 = min(p.tokens, t0 + ABSORB_TOKENS);
+    if (blockIdx.x == gridDim.x - 1) {
+        pdl_wait();
+        pdl_launch_dependents();
+        const int half = p.rot_dims / 2, per = half + (p.rot - p.rot_dims);
+        for (int item = threadIdx.x; item < (t1 - t0) * per; item += blockDim.x) {
+            const int t = t0 + item / per, i = item % per;
+            const T* src = q + (size_t)t * p.ldq + p.dim;
+            T* dst = out + (size_t)t * out_ld + p.rank;
+            if (i < half) {
+                float sn, c;
+                sincosf((float)p.token_pos[t] * p.inv_freq[i], &sn, &c);
+                c *= p.amplitude;
+                sn *= p.amplitude;
+                const float a = to_float(src[2 * i]), b = to_float(src[2 * i + 1]);
+                dst[2 * i] = from_float<T>(a * c - b * sn);
+                dst[2 * i + 1] = from_float<T>(b * c + a * sn);
+            } else {
+                const int e = p.rot_dims + (i - half);
+                dst[e] = src[e];
+            }
+        }
+        return;
+    }
+    const int lane = threadIdx.x % L, group = threadIdx.x / L, k = lane * V;
+    const bool k_ok = k < p.dim;
+    int n[ABSORB_COLS];
+    float wv[ABSORB_COLS][V];
+#pragma unroll
+    for (int c = 0; c < ABSORB_COLS; c++) {
+        n[c] = (blockIdx.x * ABSORB_COLS + c) * GROUPS + group;
+        uint4 raw = make_uint4(0, 0, 0, 0);
+        if (k_ok && n[c] < p.rank) raw = __ldg(reinterpret_cast<const uint4*>((const T*)p.uk_t + ((size_t)h * p.rank + n[c]) * p.dim + k));
+        const T* wt = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+        for (int i = 0; i < V; i++) wv[c][i] = to_float(wt[i]);
+    }
+    pdl_wait();
+    pdl_launch_dependents();
+#pragma unroll 4
+    for (int t = t0; t < t1; t++) {
+        uint4 raw = make_uint4(0, 0, 0, 0);
+        if (k_ok) raw = *reinterpret_cast<const uint4*>(q + (size_t)t * p.ldq + k);
+        const T* qt = reinterpret_cast<const T*>(&raw);
+        float acc[ABSORB_COLS];
+#pragma unroll
+        for (int c = 0; c < ABSORB_COLS; c++) {
+            acc[c] = 0.f;
+#pragma unroll
+            for (int i = 0; i < V; i++) acc[c] = fmaf(to_float(qt[i]), wv[c][i], acc[c]);
+#pragma unroll
+            for (int o = L / 2; o > 0; o >>= 1) acc[c] += __shfl_xor_sync(0xffffffffu, acc[c], o);
+            if (lane == 0 && n[c] < p.rank) out[(size_t)t * out_ld + n[c]] = from_float<T>(acc[c]);
+        }
+    }
+}
+
 }  // namespace
 
 HYMT2_API int hymt2_latent_prep(const void* proj, long ldp, int q_cols, void* q_out, void* rows_out, void* cache, int dtype,
@@ -222,7 +303,8 @@ HYMT2_API int hymt2_latent_prep(const void* proj, long ldp, int q_cols, void* q_
     p.table_stride = table_stride; p.block_tokens = block_tokens; p.heads = heads; p.dim = dim; p.rot = rot; p.rank = rank;
     p.rot_dims = rot_dims; p.eps = eps; p.amplitude = amplitude;
     const size_t smem = sizeof(float) * ((size_t)rot_dims + 33);
-    HYMT2_DISPATCH_DTYPE(dtype, T, launch_pdl(latent_prep_kernel<T>, dim3(tokens), dim3(128), smem, stream, p));
+    const int threads = tokens <= 64 ? 512 : 128;   // (few tokens: the time is one block's chain of passes)
+    HYMT2_DISPATCH_DTYPE(dtype, T, launch_pdl(latent_prep_kernel<T>, dim3(tokens), dim3(threads), smem, stream, p));
     return hymt2_check_launch("latent_prep");
 }
 
@@ -245,4 +327,31 @@ HYMT2_API int hymt2_latent_place(const void* q, long ldq, const void* kv, long l
     p.amplitude = amplitude;
     launch_pdl(latent_place_kernel, dim3(tokens), dim3(256), sizeof(float) * (size_t)rot_dims, stream, p);
     return hymt2_check_launch("latent_place");
+}
+
+// Whether latent_absorb takes heads of `dim` unrotated entries (they fill at most a warp's 16-byte pieces) for this many tokens.
+HYMT2_API int hymt2_latent_absorb_supported(int dtype, int tokens, int dim, int rot) {
+    const int v = dtype == HYMT2_BF16 ? 8 : 4;
+    return tokens <= ABSORB_MAX_TOKENS && dim > 0 && dim <= 32 * v && dim % v == 0 && rot % v == 0;
+}
+
+HYMT2_API int hymt2_latent_absorb(void* q_out, const void* q, long ldq, const void* uk_t, int dtype, const int* token_pos, const float* inv_freq,
+                                  int rot_dims, float amplitude, int tokens, int heads, int dim, int rot, int rank, cudaStream_t stream) {
+    if (tokens == 0) return HYMT2_OK;
+    HYMT2_REQUIRE(hymt2_latent_absorb_supported(dtype, tokens, dim, rot) && heads > 0 && heads <= 65535 && rank > 0, "latent_absorb: %d tokens with heads of %d + %d entries are not taken", tokens, dim, rot);
+    HYMT2_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= rot && (rot_dims == 0 || inv_freq), "latent_absorb: %d rotated entries of %d", rot_dims, rot);
+    HYMT2_DISPATCH_DTYPE(dtype, T, {
+        constexpr int v = 16 / sizeof(T);
+        HYMT2_REQUIRE(ldq % v == 0 && ((uintptr_t)q | (uintptr_t)uk_t) % 16 == 0, "latent_absorb: operands must be 16-byte aligned");
+        LatentAbsorbParams p{q, uk_t, q_out, token_pos, inv_freq, ldq, tokens, heads, dim, rot, rank, rot_dims, amplitude};
+        auto run = [&](auto kernel, int lanes) {
+            const int cols = ABSORB_THREADS / lanes * ABSORB_COLS;
+            launch_pdl(kernel, dim3((rank + cols - 1) / cols + 1, heads, (tokens + ABSORB_TOKENS - 1) / ABSORB_TOKENS), dim3(ABSORB_THREADS), 0, stream, p);
+        };
+        if (dim <= 4 * v) run(latent_absorb_kernel<T, 4>, 4);
+        else if (dim <= 8 * v) run(latent_absorb_kernel<T, 8>, 8);
+        else if (dim <= 16 * v) run(latent_absorb_kernel<T, 16>, 16);
+        else run(latent_absorb_kernel<T, 32>, 32);
+    });
+    return hymt2_check_launch("latent_absorb");
 }

@@ -1123,6 +1123,42 @@ def latent_attention_mma(out: torch.Tensor, q: torch.Tensor, cache_plane: torch.
                                              _ptr(status), _stream()), "latent_attention_mma", 2 if split_keys > 0 else 1)
 
 
+def latent_decode_supported(dtype: torch.dtype, d: int, dv: int, block_tokens: int) -> bool:
+    """Whether the decode kernel of the shared-vector attention takes these sizes (bfloat16, rows in pieces of 16)."""
+    if dtype != torch.bfloat16:
+        return False
+    key = ("decode", d, dv, block_tokens)
+    hit = _mma_ok.get(key)
+    if hit is None:
+        hit = _mma_ok[key] = bool(_lib().hymt2_latent_decode_supported(c_int(d), c_int(dv), c_int(block_tokens)))
+    return hit
+
+
+def latent_decode(out: torch.Tensor, q: torch.Tensor, cache_plane: torch.Tensor, block_table: torch.Tensor, cu_seqlens: torch.Tensor,
+                  slot_ids: torch.Tensor, kv_lens: torch.Tensor, nh: int, d: int, dv: int, scale: float, window: int = 0, split_keys: int = 0,
+                  max_splits: int = 0, part_acc: torch.Tensor | None = None, part_ml: torch.Tensor | None = None,
+                  status: torch.Tensor | None = None, sink: torch.Tensor | None = None) -> None:
+    """latent_attention_mma for a decode step (one new token a sequence): the same sums, the keys streamed through a ring of tiles."""
+    if status is None:
+        status = device_status(out.device)
+    _f32(sink, "sink", nh)
+    _need(out, "out", torch.bfloat16, 2); _need(q, "q", torch.bfloat16, 2); _need(cache_plane, "cache_plane", torch.bfloat16, 4)
+    rows = out.shape[0]
+    if out.shape[1] != nh * dv or q.shape != (rows, nh * d) or cache_plane.shape[1] != 1 or cache_plane.shape[3] != d:
+        raise KernelError(f"latent_decode: shapes out {tuple(out.shape)} q {tuple(q.shape)} cache {tuple(cache_plane.shape)}")
+    _need(block_table, "block_table", torch.int32, 2)
+    for t, n in ((cu_seqlens, "cu_seqlens"), (slot_ids, "slot_ids"), (kv_lens, "kv_lens")):
+        _need(t, n, torch.int32, 1)
+    if split_keys > 0:
+        _need(part_acc, "part_acc", torch.float32); _need(part_ml, "part_ml", torch.float32)
+        if part_acc.numel() < rows * nh * max_splits * dv or part_ml.numel() < rows * nh * max_splits * 2:
+            raise KernelError("latent_decode: the split scratch is too small")
+    _check(_lib().hymt2_latent_decode(_ptr(out), _ptr(q), _ptr(cache_plane), _ptr(block_table), c_int(block_table.stride(0)), c_int(cache_plane.shape[2]),
+                                      _ptr(cu_seqlens), _ptr(slot_ids), _ptr(kv_lens), c_int(rows), c_int(nh), c_int(d), c_int(dv), c_float(scale),
+                                      c_int(window), _ptr(sink), c_int(split_keys), c_int(max_splits), _ptr(part_acc), _ptr(part_ml), _ptr(status),
+                                      _stream()), "latent_decode", 2 if split_keys > 0 else 1)
+
+
 SKINNY_MAX_ROWS = 16
 
 
@@ -1148,6 +1184,29 @@ def latent_attention_expanded_supported(dtype: torch.dtype, dim: int, rot: int, 
     if hit is None:
         hit = _mma_ok[key] = bool(_lib().hymt2_latent_attention_expanded_supported(c_int(dim), c_int(rot), c_int(dv)))
     return hit
+
+
+def latent_absorb_supported(dtype: torch.dtype, tokens: int, dim: int, rot: int) -> bool:
+    key = ("absorb", dtype, tokens, dim, rot)
+    hit = _mma_ok.get(key)
+    if hit is None:
+        hit = _mma_ok[key] = bool(_lib().hymt2_latent_absorb_supported(c_int(dtype_code(dtype)), c_int(tokens), c_int(dim), c_int(rot)))
+    return hit
+
+
+def latent_absorb(q_out: torch.Tensor, q: torch.Tensor, uk_t: torch.Tensor, token_pos: torch.Tensor, inv_freq: torch.Tensor | None, rot_dims: int,
+                  amplitude: float, rot: int) -> None:
+    """Few tokens: q_out[t, h] = [uk_t[h] @ q[t, h, :dim] | the rot entries behind them, turned]; q [T, >= heads * (dim + rot)] (not
+    rotated), uk_t [heads, rank, dim], q_out [T, heads * (rank + rot)]."""
+    ldq = _rows_view(q, "q")
+    _need(uk_t, "uk_t", q.dtype, 3); _need(q_out, "q_out", q.dtype, 2); _need(token_pos, "token_pos", torch.int32, 1)
+    _f32(inv_freq, "inv_freq", rot_dims // 2)
+    H, rank, dim = uk_t.shape
+    if q_out.shape != (q.shape[0], H * (rank + rot)) or q.shape[1] < H * (dim + rot):
+        raise KernelError(f"latent_absorb: shapes q {tuple(q.shape)} uk_t {tuple(uk_t.shape)} q_out {tuple(q_out.shape)}")
+    _check(_lib().hymt2_latent_absorb(_ptr(q_out), _ptr(q), c_long(ldq), _ptr(uk_t), c_int(dtype_code(q.dtype)), _ptr(token_pos), _ptr(inv_freq),
+                                      c_int(rot_dims), c_float(amplitude), c_int(q.shape[0]), c_int(H), c_int(dim), c_int(rot), c_int(rank), _stream()),
+           "latent_absorb")
 
 
 LATENT_PLACE_BLOCK = 64    # tokens of a block that latent_place fills

@@ -38,8 +38,8 @@ from .linear import Linear, compute_form, matmul_batched
 
 EXPAND_FROM_TOKENS = 32   # prompts from this length on are worth one more product (keys and values per head)
 SPLIT_KEYS = 256     # decode: keys per partial, a constant so that the cut depends on nothing else
-SPLIT_KEYS_TC = 128  # the same for the tensor-core kernel, whose blocks are few and large: two tiles of keys each (one tile each
-                     # measured slower: twice the partials to write and fold)
+SPLIT_KEYS_TC = 256  # the same for the tensor-core kernel of decode steps: four tiles of keys (fewer would mean more partials to
+                     # write and fold)
 
 
 class LatentAttention:
@@ -145,11 +145,16 @@ class LatentAttention:
             self._gate_and_project(out, proj, residual, ctx, store)
             return
         q = torch.empty((T, H * dl), dtype=proj.dtype, device=proj.device)
-        source = self._prepare(proj, q, rotary, plane if slot.writes else None, table, ctx)
-        # q[t, h, :kv_rank] = W_uk[h]^T q_h[:dim]
-        ops.tag = "q_absorb"
-        matmul_batched(q, source, self.uk_t, self.dim + self.rot, dl)
-        ops.tag = None
+        # q[t, h] = [W_uk[h]^T q_h[:dim] | the rotated part]: few tokens, one kernel for both
+        fused = proj.dtype == self.uk_t.dtype and ops.latent_absorb_supported(proj.dtype, T, self.dim, self.rot)
+        source = self._prepare(proj, q, rotary, plane if slot.writes else None, table, ctx, turn_queries=not fused)
+        if fused:
+            ops.latent_absorb(q, source, self.uk_t, ctx.token_pos, rotary.inv_freq if rotary else None, rotary.rope_dim if rotary else 0,
+                              rotary.amplitude if rotary else 1.0, self.rot)
+        else:
+            ops.tag = "q_absorb"
+            matmul_batched(q, source, self.uk_t, self.dim + self.rot, dl)
+            ops.tag = None
         mixed = torch.empty((T, H * self.rank), dtype=q.dtype, device=q.device)
         self.attend(mixed, q, plane, table, ctx)
         out = torch.empty((T, H * self.vdim), dtype=q.dtype, device=q.device)
@@ -164,7 +169,11 @@ class LatentAttention:
         `turn_queries` they are left to whoever reads them."""
         table_args = (table, ctx.cache.block_tokens, ctx.token_seq, ctx.token_pos, ctx.slot_ids, self.c_gain)
         turn_args = (rotary.inv_freq if rotary else None, rotary.rope_dim if rotary else 0, rotary.amplitude if rotary else 1.0, self.eps)
+        if not turn_queries:
+            q_out = None
         if self.q_rank is None:
+            if not turn_queries and plane is None and rows_out is None:
+                return proj            # (a reader of another run's rows, whose queries are left alone)
             ops.latent_prep(proj, self.q_cols, q_out, plane, *table_args, *turn_args, self.heads if turn_queries else 0, self.dim, self.rot, self.rank, rows_out=rows_out)
             return proj
         cq = torch.empty((proj.shape[0], self.q_rank), dtype=proj.dtype, device=proj.device)
@@ -219,16 +228,21 @@ class LatentAttention:
                                     self.vdim, self.scale, self.window, self.sink is not None, ops.device_status(q.device), self.sink)
 
     def attend(self, out, q, plane, table, ctx) -> None:
-        # bfloat16 with rows in pieces of 16: the tensor-core kernel; 32-bit and odd sizes: the general CUDA-core kernel
+        # bfloat16 with rows in pieces of 16: the tensor-core kernels; 32-bit and odd sizes: the general CUDA-core kernel
         run, keys = ops.attention_shared_vector, SPLIT_KEYS
-        if ops.latent_attention_mma_supported(out.dtype, self.rank + self.rot, self.rank, plane.shape[2]):
-            run, keys = ops.latent_attention_mma, SPLIT_KEYS_TC
+        stream = ctx.decode and ops.latent_decode_supported(out.dtype, self.rank + self.rot, self.rank, plane.shape[2])
+        if stream or ops.latent_attention_mma_supported(out.dtype, self.rank + self.rot, self.rank, plane.shape[2]):
+            run, keys = ops.latent_attention_mma, SPLIT_KEYS_TC   # (the fragment kernel for prompts' portions never splits)
         split, max_splits, acc, ml = 0, 0, None, None
         if ctx.decode and ctx.max_kv_len > keys:
             split = keys
             max_splits = -(-ctx.max_kv_len // keys)
             acc = torch.empty(ctx.num_tokens * self.heads * max_splits * self.rank, dtype=torch.float32, device=out.device)
             ml = torch.empty(ctx.num_tokens * self.heads * max_splits * 2, dtype=torch.float32, device=out.device)
+        if stream:
+            ops.latent_decode(out, q, plane, table, ctx.cu_seqlens, ctx.slot_ids, ctx.kv_lens, self.heads, self.rank + self.rot, self.rank,
+                              self.scale, self.window, split, max_splits, acc, ml, sink=self.sink)
+            return
         run(out, q, plane, table, ctx.cu_seqlens, ctx.slot_ids, ctx.kv_lens, ctx.num_seqs, ctx.max_new_tokens, self.heads,
             self.rank + self.rot, self.rank, self.scale, self.window, split, max_splits, acc, ml, sink=self.sink)
 
