@@ -65,12 +65,15 @@ def layer_runs(config: dict) -> list:
 
 
 # -- latent attention ---------------------------------------------------------------------------------
-def turn(v: torch.Tensor, position: int, dims: int, base: float) -> torch.Tensor:
-    """The first `dims` entries of v [.., n] in neighbouring pairs, pair i by position * base^(-2i/dims)."""
+def turn(v: torch.Tensor, position, dims: int, base: float) -> torch.Tensor:
+    """The first `dims` entries of v [.., n] in neighbouring pairs, pair i by position * base^(-2i/dims).  `position`: one number, or
+    one for each v[t]."""
     out = v.clone()
+    p = torch.as_tensor(position, dtype=v.dtype)
+    p = p.reshape(-1, *[1] * (v.dim() - 2)) if p.dim() else p
     for i in range(dims // 2):
-        a = position * base ** (-2.0 * i / dims)
-        c, s = math.cos(a), math.sin(a)
+        a = p * base ** (-2.0 * i / dims)
+        c, s = torch.cos(a), torch.sin(a)
         out[..., 2 * i] = v[..., 2 * i] * c - v[..., 2 * i + 1] * s
         out[..., 2 * i + 1] = v[..., 2 * i + 1] * c + v[..., 2 * i] * s
     return out
@@ -90,17 +93,14 @@ def queries(h: torch.Tensor, w: dict, p: str, m: dict, eps: float) -> torch.Tens
     """[T, heads, dim + rot_dim], the last rot_dim of a head turned."""
     T = h.shape[0]
     c = norm_plain(h @ w[p + "dq"].T, w[p + "dq.norm"], eps)
-    q = (c @ w[p + "uq"].T).view(T, m["heads"], m["dim"] + m["rot_dim"]).clone()
-    for t in range(T):
-        q[t, :, m["dim"]:] = turn(q[t, :, m["dim"]:], t, m["rot"]["dims"], m["rot"]["base"])
-    return q
+    q = (c @ w[p + "uq"].T).view(T, m["heads"], m["dim"] + m["rot_dim"])
+    return torch.cat([q[..., :m["dim"]], turn(q[..., m["dim"]:], list(range(T)), m["rot"]["dims"], m["rot"]["base"])], dim=-1)
 
 
 def compressed(h: torch.Tensor, w: dict, p: str, m: dict, eps: float):
     """The latent vectors [T, kv_rank] and the shared rotated key parts [T, rot_dim]."""
     z = h @ w[p + "dkv"].T
-    k = z[:, m["kv_rank"]:]
-    k = torch.stack([turn(k[t], t, m["rot"]["dims"], m["rot"]["base"]) for t in range(h.shape[0])])
+    k = turn(z[:, m["kv_rank"]:], list(range(h.shape[0])), m["rot"]["dims"], m["rot"]["base"])
     return norm_plain(z[:, :m["kv_rank"]], w[p + "dkv.norm"], eps), k
 
 
