@@ -32,6 +32,7 @@ struct LatentDecodeParams {
     float* part_ml;       // [rows * nh, splits, 2]
     const float* sink;    // [nh] or null
     int table_stride, nh, d, dv, window, split_keys, max_splits, stages;
+    int grid_splits;      // chunks that blocks are launched for: all, or with a window as many as it can touch
     float scale;
 };
 
@@ -74,13 +75,15 @@ latent_decode_kernel(LatentDecodeParams p) {
     bf16* Ps = Ks + (size_t)p.stages * KEYS * ld;                     // [2][ROWS][P_LD]
     float* red = reinterpret_cast<float*>(Ps + 2 * ROWS * P_LD);      // [2][WARPS][ROWS]
 
-    const int b = blockIdx.y / p.max_splits, split = blockIdx.y % p.max_splits, h0 = blockIdx.x * ROWS;
+    const int b = blockIdx.y / p.grid_splits, h0 = blockIdx.x * ROWS;
     const int slot = p.slot_ids[b];
     if (slot < 0) return;
     const int kv_len = p.kv_lens[b], pos = kv_len - 1;
     const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
-    int begin = lo, end = kv_len;
+    int begin = lo, end = kv_len, split = 0;
     if (p.split_keys > 0) {
+        split = lo / p.split_keys + blockIdx.y % p.grid_splits;
+        if (split >= p.max_splits) return;
         begin = max(begin, split * p.split_keys);
         end = min(end, (split + 1) * p.split_keys);
     }
@@ -302,14 +305,16 @@ HYMT2_API int hymt2_latent_decode(void* out, const void* q, const void* cache, c
     p.q = (const bf16*)q; p.out = (bf16*)out; p.cache = (const bf16*)cache; p.block_table = block_table; p.slot_ids = slot_ids; p.kv_lens = kv_lens;
     p.part_acc = part_acc; p.part_ml = part_ml; p.sink = sink; p.table_stride = table_stride; p.nh = nh; p.d = d; p.dv = dv; p.window = window;
     p.split_keys = split_keys; p.max_splits = split_keys > 0 ? max_splits : 1; p.scale = scale;
-    HYMT2_REQUIRE((long)rows * p.max_splits <= 65535, "latent_decode: grid too large (%d rows x %d splits)", rows, p.max_splits);
+    p.grid_splits = p.max_splits;
+    if (split_keys > 0 && window > 0 && (window - 1) / split_keys + 2 < p.grid_splits) p.grid_splits = (window - 1) / split_keys + 2;
+    HYMT2_REQUIRE((long)rows * p.grid_splits <= 65535, "latent_decode: grid too large (%d rows x %d splits)", rows, p.max_splits);
     const int block_rows = nh <= 16 ? 16 : 32;
     p.stages = 2;
     // as many stages as leave room for a second block beside this one; else as many as fit
     while (p.stages < 4 && (smem_bytes(block_rows, d, p.stages + 1) <= SMEM_LIMIT / 2 || (smem_bytes(block_rows, d, p.stages) > SMEM_LIMIT / 2 &&
            smem_bytes(block_rows, d, p.stages + 1) <= SMEM_LIMIT))) p.stages++;
     const size_t smem = smem_bytes(block_rows, d, p.stages);
-    const dim3 grid((nh + block_rows - 1) / block_rows, rows * p.max_splits);
+    const dim3 grid((nh + block_rows - 1) / block_rows, rows * p.grid_splits);
     auto launch = [&](auto kernel) -> int {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) { hymt2_set_error("latent_decode: %s", cudaGetErrorString(e)); return HYMT2_ERR_LAUNCH; }
