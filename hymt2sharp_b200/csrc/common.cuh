@@ -139,16 +139,6 @@ __device__ __forceinline__ float glu_at(const GluRule& r, float g, float u, int 
     u = fminf(fmaxf(u, -r.limit), r.limit);
     return g / (1.0f + expf(-r.alpha * g)) * (u + 1.0f);
 }
-// V neighbouring features from n on (those from N on are computed without a bias and never used); the rule is looked at once
-template <int V> __device__ __forceinline__ void glu_pack(const GluRule& r, const float* g, const float* u, float* o, int n, int N) {
-    if (r.kind == GLU_SILU && !r.bias) {
-#pragma unroll
-        for (int i = 0; i < V; i++) o[i] = silu_mul(g[i], u[i]);
-        return;
-    }
-#pragma unroll
-    for (int i = 0; i < V; i++) o[i] = n + i < N ? glu_at(r, g[i], u[i], n + i, N) : 0.f;
-}
 
 // V neighbouring elements in one access of V * sizeof(T) bytes (the caller has checked the alignment).
 template <typename T, int V> struct Pack { T v[V]; };

@@ -38,13 +38,21 @@ constexpr int EPILOGUE_GROUPS = 2;        // persistent kernel: groups of four e
 constexpr int NUM_THREADS = 64 + 128 * EPILOGUE_GROUPS;   // warp 0 TMA, warp 1 MMAs, then the epilogue groups
 // one-tile kernel: with few accumulator columns a second warp issues MMAs too (warp 6), see ISSUERS in the kernel
 __host__ __device__ constexpr int tile_issuers(int bn, int epi) {
-    return bn * (epi == 2 ? 2 : 1) <= 32 ? 2 : 1;   // measured: no gain with 64 columns and more
+    return bn * (epi == 2 || epi == 4 ? 2 : 1) <= 32 ? 2 : 1;   // measured: no gain with 64 columns and more
 }
 __host__ __device__ constexpr int tile_threads(int bn, int epi) { return tile_issuers(bn, epi) > 1 ? 224 : 192; }
 constexpr int A_TILE_BYTES = TILE_M * BLOCK_K * 2;
 constexpr int PERSISTENT_BN = 256;   // tile width of the persistent kernel for many tokens
 
-enum { EPI_STORE = 0, EPI_ACCUMULATE = 1, EPI_SWIGLU = 2, EPI_ROPE_KV = 3 };
+// EPI_GLU is EPI_SWIGLU with another rule than silu(gate) * up, or with biases: an instance of its own, so that the plain one keeps
+// its registers (callers always say EPI_SWIGLU; the launch picks the instance by the rule).
+enum { EPI_STORE = 0, EPI_ACCUMULATE = 1, EPI_SWIGLU = 2, EPI_ROPE_KV = 3, EPI_GLU = 4 };
+__host__ __device__ constexpr bool is_gated(int epi) { return epi == EPI_SWIGLU || epi == EPI_GLU; }
+// what a gate and an up entry of output feature n become
+template <int EPI> __device__ __forceinline__ float gated_at(const GluRule& r, float g, float u, int n, int N) {
+    if constexpr (EPI == EPI_GLU) return n < N ? glu_at(r, g, u, n, N) : 0.f;
+    else return silu_mul(g, u);
+}
 
 // What the EPI_ROPE_KV epilogue needs: the product is the fused q/k/v projection of a few tokens with heads of 128 (one
 // tile of 128 output features = one head), and the epilogue does what the rotation kernel would do next
@@ -132,7 +140,7 @@ struct GemmTcParams {
     const int* tile_group = nullptr;
     long group_rows = 0;
     int act = 0;             // store epilogue: 1 = the square of relu on the way out
-    GluRule glu;             // EPI_SWIGLU: what a gate and an up entry become
+    GluRule glu;             // EPI_GLU: what a gate and an up entry become
 };
 
 // The copies of one stage (activations, weights, and for a split weight tile its second half) with, in front of them, a
@@ -289,7 +297,7 @@ __device__ __noinline__ void sincos_once(float angle, float* sn, float* cs) { si
 template <int BN, int EPI, typename TC>
 __global__ void __launch_bounds__(tile_threads(BN, EPI), 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, GemmTcParams p) {
-    constexpr int NUM_ACC = EPI == EPI_SWIGLU ? 2 : 1;   // accumulators = A tiles per stage (gate rows, up rows)
+    constexpr int NUM_ACC = is_gated(EPI) ? 2 : 1;   // accumulators = A tiles per stage (gate rows, up rows)
     constexpr int B_TILE_BYTES = BN * BLOCK_K * 2;
     constexpr int STAGE_BYTES = NUM_ACC * A_TILE_BYTES + B_TILE_BYTES;
     constexpr int ACC_COLS = NUM_ACC * BN;
@@ -441,7 +449,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
         // In the fold a warp owns a column (a token) and a lane four neighbouring rows (features): 16-byte loads from the
         // ranks' shared memory, a column's 128 features inside one warp (sums of squares and rotation partners need
         // no barrier), the four warps on four columns at a time, FOLD_COLS of each warp's columns in flight.
-        constexpr int FOLD_COLS = (EPI == EPI_SWIGLU || BN < 64) ? 1 : 2;   // (narrow tiles: a warp rarely has a second column, and the registers are worth more)
+        constexpr int FOLD_COLS = (is_gated(EPI) || BN < 64) ? 1 : 2;   // (narrow tiles: a warp rarely has a second column, and the registers are worth more)
         const int n4 = a_row0 + 4 * lane;                      // this lane's first feature in the fold
         int c_begin = 0, c_end = 0;
         float4 old_first[FOLD_COLS];
@@ -516,7 +524,6 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
             }
         };
 
-        const bool plain_glu = p.glu.kind == GLU_SILU && !p.glu.bias;
         // one chunk of CH accumulator columns: g (and u for SwiGLU) -> C
         auto emit = [&](int c, const float* g, const float* u) {
             const int n = a_row0 + row;                    // output feature
@@ -537,7 +544,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 const float r = scaled ? scale_s[c + j] : 1.0f;
                 if (EPI == EPI_STORE) *dst = from_float<TC>(g[j] * r);
                 else if (EPI == EPI_ACCUMULATE) *dst = from_float<TC>(old[j] + g[j]);
-                else *dst = from_float<TC>(plain_glu ? silu_mul(g[j] * r, u[j] * r) : glu_at(p.glu, g[j] * r, u[j] * r, n, p.N));
+                else *dst = from_float<TC>(gated_at<EPI>(p.glu, g[j] * r, u[j] * r, n, p.N));
             }
         };
 
@@ -546,7 +553,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 for (int c = 0; c < OUT_COLS; c += CH) {
                     float g[CH], u[CH];
                     acc_load(c, g);
-                    if (EPI == EPI_SWIGLU) acc_load(BN + c, u);
+                    if (is_gated(EPI)) acc_load(BN + c, u);
                     emit(c, g, u);
                 }
             }
@@ -591,7 +598,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                             const int c = c0 + 4 * q;
                             const bool in = r < p.splits && c < c_end;
                             pg[q][r] = in ? ld_cluster_f32x4(tiles + (c * TILE_M + 4 * lane) * 4, r) : make_float4(0.f, 0.f, 0.f, 0.f);
-                            pu[q][r] = (in && EPI == EPI_SWIGLU) ? ld_cluster_f32x4(tiles + ((BN + c) * TILE_M + 4 * lane) * 4, r)
+                            pu[q][r] = (in && is_gated(EPI)) ? ld_cluster_f32x4(tiles + ((BN + c) * TILE_M + 4 * lane) * 4, r)
                                                                   : make_float4(0.f, 0.f, 0.f, 0.f);
                         }
 #pragma unroll
@@ -667,11 +674,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                                 for (int i = 0; i < 4; i++) o[i] = n4 + i < p.N ? to_float(dst[i]) + gv[i] : 0.f;
                             }
                         } else {
-if constexpr (EPI == EPI_SWIGLU) glu_pack<4>(p.glu, gv, uv, o, n4, p.N);
-                            else {
 #pragma unroll
-                                for (int i = 0; i < 4; i++) o[i] = gv[i];
-                            }
+                            for (int i = 0; i < 4; i++) o[i] = EPI == EPI_STORE ? gv[i] : gated_at<EPI>(p.glu, gv[i], uv[i], n4 + i, p.N);
                         }
                         if (c_vec) {
                             if constexpr (sizeof(TC) == 4) *reinterpret_cast<float4*>(dst) = make_float4(o[0], o[1], o[2], o[3]);
@@ -748,7 +752,7 @@ if constexpr (EPI == EPI_SWIGLU) glu_pack<4>(p.glu, gv, uv, o, n4, p.N);
                                 const int c = c0 + 4 * q;
                                 const bool in = in_s && c < col_end;
                                 pg[k][q] = in ? __ldcg(reinterpret_cast<const float4*>(part + (size_t)c * TILE_M)) : make_float4(0.f, 0.f, 0.f, 0.f);
-                                pu[k][q] = (in && EPI == EPI_SWIGLU) ? __ldcg(reinterpret_cast<const float4*>(part + (size_t)(BN + c) * TILE_M))
+                                pu[k][q] = (in && is_gated(EPI)) ? __ldcg(reinterpret_cast<const float4*>(part + (size_t)(BN + c) * TILE_M))
                                                                       : make_float4(0.f, 0.f, 0.f, 0.f);
                             }
                         }
@@ -770,8 +774,7 @@ if constexpr (EPI == EPI_SWIGLU) glu_pack<4>(p.glu, gv, uv, o, n4, p.N);
                         float o[4];
 #pragma unroll
                         for (int i = 0; i < 4; i++)
-                            o[i] = EPI == EPI_STORE ? gv[i] * r : EPI == EPI_ACCUMULATE ? gv[i] : plain_glu ? silu_mul(gv[i] * r, uv[i] * r)
-                                 : n0 + i < p.N ? glu_at(p.glu, gv[i] * r, uv[i] * r, n0 + i, p.N) : 0.f;
+                            o[i] = EPI == EPI_STORE ? gv[i] * r : EPI == EPI_ACCUMULATE ? gv[i] : gated_at<EPI>(p.glu, gv[i] * r, uv[i] * r, n0 + i, p.N);
                         if (whole && (((uintptr_t)dst) & (4 * sizeof(TC) - 1)) == 0) {
                             if constexpr (sizeof(TC) == 4) {
                                 float4 v = make_float4(o[0], o[1], o[2], o[3]);
@@ -866,7 +869,7 @@ __global__ void __launch_bounds__(NUM_THREADS, 1)
 gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, GemmTcParams p) {
     // BN is the widest tile (the accumulators lie BN columns apart); the width in use comes with the launch, chosen so
     // that the tiles fill whole waves of SMs
-    constexpr bool SPLIT_B = EPI == EPI_SWIGLU;
+    constexpr bool SPLIT_B = is_gated(EPI);
     const int bn = p.bn;
     const int B_TILE_BYTES = bn * BLOCK_K * 2;
     const int STAGE_BYTES = A_TILE_BYTES + B_TILE_BYTES;
@@ -1040,7 +1043,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __gri
             for (int c = c_begin; c < c_end; c += 16) {
                 float g[16], u[16];
                 tmem_load<16>(lane_addr + c, g);
-                if (EPI == EPI_SWIGLU) tmem_load<16>(lane_addr + bn / 2 + c, u);
+                if (is_gated(EPI)) tmem_load<16>(lane_addr + bn / 2 + c, u);
                 if (m >= p.T) continue;
                 const int n0 = b_row0 + c;
                 if (n0 >= p.N) continue;
@@ -1050,14 +1053,10 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __gri
 #pragma unroll
                 for (int j8 = 0; j8 < 16; j8 += 8) {
                     float o[8];
-                    if constexpr (EPI == EPI_SWIGLU) {
 #pragma unroll
-                        for (int q = 0; q < 8; q++) { g[j8 + q] *= row_scale; u[j8 + q] *= row_scale; }
-                        glu_pack<8>(p.glu, g + j8, u + j8, o, n0 + j8, p.N);
-                    } else {
-#pragma unroll
-                        for (int q = 0; q < 8; q++) o[q] = EPI == EPI_STORE ? g[j8 + q] * row_scale : g[j8 + q];
-                    }
+                    for (int q = 0; q < 8; q++)
+                        o[q] = is_gated(EPI) ? gated_at<EPI>(p.glu, g[j8 + q] * row_scale, u[j8 + q] * row_scale, n0 + j8 + q, p.N)
+                             : EPI == EPI_STORE ? g[j8 + q] * row_scale : g[j8 + q];
                     if (EPI == EPI_STORE && p.act == 1) {
 #pragma unroll
                         for (int q = 0; q < 8; q++) { const float z = fmaxf(o[q], 0.f); o[q] = z * z; }
@@ -1156,12 +1155,15 @@ int launch(const CUtensorMap& ma, const CUtensorMap& mb, const GemmTcParams& p, 
     return hymt2_check_launch("gemm_tc");
 }
 
+inline bool plain_rule(const GluRule& r) { return r.kind == GLU_SILU && !r.bias; }
+
 template <int BN>
 int dispatch_epilogue(const CUtensorMap& ma, const CUtensorMap& mb, const GemmTcParams& p, dim3 grid, size_t smem,
                       int epilogue, int c_dtype, cudaStream_t stream) {
     if (epilogue == EPI_STORE && c_dtype == HYMT2_BF16) return launch<BN, EPI_STORE, __nv_bfloat16>(ma, mb, p, grid, smem, stream);
     if (epilogue == EPI_STORE && c_dtype == HYMT2_F32) return launch<BN, EPI_STORE, float>(ma, mb, p, grid, smem, stream);
     if (epilogue == EPI_ACCUMULATE && c_dtype == HYMT2_F32) return launch<BN, EPI_ACCUMULATE, float>(ma, mb, p, grid, smem, stream);
+    if (epilogue == EPI_SWIGLU && c_dtype == HYMT2_BF16 && !plain_rule(p.glu)) return launch<BN, EPI_GLU, __nv_bfloat16>(ma, mb, p, grid, smem, stream);
     if (epilogue == EPI_SWIGLU && c_dtype == HYMT2_BF16) return launch<BN, EPI_SWIGLU, __nv_bfloat16>(ma, mb, p, grid, smem, stream);
     hymt2_set_error("gemm_tc: epilogue %d with output type %d is not built", epilogue, c_dtype);
     return HYMT2_ERR_ARGUMENT;
@@ -1280,6 +1282,7 @@ int launch_persistent(const CUtensorMap& ma, const CUtensorMap& mb, const GemmTc
     if (epilogue == EPI_STORE && c_dtype == HYMT2_BF16) return launch_persistent_one<PERSISTENT_BN, EPI_STORE, __nv_bfloat16>(ma, mb, p, ctas, pl.smem, stream);
     if (epilogue == EPI_STORE && c_dtype == HYMT2_F32) return launch_persistent_one<PERSISTENT_BN, EPI_STORE, float>(ma, mb, p, ctas, pl.smem, stream);
     if (epilogue == EPI_ACCUMULATE && c_dtype == HYMT2_F32) return launch_persistent_one<PERSISTENT_BN, EPI_ACCUMULATE, float>(ma, mb, p, ctas, pl.smem, stream);
+    if (epilogue == EPI_SWIGLU && c_dtype == HYMT2_BF16 && !plain_rule(p.glu)) return launch_persistent_one<PERSISTENT_BN, EPI_GLU, __nv_bfloat16>(ma, mb, p, ctas, pl.smem, stream);
     if (epilogue == EPI_SWIGLU && c_dtype == HYMT2_BF16) return launch_persistent_one<PERSISTENT_BN, EPI_SWIGLU, __nv_bfloat16>(ma, mb, p, ctas, pl.smem, stream);
     hymt2_set_error("gemm_tc: epilogue %d with output type %d is not built", epilogue, c_dtype);
     return HYMT2_ERR_ARGUMENT;
